@@ -3,6 +3,7 @@
 // fallback: without a usable GPU ainfer_device_open fails.
 #include "../../../include/ainfer_cuda.h"
 
+#include <cuda.h>
 #include <cuda_runtime.h>
 #include <time.h>
 
@@ -328,6 +329,33 @@ int ainfer_memcpy_h2d_async(ainfer_device_t dev, void *dst, const void *src, siz
 int ainfer_memcpy_d2h_async(ainfer_device_t dev, void *dst, const void *src, size_t bytes) {
   if (!dev) return AINFER_ERR_INVALID;
   CU(dev, cudaMemcpyAsync(dst, src, bytes, cudaMemcpyDeviceToHost, dev->stream));
+  return AINFER_OK;
+}
+
+int ainfer_tensor_map_bf16(ainfer_device_t dev, void *map128, const void *base, uint64_t rows, uint64_t cols, uint64_t ld,
+                           uint32_t box_rows) {
+  if (!dev || !map128 || !base) return AINFER_ERR_INVALID;
+  if (((uintptr_t)base & 15u) || ld % 8 || ld < cols || rows == 0 || cols == 0 || box_rows == 0 || box_rows > 256)
+    return fail(dev, AINFER_ERR_INVALID, "tensor map: base must be 16-byte aligned, ld a multiple of 8 and at least cols, 1..256 box rows");
+  typedef CUresult (*EncodeFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
+                               const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion,
+                               CUtensorMapFloatOOBfill);
+  static EncodeFn encode = nullptr;
+  if (!encode) {
+    void *fn = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    CU(dev, cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q));
+    if (q != cudaDriverEntryPointSuccess || !fn) return fail(dev, AINFER_ERR_DEVICE, "cuTensorMapEncodeTiled is not available");
+    encode = (EncodeFn)fn;
+  }
+  alignas(64) CUtensorMap m;
+  const cuuint64_t dims[2] = {cols, rows}, strides[1] = {ld * 2};
+  const cuuint32_t box[2] = {64, box_rows}, step[2] = {1, 1};
+  const CUresult r = encode(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, step,
+                            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) return fail(dev, AINFER_ERR_DEVICE, "cuTensorMapEncodeTiled failed (" + std::to_string((int)r) + ")");
+  std::memcpy(map128, &m, sizeof m);
   return AINFER_OK;
 }
 

@@ -1,0 +1,250 @@
+// LinearTc: Y[r][n] = act(sum_k X[r][k] W[n][k] + bias[n]) for many rows, bf16 operands, fp32 sums, on
+// the 5th-generation tensor cores: operands by TMA (128-byte swizzle) into a ring of stages, products
+// by tcgen05.mma kind::f16 with the weights as the M operand (128 output features per tile) and the
+// activation rows as the N operand (`nt` of them, 16..256), accumulators in tensor memory, two buffers,
+// so that a tile's epilogue overlaps the next tile's products.
+//
+// One block per SM walks (tile, split) units. Roles: warp 0 lane 0 issues the copies, warp 1 lane 0 the
+// products, warps 4..7 read the accumulators (a lane = one output feature, so a warp stores 32
+// consecutive features of a row at a time). With splits > 1 a unit covers a share of K: it leaves fp32
+// partials, and the last unit of a tile to finish adds them in split order and applies the epilogue.
+//
+// Every wait is bounded: one that runs out stores a code in the host-visible fault word, after which
+// the block's other waits return at once and the kernel ends (copies in flight awaited, tensor memory
+// freed).
+#include <cuda.h>
+
+#include "weight_ring.cuh"
+
+namespace ainfer {
+
+struct LinearTcArgs {
+  CUtensorMap Wm;        // [N][K], box 64 x 128
+  CUtensorMap Xm;        // [rows][K], box 64 x nt
+  const float *Bias;     // [N] or null
+  void *Y;               // [rows][ldy]
+  float *Part;           // [splits][tiles][nt][128] when splits > 1
+  uint32_t *Count;       // [tiles], zero between launches
+  int32_t rows, N, K, nt, ldy, act, out16, splits;
+  float cap;
+};
+
+constexpr int kLtThreads = 256, kLtBudget = 200 * 1024;
+constexpr uint32_t kLtSpin = 1u << 22;
+__host__ __device__ inline uint32_t lt_stage_bytes(int nt) { return (128u + (uint32_t)nt) * 128u; }
+__host__ __device__ inline uint32_t lt_stages(int nt) {
+  const uint32_t s = (uint32_t)kLtBudget / lt_stage_bytes(nt);
+  return s > 8 ? 8 : s;
+}
+
+__device__ __forceinline__ uint64_t lt_desc(uint32_t addr) {
+  // K-major operand, 128-byte swizzle: rows of 128 bytes in groups of eight (1024 bytes apart)
+  return (uint64_t)((addr >> 4) & 0x3FFFu) | (1ull << 16) | ((uint64_t)(1024u >> 4) << 32) | (1ull << 46) | (2ull << 61);
+}
+__device__ __forceinline__ void lt_mma(uint32_t d, uint64_t da, uint64_t db, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(d), "l"(da), "l"(db), "r"(idesc), "r"(acc)
+      : "memory");
+}
+__device__ __forceinline__ void lt_commit(uint32_t bar) {
+  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+__device__ __forceinline__ void lt_tma(uint32_t dst, const CUtensorMap *m, uint32_t bar, int x, int y) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];" ::"r"(dst),
+               "l"(reinterpret_cast<uint64_t>(m)), "r"(bar), "r"(x), "r"(y)
+               : "memory");
+}
+__device__ __forceinline__ void lt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]), "=r"(v[10]),
+        "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+      : "r"(taddr)
+      : "memory");
+}
+
+struct LtShared {
+  unsigned long long full[8], empty[8], acc_full[2], acc_empty[2], drain;
+  uint32_t tmem, fail, last;
+};
+__device__ __forceinline__ bool lt_wait(LtShared *s, unsigned long long *b, uint32_t parity) {
+  if (mbar_try(b, parity)) return true;
+  for (uint32_t i = 0; i < kLtSpin; ++i) {
+    if (mbar_try(b, parity)) return true;
+    if (*reinterpret_cast<volatile uint32_t *>(&s->fail)) return false;
+  }
+  *reinterpret_cast<volatile uint32_t *>(&s->fail) = 1;
+  if (g_stream_fault_word) *reinterpret_cast<volatile unsigned int *>(g_stream_fault_word) = 1;
+  return false;
+}
+
+__device__ __forceinline__ float lt_act(float v, int act, float cap) {
+  if (act == 1) { v = v > 0.0f ? v : 0.0f; return v * v; }
+  if (act == 2) return cap * tanhf(v / cap);
+  return v;
+}
+
+__global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant__ LinearTcArgs a) {
+  extern __shared__ __align__(1024) unsigned char lt_smem_raw[];
+  __shared__ LtShared sh;
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t base = (smem_addr(lt_smem_raw) + 1023u) & ~1023u;
+  const int nt = a.nt, nst = (int)lt_stages(nt);
+  const uint32_t stage_bytes = lt_stage_bytes(nt);
+  const int n_tiles = (a.N + 127) / 128, r_tiles = (a.rows + nt - 1) / nt, tiles = n_tiles * r_tiles;
+  const int units = tiles * a.splits, kb = (a.K + 63) / 64;
+  uint32_t cols = 32;
+  while (cols < 2u * (uint32_t)nt) cols <<= 1;
+  if (tid == 0) {
+    for (int i = 0; i < nst; ++i) { mbar_init(&sh.full[i], 1); mbar_init(&sh.empty[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&sh.acc_full[i], 1); mbar_init(&sh.acc_empty[i], 128); }
+    mbar_init(&sh.drain, 1);
+    sh.fail = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&a.Wm)) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&a.Xm)) : "memory");
+  }
+  if (warp == 2) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_addr(&sh.tmem)), "r"(cols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+  const uint32_t tmem = sh.tmem;
+  pdl_wait();
+
+  if (warp == 0 && lane == 0) {
+    // ---- copies ----
+    uint32_t st = 0, ph = 1, issued = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x) {
+      const int tile = u % tiles, sp = u / tiles;
+      const int n0 = (tile % n_tiles) * 128, r0 = (tile / n_tiles) * nt;
+      const int k_lo = kb * sp / a.splits, k_hi = kb * (sp + 1) / a.splits;
+      for (int k = k_lo; k < k_hi; ++k) {
+        if (!lt_wait(&sh, &sh.empty[st], ph)) break;
+        const uint32_t dst = base + st * stage_bytes, bar = smem_addr(&sh.full[st]);
+        mbar_arrive_expect(&sh.full[st], stage_bytes);
+        lt_tma(dst, &a.Wm, bar, k * 64, n0);
+        lt_tma(dst + 128u * 128u, &a.Xm, bar, k * 64, r0);
+        ++issued;
+        if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
+      }
+      if (*reinterpret_cast<volatile uint32_t *>(&sh.fail)) break;
+    }
+    if (*reinterpret_cast<volatile uint32_t *>(&sh.fail)) {
+      // await every copy still in flight (each stage's last use) before the block may end
+      for (int i = 0; i < nst && (uint32_t)i < issued; ++i) {
+        const uint32_t uses = (issued - (uint32_t)i + (uint32_t)nst - 1) / (uint32_t)nst;
+        for (uint32_t s = 0; s < kLtSpin && !mbar_try(&sh.full[i], (uses - 1) & 1); ++s) {}
+      }
+    }
+  } else if (warp == 1 && lane == 0) {
+    // ---- products ----
+    const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nt >> 3) << 17) | ((128u >> 4) << 24);
+    uint32_t st = 0, ph = 0, buf = 0, aph = 1;
+    for (int u = blockIdx.x; u < units; u += gridDim.x) {
+      const int sp = u / tiles;
+      const int k_lo = kb * sp / a.splits, k_hi = kb * (sp + 1) / a.splits;
+      if (!lt_wait(&sh, &sh.acc_empty[buf], aph)) break;
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const uint32_t d = tmem + buf * (uint32_t)nt;
+      bool ok = true;
+      for (int k = k_lo; k < k_hi; ++k) {
+        ok = lt_wait(&sh, &sh.full[st], ph);
+        if (!ok) break;
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        const uint64_t da = lt_desc(base + st * stage_bytes), db = lt_desc(base + st * stage_bytes + 128u * 128u);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) lt_mma(d, da + (uint64_t)(2 * q), db + (uint64_t)(2 * q), idesc, k > k_lo || q > 0 ? 1u : 0u);
+        lt_commit(smem_addr(&sh.empty[st]));
+        if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
+      }
+      if (!ok) break;
+      lt_commit(smem_addr(&sh.acc_full[buf]));
+      if (++buf == 2) { buf = 0; aph ^= 1; }
+    }
+    if (*reinterpret_cast<volatile uint32_t *>(&sh.fail)) {   // await the products already issued
+      lt_commit(smem_addr(&sh.drain));
+      for (uint32_t s = 0; s < kLtSpin && !mbar_try(&sh.drain, 0); ++s) {}
+    }
+  } else if (warp >= 4) {
+    // ---- epilogue ----
+    const int lw = (warp & 3) * 32 + lane;
+    uint32_t buf = 0, ph = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x) {
+      const int tile = u % tiles, sp = u / tiles;
+      const int n = (tile % n_tiles) * 128 + lw, r0 = (tile / n_tiles) * nt, nr = min(nt, a.rows - r0);
+      const float bias = a.Bias && n < a.N ? a.Bias[n] : 0.0f;
+      // after a failed wait the unit's values are garbage, but the four warps still meet at their barriers
+      lt_wait(&sh, &sh.acc_full[buf], ph);
+      __syncwarp();
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const uint32_t taddr = tmem + buf * (uint32_t)nt + ((uint32_t)((warp & 3) * 32) << 16);
+      auto emit = [&](int r, float v) {
+        if (n >= a.N) return;
+        v = lt_act(v + bias, a.act, a.cap);
+        const size_t o = (size_t)(r0 + r) * a.ldy + n;
+        if (a.out16) reinterpret_cast<uint16_t *>(a.Y)[o] = f32_to_bf16(v);
+        else reinterpret_cast<float *>(a.Y)[o] = v;
+      };
+      float *part = a.splits > 1 ? a.Part + ((size_t)sp * tiles + tile) * nt * 128 + lw : nullptr;
+      for (int c = 0; c < nt; c += 16) {
+        if (c >= nr) break;
+        uint32_t v[16];
+        lt_ld16(taddr + (uint32_t)c, v);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        if (part) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            if (c + i < nr) __stcg(part + (size_t)(c + i) * 128, __uint_as_float(v[i]));
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            if (c + i < nr) emit(c + i, __uint_as_float(v[i]));
+        }
+      }
+      asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      mbar_arrive(&sh.acc_empty[buf]);
+      if (++buf == 2) { buf = 0; ph ^= 1; }
+      if (part) {
+        __threadfence();
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (tid == 128) {
+          const uint32_t c = atomicAdd(a.Count + tile, 1u);
+          sh.last = c + 1 == (uint32_t)a.splits;
+          if (sh.last) a.Count[tile] = 0;
+        }
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (sh.last) {
+          __threadfence();
+          const float *p0 = a.Part + (size_t)tile * nt * 128 + lw;
+          const size_t stride = (size_t)tiles * nt * 128;
+          for (int r = 0; r < nr; ++r) {
+            float v = 0.0f;
+            for (int s = 0; s < a.splits; ++s) v += __ldcg(p0 + (size_t)s * stride + (size_t)r * 128);
+            emit(r, v);
+          }
+        }
+      }
+    }
+  }
+  __syncwarp();
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
+}
+static uint32_t linear_tc_smem(const void *args) {
+  const int nt = ((const LinearTcArgs *)args)->nt;
+  return lt_stages(nt) * lt_stage_bytes(nt) + 1024;
+}
+#define F(f) AINFER_ARG(LinearTcArgs, f)
+AINFER_REGISTER(LinearTc, LinearTcArgs, kLtThreads, 0, 0, linear_tc_smem, F(Wm), F(Xm), F(Bias), F(Y), F(Part), F(Count), F(rows), F(N), F(K),
+                F(nt), F(ldy), F(act), F(out16), F(splits), F(cap));
+#undef F
+
+AINFER_EARLY_LAUNCH(LinearTc);
+
+}  // namespace ainfer

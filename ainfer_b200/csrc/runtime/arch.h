@@ -1,0 +1,57 @@
+// Architectures the runtime serves. A model names its architecture in its configuration; the loader
+// (model.cpp) and the block executor (executor.cpp, prefill.cpp, batch.cpp) look it up here and call
+// what differs between architectures through these tables. The token loop, control block, prompt
+// passes, sampler, batch interface, command line and server are common to all.
+#pragma once
+#include <string>
+#include <vector>
+
+#include "launcher.h"
+#include "model.h"
+
+namespace ainfer {
+
+struct Session;
+struct Json;
+
+// Configuration and weights.
+struct ModelArch {
+  const char *name;
+  bool int4;                                                             // projection weights are INT4 g128 (else bf16)
+  bool (*parse)(const Json &js, ModelConfig &out, std::string &err);     // null: the flat INT4 form
+  std::string (*to_json)(const ModelConfig &c);
+  bool (*check)(const ModelConfig &c, std::string &err);
+  void (*plan)(const ModelConfig &c, Container &dir, std::vector<SynthSpec> &specs);
+  int (*check_directory)(const Container &dir, const ModelConfig &c, std::string &err);
+  int (*prepare)(DeviceModel *m, std::string &err);                      // after the weights are on the device
+};
+const ModelArch *model_arch(const std::string &name);                    // null: unknown
+
+// Rows of a prompt pass or of a batched step, as the architecture's row path sees them.
+struct RowSpan {
+  const int32_t *ctrl = nullptr, *seq = nullptr, *first = nullptr;   // device: [rows][4], [rows], [rows]
+  int rows = 0;
+  bool one_sequence = true;       // rows are consecutive positions of one sequence; else one row per sequence
+  const int32_t *want = nullptr;  // device: rows whose logits are asked for
+  int n_want = 0;
+  float *logits = nullptr;        // device: [n_want][vocab]
+};
+struct RowEngine {                // state of `nseq` sequences plus the buffers of a pass of `rows_cap` rows
+  virtual ~RowEngine() {}
+  virtual void emit(KernelCalls &k, const RowSpan &span) = 0;
+  virtual int reset(std::string &err) = 0;
+  virtual bool buffer(const std::string &which, void **dptr, uint64_t *bytes) = 0;
+  // one decode step of sequence 0 as recorded launches: embedding, one layer, final norm + head
+  virtual void record_embed(KernelCalls &k, const int32_t *ctrl) = 0;
+  virtual void record_layer(KernelCalls &k, int layer, const int32_t *ctrl) = 0;
+  virtual void record_head(KernelCalls &k, float *logits) = 0;
+  int rows_cap = 0;
+};
+// Creates the row engine of an architecture that has one. max_ctx: positions a sequence may reach;
+// f32: activations and cache in 32-bit. Returns 0, 1 (device) or 2 (usage).
+int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err);
+
+const ModelArch *sinepel_model_arch();
+const ModelArch *int4_hybrid_model_arch();
+
+}  // namespace ainfer

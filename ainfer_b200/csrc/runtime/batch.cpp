@@ -17,31 +17,9 @@
 namespace ainfer {
 
 namespace {
-struct Rec {   // appends launches to a list; arguments by index in member order
+struct Rec : KernelCalls {   // appends launches to a list; arguments by index in member order
   BatchDecode *b;
-  ainfer_list_t list;
-  int status = 0;
-  template <typename T>
-  void set(ainfer_kernel_t k, uint32_t &idx, const T &v) {
-    if (status) return;
-    if (ainfer_kernel_set_arg(k, idx, sizeof(T), &v) != AINFER_OK) { b->err = ainfer_last_error(b->dev); status = 1; }
-    ++idx;
-  }
-  template <typename... A>
-  void launch(const char *name, uint32_t groups, const A &...args) {
-    if (status) return;
-    ainfer_kernel_t k = nullptr;
-    auto it = b->kernels.find(name);
-    if (it != b->kernels.end()) k = it->second;
-    else {
-      if (ainfer_kernel_get(b->dev, name, &k) != AINFER_OK) { b->err = std::string("entry ") + name + " not found"; status = 1; return; }
-      b->kernels[name] = k;
-    }
-    uint32_t idx = 0;
-    (set(k, idx, args), ...);
-    if (status) return;
-    if (ainfer_list_append_launch(list, k, groups ? groups : 1) != AINFER_OK) { b->err = ainfer_last_error(b->dev); status = 1; }
-  }
+  Rec(BatchDecode *bd, ainfer_list_t l) : KernelCalls(bd->dev, &bd->kernels, &bd->err, l), b(bd) {}
   void gemm(const DeviceTensor &t, const int8_t *XQ, const float *SQ, float *Y, int K, int rows) {
     if (status) return;
     if (!t.entry || (int)t.entry->shape[1] != K || t.entry->storage != DT_INT4_SYM_G128) {
@@ -92,6 +70,8 @@ int BatchDecode::create(DeviceModel *model, const void *id128, int rank, int wor
   max_ctx = max_ctx_;
   const ModelConfig &c = m->cfg;
   if (batch < world || batch % world || max_ctx < 1) { err = "usage: the batch must divide over the ranks"; return 2; }
+  if (m->rows) return create_rows(batch / world, (flags & BATCH_F32) != 0);
+  if (flags & BATCH_F32) { err = "usage: this architecture computes on INT8 activations and has no 32-bit form"; return 2; }
   const int ratio = c.kv_heads ? c.q_heads / c.kv_heads : 0;
   if (c.head_dim != 256 || !(ratio == 1 || ratio == 2 || ratio == 4 || ratio == 6 || ratio == 8)) { err = "usage: unsupported attention shape"; return 2; }
   n = batch / world;
@@ -127,6 +107,37 @@ int BatchDecode::create(DeviceModel *model, const void *id128, int rank, int wor
   return record();
 }
 
+// Architectures with a row engine: a step is one recorded list over the owned sequences (no exchange
+// between ranks: every rank decodes its own sequences).
+int BatchDecode::create_rows(int owned, bool f32) {
+  const ModelConfig &c = m->cfg;
+  n = owned;
+  max_ctx = std::min(max_ctx, c.max_positions);
+  int r = row_engine_create(m, n, max_ctx, n, f32, &rows, err);
+  if (r) return r;
+  int32_t *seq = nullptr;   // row = sequence = first row of its sequence = row whose logits are wanted
+  r |= alloc(&Ctrl, (size_t)n * 4); r |= alloc(&OutT, (size_t)n); r |= alloc(&Logits, (size_t)n * c.vocab); r |= alloc(&seq, (size_t)n);
+  if (r) return 1;
+  std::vector<int32_t> id((size_t)n);
+  for (int i = 0; i < n; ++i) id[(size_t)i] = i;
+  if (ainfer_memcpy_h2d(dev, seq, id.data(), id.size() * 4) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
+  ainfer_list_t l = nullptr;
+  if (ainfer_list_create(dev, &l) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
+  lists.push_back(l);
+  tail_list = l;
+  Rec rec(this, l);
+  RowSpan span;
+  span.ctrl = Ctrl; span.seq = span.first = span.want = seq;
+  span.rows = span.n_want = n;
+  span.one_sequence = false;
+  span.logits = Logits;
+  rows->emit(rec, span);
+  rec.launch("BatchArgmax", (uint32_t)n, (const float *)Logits, OutT, Ctrl, (int32_t)c.vocab, (int32_t)1);
+  if (rec.status) return rec.status;
+  if (ainfer_list_close(l) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
+  return 0;
+}
+
 int BatchDecode::record() {
   const ModelConfig &c = m->cfg;
   const int H = c.hidden, C = c.conv_dim(), VD = c.value_dim(), nK = c.lin_k_heads, nV = c.lin_v_heads;
@@ -149,14 +160,14 @@ int BatchDecode::record() {
   if (new_list(&l)) return 1;
   embed_list = l;
   {
-    Rec r{this, l};
+    Rec r(this, l);
     r.launch("EmbedRow", (uint32_t)n, X, (const uint16_t *)emb.data, (const int32_t *)Ctrl, (int32_t)H, (int32_t)c.vocab, (int32_t)4);
     if (int e = close(r)) return e;
   }
   for (int L = 0; L < c.layers; ++L) {
     if (new_list(&l)) return 1;
     layer_lists.push_back(l);
-    Rec r{this, l};
+    Rec r(this, l);
     const std::string pf = layer_prefix(L);
     const int slot = m->slot[L];
     r.launch("RmsNormQuant", (uint32_t)n, (const float *)X, (const float *)nullptr, (float *)nullptr,
@@ -198,7 +209,7 @@ int BatchDecode::record() {
   if (new_list(&l)) return 1;
   tail_list = l;
   {
-    Rec r{this, l};
+    Rec r(this, l);
     r.launch("RmsNormQuant", (uint32_t)n, (const float *)X, (const float *)nullptr, (float *)nullptr, (const float *)m->final_norm,
              (float *)nullptr, Q8, SQ, (int32_t)H, eps);
     r.gemm(m->tensor("lm_head.weight"), Q8, SQ, Logits, H, n);
@@ -209,6 +220,10 @@ int BatchDecode::record() {
 }
 
 int BatchDecode::step() {
+  if (rows) {
+    if (ainfer_list_execute(tail_list) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
+    return 0;
+  }
   if (ainfer_list_execute(embed_list) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
   for (int L = 0; L < m->cfg.layers; ++L) {
     if (ainfer_list_execute(layer_lists[L]) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
@@ -228,6 +243,8 @@ void BatchDecode::destroy() {
   ep_ready = false;
   for (auto &kv : kernels) ainfer_kernel_release(kv.second);
   kernels.clear();
+  delete rows;
+  rows = nullptr;
   for (void *q : owned) ainfer_mem_free(dev, q);
   owned.clear();
 }

@@ -4,13 +4,17 @@
 #include <string>
 #include <vector>
 
+#include "arch.h"
 #include "ep.h"
 #include "model.h"
 #include "row_slabs.h"
 
 namespace ainfer {
 
+enum BatchFlags { BATCH_F32 = 32 };   // activations and cache in 32-bit (architectures with a row engine)
+
 struct BatchDecode {
+  RowEngine *rows = nullptr;   // architectures with a row engine: state and row buffers of the sequences
   DeviceModel *m = nullptr;
   ainfer_device_t dev = nullptr;
   std::string err;
@@ -44,6 +48,7 @@ struct BatchDecode {
   template <typename T>
   int alloc(T **p, size_t count);
   int record();
+  int create_rows(int owned, bool f32);
 };
 
 }  // namespace ainfer

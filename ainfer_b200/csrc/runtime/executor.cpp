@@ -7,67 +7,22 @@
 
 #include "../common/step_plan.h"
 #include "../common/tables.h"
+#include "arch.h"
 
 namespace ainfer {
 
 namespace {
 
 // ---- recording helpers ----------------------------------------------------
-struct Recorder {
+struct Recorder : KernelCalls {
   Session *s;
-  ainfer_list_t list;
-  int status = 0;
   // Residual stream and control block the recorded layer works on: the trunk's by default,
   // the MTP head's own when its list is recorded.
   float *x_override = nullptr;
   int32_t *ctrl_override = nullptr;
+  explicit Recorder(Session *session) : KernelCalls(session->dev, &session->kernels, &session->err), s(session) {}
   float *X() const { return x_override ? x_override : s->X; }
   int32_t *ctrl() const { return ctrl_override ? ctrl_override : s->ctrl; }
-
-  ainfer_kernel_t kernel(const char *name) {
-    auto it = s->kernels.find(name);
-    if (it != s->kernels.end()) return it->second;
-    ainfer_kernel_t k = nullptr;
-    if (ainfer_kernel_get(s->dev, name, &k) != AINFER_OK) {
-      s->err = std::string("entry ") + name + " not found";
-      status = 1;
-      return nullptr;
-    }
-    s->kernels[name] = k;
-    return k;
-  }
-  template <typename T>
-  void set(ainfer_kernel_t k, uint32_t &idx, const T &v) {
-    if (status) return;
-    if (ainfer_kernel_set_arg(k, idx, sizeof(T), &v) != AINFER_OK) {
-      s->err = ainfer_last_error(s->dev);
-      status = 1;
-    }
-    ++idx;
-  }
-  // Appends one launch; arguments are set by index in the order given, which is
-  // the member order of the kernel's argument struct.
-  template <typename... A>
-  void launch(const char *name, uint32_t groups, const A &...args) {
-    if (status) return;
-    ainfer_kernel_t k = kernel(name);
-    if (!k) return;
-    uint32_t idx = 0;
-    (set(k, idx, args), ...);
-    if (status) return;
-    if (ainfer_list_append_launch(list, k, groups ? groups : 1) != AINFER_OK) {
-      s->err = std::string("append failed: ") + ainfer_last_error(s->dev);
-      status = 1;
-    }
-    s->launches_per_token += 1;
-  }
-  void copy(void *dst, const void *src, size_t bytes) {
-    if (status) return;
-    if (ainfer_list_append_memcpy(list, dst, src, bytes) != AINFER_OK) {
-      s->err = std::string("append failed: ") + ainfer_last_error(s->dev);
-      status = 1;
-    }
-  }
 };
 
 // Thread groups for a weight-streaming launch: a group should own at least one
@@ -249,12 +204,20 @@ void record_attn_layer(Recorder &r, int L, const std::string &p) {
 }
 
 void record_layer(Recorder &r, int L) {
+  if (r.s->rows) {
+    r.s->rows->record_layer(r, L, r.s->ctrl);
+    return;
+  }
   if (r.s->m->cfg.layer_types[L] == 'A') record_attn_layer(r, L, layer_prefix(L));
   else record_linear_layer(r, L);
 }
 
 void record_embed(Recorder &r) {
   Session *s = r.s;
+  if (s->rows) {
+    s->rows->record_embed(r, s->ctrl);
+    return;
+  }
   DeviceTensor emb = s->m->tensor("model.language_model.embed_tokens.weight");
   if (!emb.entry) { s->err = "missing model.language_model.embed_tokens.weight"; r.status = 1; return; }
   r.launch("EmbedRow", 1, s->X, (const uint16_t *)emb.data, (const int32_t *)s->ctrl,
@@ -266,11 +229,15 @@ void record_tail(Recorder &r, bool advance) {
   Session *s = r.s;
   DeviceModel *m = s->m;
   const ModelConfig &c = m->cfg;
-  r.launch("RmsNormQuant", 1, (const float *)s->X, (const float *)nullptr, (float *)nullptr,
-           (const float *)m->final_norm, (float *)nullptr, s->Q8, s->SQ, (int32_t)c.hidden,
-           (float)c.rms_eps);
-  record_gemv(r, {{m->tensor("lm_head.weight"), s->Logits, EPI_STORE, nullptr, nullptr, nullptr}},
-              c.hidden, s->Q8, s->SQ);
+  if (s->rows) {
+    s->rows->record_head(r, s->Logits);
+  } else {
+    r.launch("RmsNormQuant", 1, (const float *)s->X, (const float *)nullptr, (float *)nullptr,
+             (const float *)m->final_norm, (float *)nullptr, s->Q8, s->SQ, (int32_t)c.hidden,
+             (float)c.rms_eps);
+    record_gemv(r, {{m->tensor("lm_head.weight"), s->Logits, EPI_STORE, nullptr, nullptr, nullptr}},
+                c.hidden, s->Q8, s->SQ);
+  }
   r.launch("ArgmaxStage1", (uint32_t)s->argmax_parts, (const float *)s->Logits, s->PV, s->PI,
            (int32_t)c.vocab);
   r.launch("ArgmaxStage2", 1, (const float *)s->PV, (const int32_t *)s->PI, s->out_tok, s->ctrl,
@@ -479,8 +446,12 @@ int close_list(Session *s, ainfer_list_t l) {
 
 }  // namespace
 
+// Rows of a prompt pass of architectures with a row engine.
+constexpr int kRowEnginePassRows = 2048;
+
 int session_reset(Session *s) {
   const ModelConfig &c = s->m->cfg;
+  if (s->rows) return s->rows->reset(s->err);
   size_t n_kv = (size_t)(c.n_attn() + c.mtp_layers) * s->max_ctx * c.kv_heads;
   int r = 0;
   r |= ainfer_mem_fill(s->dev, s->conv, 0, std::max<size_t>((size_t)c.n_lin() * c.conv_dim() * 3 * 4, 16));
@@ -506,71 +477,84 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
   if (ainfer_device_get_info(s->dev, &info) != AINFER_OK) { s->err = ainfer_last_error(s->dev); return fail(1); }
   s->sm_count = info.sm_count;
   const ModelConfig &c = m->cfg;
+  const bool row_arch = m->rows != nullptr;
+  if (row_arch) {
+    // learned positions bound the context; the persistent step is the INT4 hybrid's, here a token is always a recorded list
+    s->max_ctx = max_ctx = std::min(max_ctx, c.max_positions);
+    s->flags = flags &= ~(SESSION_PERSISTENT | SESSION_STAGE_CLOCK | SESSION_DIAG);
+    const int e = row_engine_create(m, 1, max_ctx, std::min(max_ctx, kRowEnginePassRows), (flags & SESSION_F32) != 0, &s->rows, s->err);
+    if (e) return fail(e);
+  } else if (flags & SESSION_F32) {
+    s->err = "usage: this architecture computes on INT8 activations and has no 32-bit form";
+    return fail(2);
+  }
   const int H = c.hidden, D = c.head_dim, nQ = c.q_heads, nKV = c.kv_heads, nV = c.lin_v_heads;
   const int C = std::max(c.conv_dim(), 1), VD = std::max(c.value_dim(), 1);
   const int n_kv_layers = c.n_attn() + c.mtp_layers;
   s->max_chunks = (max_ctx + 63) / 64;
   s->argmax_parts = s->sm_count * 2;  // also the partial count of the persistent kernel (one per block)
-  if (model_ensure_rope(m, max_ctx, s->err)) return fail(1);
   int r = 0;
-  size_t n_kv = (size_t)n_kv_layers * max_ctx * nKV;
-  r |= salloc(s, (size_t)c.n_lin() * C * 3, &s->conv);
-  r |= salloc(s, (size_t)c.n_lin() * nV * 128 * 128, &s->S);
-  r |= salloc(s, n_kv * D, &s->Kc);
-  r |= salloc(s, n_kv * D, &s->Vc);
-  r |= salloc(s, n_kv, &s->Ks);
-  r |= salloc(s, n_kv, &s->Vs);
   r |= salloc(s, 4, &s->ctrl);
   r |= salloc(s, (size_t)max_ctx, &s->ids);
   r |= salloc(s, (size_t)max_ctx, &s->history);
   r |= salloc(s, 1, &s->out_tok);
-  r |= salloc(s, (size_t)H, &s->X);
-  r |= salloc(s, (size_t)H, &s->Tmp);
-  r |= salloc(s, (size_t)H, &s->Hn);
-  r |= salloc(s, (size_t)H, &s->Mix);
-  int maxK = std::max(std::max(2 * H, VD), nQ * D);
-  r |= salloc(s, (size_t)maxK, &s->Q8);
-  r |= salloc(s, (size_t)maxK / 128, &s->SQ);
-  r |= salloc(s, (size_t)C, &s->Mx);
-  r |= salloc(s, (size_t)VD, &s->Z);
-  r |= salloc(s, (size_t)std::max(nV, 1), &s->Bt);
-  r |= salloc(s, (size_t)std::max(nV, 1), &s->Gt);
-  r |= salloc(s, (size_t)VD, &s->O);
-  r |= salloc(s, (size_t)nQ * 2 * D, &s->Q16);
-  r |= salloc(s, (size_t)nKV * D, &s->K16);
-  r |= salloc(s, (size_t)nKV * D, &s->V16);
-  r |= salloc(s, (size_t)nQ * D, &s->Qn);
-  r |= salloc(s, (size_t)nQ * s->max_chunks, &s->Pm);
-  r |= salloc(s, (size_t)nQ * s->max_chunks, &s->Pse);
-  r |= salloc(s, (size_t)nQ * s->max_chunks * D, &s->Pacc);
-  r |= salloc(s, (size_t)c.experts + 1, &s->RLogits);
-  r |= salloc(s, 1, &s->Counter);
-  r |= salloc(s, (size_t)c.top_k + 1, &s->SelIdx);
-  r |= salloc(s, (size_t)c.top_k + 1, &s->SelRows);
-  r |= salloc(s, (size_t)c.top_k + 1, &s->SelW);
-  r |= salloc(s, 1, &s->NearGap);
-  r |= salloc(s, (size_t)(c.top_k + 1) * c.expert_inter, &s->Act);
   r |= salloc(s, (size_t)c.vocab, &s->Logits);
-  if (c.mtp_layers) {
-    r |= salloc(s, (size_t)H, &s->Xm);
-    r |= salloc(s, (size_t)H, &s->Hm);
-    r |= salloc(s, (size_t)2 * H, &s->Cat);
-    r |= salloc(s, (size_t)c.vocab, &s->LogitsM);
-    r |= salloc(s, 4, &s->ctrl_m);
-    r |= salloc(s, 1, &s->out_tok_m);
-  }
   r |= salloc(s, (size_t)s->argmax_parts, &s->PV);
   r |= salloc(s, (size_t)s->argmax_parts, &s->PI);
-  if (flags & SESSION_DIAG) {
-    r |= salloc(s, (size_t)c.layers * H, &s->layer_out);
-    r |= salloc(s, (size_t)c.layers * (c.top_k + 1), &s->routed);
-    r |= salloc(s, (size_t)c.layers, &s->near_gap);
-  }
-  s->gemv_tables_cap = (size_t)(c.layers + 2) * 8 * sizeof(GemvMat) * 2 + 4096;
-  {
-    unsigned char *p = nullptr;
-    r |= salloc(s, s->gemv_tables_cap, &p);
-    s->gemv_tables = p;
+  if (!row_arch) {
+    if (model_ensure_rope(m, max_ctx, s->err)) return fail(1);
+    size_t n_kv = (size_t)n_kv_layers * max_ctx * nKV;
+    r |= salloc(s, (size_t)c.n_lin() * C * 3, &s->conv);
+    r |= salloc(s, (size_t)c.n_lin() * nV * 128 * 128, &s->S);
+    r |= salloc(s, n_kv * D, &s->Kc);
+    r |= salloc(s, n_kv * D, &s->Vc);
+    r |= salloc(s, n_kv, &s->Ks);
+    r |= salloc(s, n_kv, &s->Vs);
+    r |= salloc(s, (size_t)H, &s->X);
+    r |= salloc(s, (size_t)H, &s->Tmp);
+    r |= salloc(s, (size_t)H, &s->Hn);
+    r |= salloc(s, (size_t)H, &s->Mix);
+    int maxK = std::max(std::max(2 * H, VD), nQ * D);
+    r |= salloc(s, (size_t)maxK, &s->Q8);
+    r |= salloc(s, (size_t)maxK / 128, &s->SQ);
+    r |= salloc(s, (size_t)C, &s->Mx);
+    r |= salloc(s, (size_t)VD, &s->Z);
+    r |= salloc(s, (size_t)std::max(nV, 1), &s->Bt);
+    r |= salloc(s, (size_t)std::max(nV, 1), &s->Gt);
+    r |= salloc(s, (size_t)VD, &s->O);
+    r |= salloc(s, (size_t)nQ * 2 * D, &s->Q16);
+    r |= salloc(s, (size_t)nKV * D, &s->K16);
+    r |= salloc(s, (size_t)nKV * D, &s->V16);
+    r |= salloc(s, (size_t)nQ * D, &s->Qn);
+    r |= salloc(s, (size_t)nQ * s->max_chunks, &s->Pm);
+    r |= salloc(s, (size_t)nQ * s->max_chunks, &s->Pse);
+    r |= salloc(s, (size_t)nQ * s->max_chunks * D, &s->Pacc);
+    r |= salloc(s, (size_t)c.experts + 1, &s->RLogits);
+    r |= salloc(s, 1, &s->Counter);
+    r |= salloc(s, (size_t)c.top_k + 1, &s->SelIdx);
+    r |= salloc(s, (size_t)c.top_k + 1, &s->SelRows);
+    r |= salloc(s, (size_t)c.top_k + 1, &s->SelW);
+    r |= salloc(s, 1, &s->NearGap);
+    r |= salloc(s, (size_t)(c.top_k + 1) * c.expert_inter, &s->Act);
+    if (c.mtp_layers) {
+      r |= salloc(s, (size_t)H, &s->Xm);
+      r |= salloc(s, (size_t)H, &s->Hm);
+      r |= salloc(s, (size_t)2 * H, &s->Cat);
+      r |= salloc(s, (size_t)c.vocab, &s->LogitsM);
+      r |= salloc(s, 4, &s->ctrl_m);
+      r |= salloc(s, 1, &s->out_tok_m);
+    }
+    if (flags & SESSION_DIAG) {
+      r |= salloc(s, (size_t)c.layers * H, &s->layer_out);
+      r |= salloc(s, (size_t)c.layers * (c.top_k + 1), &s->routed);
+      r |= salloc(s, (size_t)c.layers, &s->near_gap);
+    }
+    s->gemv_tables_cap = (size_t)(c.layers + 2) * 8 * sizeof(GemvMat) * 2 + 4096;
+    {
+      unsigned char *p = nullptr;
+      r |= salloc(s, s->gemv_tables_cap, &p);
+      s->gemv_tables = p;
+    }
   }
   if (r) return fail(1);
   void *hp = nullptr;
@@ -578,7 +562,7 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
   s->host_tok = (int32_t *)hp;
 
   // ---- record ----
-  Recorder rec{s, nullptr};
+  Recorder rec(s);
   auto new_list = [&](ainfer_list_t *l) {
     if (ainfer_list_create(s->dev, l) != AINFER_OK) { s->err = "list create failed"; rec.status = 1; }
     rec.list = *l;
@@ -606,13 +590,14 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
       rec.launch("ControlAdvance", 1, s->ctrl, (const int32_t *)s->ids, (int32_t)max_ctx);
       if (!rec.status) rec.status = close_list(s, s->advance_list);
     }
+    s->launches_per_token = rec.launches;
   } else {
     new_list(&s->gen_list);
-    s->launches_per_token = 0;
+    rec.launches = 0;
     record_embed(rec);
     for (int L = 0; L < c.layers && !rec.status; ++L) record_layer(rec, L);
     record_tail(rec, true);
-    uint64_t per_token = s->launches_per_token;
+    s->launches_per_token = rec.launches;
     if (!rec.status) rec.status = close_list(s, s->gen_list);
     if (!rec.status) {
       new_list(&s->body_list);
@@ -621,14 +606,11 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
       rec.launch("ControlAdvance", 1, s->ctrl, (const int32_t *)s->ids, (int32_t)max_ctx);
       if (!rec.status) rec.status = close_list(s, s->body_list);
     }
-    s->launches_per_token = per_token;
   }
   if (!rec.status && c.mtp_layers) {
-    const uint64_t per_token = s->launches_per_token;
     new_list(&s->mtp_list);
     record_mtp(rec);
     if (!rec.status) rec.status = close_list(s, s->mtp_list);
-    s->launches_per_token = per_token;
   }
   if (rec.status) return fail(rec.status);
   if (!s->gemv_tables_host.empty() &&
@@ -645,6 +627,7 @@ void session_destroy(Session *s) {
   if (s && s->verifier) { prefill_destroy(s->verifier); s->verifier = nullptr; }
   if (!s) return;
   ainfer_sync(s->dev, UINT64_MAX);
+  delete s->rows;
   for (auto l : s->layer_lists) ainfer_list_destroy(l);
   for (ainfer_list_t l : {s->gen_list, s->body_list, s->embed_list, s->tail_list, s->advance_list, s->mtp_list})
     if (l) ainfer_list_destroy(l);
@@ -683,7 +666,7 @@ static int run_token(Session *s, bool with_tail) {
     // the reference's execution model: execute + fence per list (decode_l0.cpp:714-721)
     int r = exec_fenced(s, s->embed_list, "embed");
     for (size_t L = 0; L < s->layer_lists.size() && !r; ++L)
-      r = exec_fenced(s, s->layer_lists[L], s->m->cfg.layer_types[L] == 'A' ? "attn_layer" : "linear_layer");
+      r = exec_fenced(s, s->layer_lists[L], s->rows || s->m->cfg.layer_types[L] == 'A' ? "attn_layer" : "linear_layer");
     if (!r) r = exec_fenced(s, with_tail ? s->tail_list : s->advance_list, with_tail ? "tail" : "control");
     return r;
   }

@@ -22,10 +22,12 @@ enum SessionFlags {
   SESSION_PER_LAYER_LISTS = 2,  // one list per layer + embed + tail, executed and fenced one by one
   SESSION_MULTI_KERNEL = 4,     // one list per token of ~450 stand-alone launches (the default; flag kept for callers)
   SESSION_STAGE_CLOCK = 8,      // persistent step (implies it): keep a device timestamp after every grid barrier
+  SESSION_F32 = 32,             // activations and cache in 32-bit (architectures with a row engine)
   SESSION_PERSISTENT = 16       // one persistent cooperative launch per token (DecodeStep)
 };
 
 struct Prefill;
+struct RowEngine;
 
 struct Session {
   DeviceModel *m = nullptr;
@@ -34,6 +36,9 @@ struct Session {
   int flags = 0;
   int sm_count = 0;
   std::string err;
+
+  RowEngine *rows = nullptr;    // architectures with a row engine: state and row buffers (then most of the fields
+                                // below up to the diagnostics are unused)
 
   // persistent state (decode_l0.cpp:286-289): conv history, DeltaNet state, KV cache
   float *conv = nullptr;        // [n_lin][conv_dim][3]
@@ -109,6 +114,8 @@ int prefill_create(Session *s, int rows_cap, bool verify, Prefill **out, int ep_
                    const void *id128 = nullptr);
 void prefill_destroy(Prefill *p);
 int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predictions);
+// prefill_run that also returns the logits [n_want][V] of the listed rows (0 <= row < n, ascending).
+int prefill_logits(Prefill *p, const int *tokens, int n, int start_pos, const int *want, int n_want, float *out);
 int prefill_rollback(Prefill *p, int keep);
 int prefill_row_hidden(Prefill *p, int row, float *dst);
 int prefill_rows_cap(const Prefill *p);

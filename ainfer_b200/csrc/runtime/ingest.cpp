@@ -22,6 +22,7 @@
 #include "binfer.h"
 #include "model.h"
 #include "rt_util.h"
+#include "safetensors.h"
 
 namespace ainfer {
 
@@ -82,23 +83,6 @@ struct JsonCursor {
   }
 };
 
-struct SrcTensor {
-  std::string name, dtype;
-  std::vector<uint64_t> shape;
-  const uint8_t *data = nullptr;
-  uint64_t bytes = 0;
-};
-
-struct Shard {
-  int fd = -1;
-  const uint8_t *map = nullptr;
-  size_t size = 0;
-  ~Shard() {
-    if (map) munmap((void *)map, size);
-    if (fd >= 0) close(fd);
-  }
-};
-
 bool open_shard(const std::string &path, Shard &s, std::vector<SrcTensor> &out, std::string &err) {
   s.fd = open(path.c_str(), O_RDONLY);
   struct stat st;
@@ -148,8 +132,6 @@ bool open_shard(const std::string &path, Shard &s, std::vector<SrcTensor> &out, 
   if (!c.lit('}')) { err = path + ": bad header end"; return false; }
   return true;
 }
-
-int elem_bytes(const std::string &dt) { return dt == "BF16" || dt == "F16" ? 2 : (dt == "F32" ? 4 : 0); }
 
 float load_elem(const SrcTensor &t, int eb, uint64_t i) {
   if (eb == 4) { float v; std::memcpy(&v, t.data + i * 4, 4); return v; }
@@ -204,12 +186,26 @@ void quantize_group128(const float *v, uint8_t *packed, uint16_t *scale) {
 
 }  // namespace
 
-int binfer_from_safetensors(const char *src, const char *arch_json, const char *out_path, std::string &err) {
-  if (!src || !arch_json || !out_path) { err = "usage: source, architecture JSON and output path are required"; return 2; }
-  // ---- the shards ----
+Shard::~Shard() {
+  if (map) munmap((void *)map, size);
+  if (fd >= 0) close(fd);
+}
+
+int st_elem_bytes(const std::string &dt) { return dt == "BF16" || dt == "F16" ? 2 : (dt == "F32" ? 4 : 0); }
+
+void st_to_bf16(const SrcTensor &t, uint16_t *out) {
+  const int eb = st_elem_bytes(t.dtype);
+  if (t.dtype == "BF16") {
+    std::memcpy(out, t.data, t.bytes);
+    return;
+  }
+  parallel_for(t.bytes / (uint64_t)eb, [&](uint64_t i) { out[i] = f32_to_bf16(load_elem(t, eb, i)); });
+}
+
+bool SafeTensors::open(const char *src, std::string &err) {
   std::vector<std::string> files;
   struct stat st;
-  if (stat(src, &st) != 0) { err = std::string("cannot open ") + src; return 2; }
+  if (stat(src, &st) != 0) { err = std::string("cannot open ") + src; return false; }
   if (S_ISDIR(st.st_mode)) {
     const std::string dir = src, idx = dir + "/model.safetensors.index.json";
     FILE *f = std::fopen(idx.c_str(), "rb");
@@ -221,13 +217,13 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
       std::fclose(f);
       // "weight_map": {"tensor": "shard file", ...}
       size_t at = js.find("\"weight_map\"");
-      if (at == std::string::npos) { err = idx + ": no weight_map"; return 2; }
+      if (at == std::string::npos) { err = idx + ": no weight_map"; return false; }
       JsonCursor c{js.data() + at + 12, js.data() + js.size(), ""};
-      if (!c.lit(':') || !c.lit('{')) { err = idx + ": bad weight_map"; return 2; }
+      if (!c.lit(':') || !c.lit('{')) { err = idx + ": bad weight_map"; return false; }
       if (!c.lit('}')) {
         do {
           std::string k, v;
-          if (!c.str(k) || !c.lit(':') || !c.str(v)) { err = idx + ": bad weight_map"; return 2; }
+          if (!c.str(k) || !c.lit(':') || !c.str(v)) { err = idx + ": bad weight_map"; return false; }
           if (std::find(files.begin(), files.end(), dir + "/" + v) == files.end()) files.push_back(dir + "/" + v);
         } while (c.lit(','));
       }
@@ -237,24 +233,30 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
   } else {
     files.push_back(src);
   }
-  std::vector<Shard> shards(files.size());
-  std::vector<SrcTensor> srcs;
+  shards = std::vector<Shard>(files.size());
   for (size_t i = 0; i < files.size(); ++i)
-    if (!open_shard(files[i], shards[i], srcs, err)) return 2;
+    if (!open_shard(files[i], shards[i], tensors, err)) return false;
+  return true;
+}
+
+int binfer_from_safetensors(const char *src, const char *arch_json, const char *out_path, std::string &err) {
+  if (!src || !arch_json || !out_path) { err = "usage: source, architecture JSON and output path are required"; return 2; }
+  SafeTensors files;
+  if (!files.open(src, err)) return 2;
   // ---- the plan: names sorted, vision tower left out, policy per tensor ----
   ModelConfig cfg;
   if (!ModelConfig::from_json(arch_json, cfg, err) || !cfg.check(err)) return 2;
   std::vector<std::pair<std::string, const SrcTensor *>> plan;
-  for (const SrcTensor &t : srcs) {
+  for (const SrcTensor &t : files.tensors) {
     if (t.name.find("visual") != std::string::npos) continue;
-    plan.emplace_back(canonical_name(t.name), &t);
+    plan.emplace_back(cfg.int4_weights() ? canonical_name(t.name) : t.name, &t);
   }
   std::sort(plan.begin(), plan.end(), [](const auto &a, const auto &b) { return a.first < b.first; });
   Container c;
   std::vector<const SrcTensor *> by_entry;
   for (auto &pr : plan) {
     const SrcTensor &t = *pr.second;
-    const int eb = elem_bytes(t.dtype);
+    const int eb = st_elem_bytes(t.dtype);
     if (!eb) { err = "unsupported source dtype " + t.dtype + " for " + t.name; return 2; }
     if (pr.first.size() > 63) { err = "tensor name longer than 63 bytes: " + pr.first; return 2; }
     if (t.shape.empty() || t.shape.size() > 8) { err = "unsupported rank for " + t.name; return 2; }
@@ -265,7 +267,7 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
     uint64_t n = 1;
     for (int i = 0; i < e.ndim; ++i) { e.shape[i] = t.shape[i]; n *= t.shape[i]; }
     if (n * (uint64_t)eb != t.bytes) { err = "payload size does not match shape: " + t.name; return 2; }
-    const bool keep = e.ndim != 2 || ends_with(e.name, "embed_tokens.weight") || ends_with(e.name, "mlp.gate.weight") ||
+    const bool keep = !cfg.int4_weights() || e.ndim != 2 || ends_with(e.name, "embed_tokens.weight") || ends_with(e.name, "mlp.gate.weight") ||
                       ends_with(e.name, "shared_expert_gate.weight");
     e.logical = DT_BF16;
     if (keep) {
@@ -287,7 +289,7 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
                     "\"0000000000000000000000000000000000000000\",\"source_total_bytes\":0}";
   c.arch_json = cfg.to_json();
   c.tokenizer_json = "{\"format\":\"none\",\"vocab_size\":" + std::to_string(cfg.vocab) + "}";
-  c.policy_json =
+  c.policy_json = !cfg.int4_weights() ? std::string("{\"default\":\"BF16\"}") :
       "{\"default\":\"INT4 symmetric g128 BF16 scales\",\"exceptions\":[\"embed_tokens BF16\","
       "\"1-D norms source precision\",\"A_log/dt_bias/conv1d source precision\","
       "\"mlp.gate (router) BF16\",\"mlp.shared_expert_gate BF16\"],\"group_size\":128}";
@@ -298,7 +300,7 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
   auto fill = [](void *user, const TensorEntry &e, uint8_t *payload, uint8_t *scales) {
     Ctx *x = (Ctx *)user;
     const SrcTensor &t = *(*x->src)[x->c->index[e.name]];
-    const int eb = elem_bytes(t.dtype);
+    const int eb = st_elem_bytes(t.dtype);
     const uint64_t n = e.numel();
     if (e.storage == DT_INT4_SYM_G128) {
       parallel_for(n / 128, [&](uint64_t g) {
@@ -306,11 +308,8 @@ int binfer_from_safetensors(const char *src, const char *arch_json, const char *
         for (int j = 0; j < 128; ++j) v[j] = load_elem(t, eb, g * 128 + j);
         quantize_group128(v, payload + g * 64, (uint16_t *)scales + g);
       });
-    } else if (t.dtype == "BF16") {
-      std::memcpy(payload, t.data, n * 2);
     } else {
-      uint16_t *out = (uint16_t *)payload;
-      parallel_for(n, [&](uint64_t i) { out[i] = f32_to_bf16(load_elem(t, eb, i)); });
+      st_to_bf16(t, (uint16_t *)payload);
     }
   };
   return container_write(out_path, c, fill, &ctx, err);

@@ -1,5 +1,7 @@
 #include "model.h"
 
+#include <sys/stat.h>
+
 #include <cmath>
 #include <cstdlib>
 #include <cstring>
@@ -8,14 +10,34 @@
 
 #include "../common/detmath.h"
 #include "../common/tables.h"
+#include "arch.h"
+#include "json.h"
 #include "rt_util.h"
+#include "safetensors.h"
 
 namespace ainfer {
 
 std::string layer_prefix(int L) { return "model.language_model.layers." + std::to_string(L) + "."; }
 
+// ----------------------------------------------------------- registry ---
+const ModelArch *model_arch(const std::string &name) {
+  const ModelArch *row[] = {sinepel_model_arch()};
+  for (const ModelArch *a : row)
+    if (name == a->name) return a;
+  return nullptr;
+}
+// A configuration's architecture: the registered one, else the INT4 hybrid (whose "arch" is free text).
+static const ModelArch &arch_of(const ModelConfig &c) {
+  const ModelArch *a = model_arch(c.arch);
+  return a ? *a : *int4_hybrid_model_arch();
+}
+std::string ModelConfig::to_json() const { return arch_of(*this).to_json(*this); }
+bool ModelConfig::check(std::string &err) const { return arch_of(*this).check(*this, err); }
+void build_plan(const ModelConfig &cfg, Container &c, std::vector<SynthSpec> &specs) { arch_of(cfg).plan(cfg, c, specs); }
+int check_directory_shapes(const Container &dir, const ModelConfig &cfg, std::string &err) { return arch_of(cfg).check_directory(dir, cfg, err); }
+
 // ------------------------------------------------------------- config ---
-std::string ModelConfig::to_json() const {
+static std::string int4_to_json(const ModelConfig &c) {
   char b[1024];
   std::snprintf(
       b, sizeof b,
@@ -25,9 +47,9 @@ std::string ModelConfig::to_json() const {
       "\"experts\":%d,\"top_k\":%d,\"shared_experts\":%d,\"expert_intermediate\":%d,"
       "\"mtp_layers\":%d,\"rms_eps\":%.9g,\"kv_cache\":\"int8_per_token_head_fp16_scale\","
       "\"attn_output_gate\":true,\"mlp_act\":\"silu\",\"vision\":\"absent\"}",
-      arch.c_str(), layers, layer_types.c_str(), hidden, vocab, q_heads, kv_heads, head_dim,
-      rotary_dim, rope_theta, lin_k_heads, lin_v_heads, lin_head_dim, conv_kernel, experts, top_k,
-      shared_experts, expert_inter, mtp_layers, rms_eps);
+      c.arch.c_str(), c.layers, c.layer_types.c_str(), c.hidden, c.vocab, c.q_heads, c.kv_heads, c.head_dim,
+      c.rotary_dim, c.rope_theta, c.lin_k_heads, c.lin_v_heads, c.lin_head_dim, c.conv_kernel, c.experts, c.top_k,
+      c.shared_experts, c.expert_inter, c.mtp_layers, c.rms_eps);
   return b;
 }
 
@@ -59,7 +81,15 @@ static double jnum(const std::string &js, const char *k, double d) {
 
 bool ModelConfig::from_json(const std::string &js, ModelConfig &c, std::string &err) {
   c = ModelConfig();
+  Json tree;
+  std::string why;
+  if (Json::parse(js, tree, why) && tree.has("architecture")) {   // a registered architecture's own form
+    const ModelArch *a = model_arch(tree.at("architecture").str());
+    if (!a) { err = "unknown architecture \"" + tree.at("architecture").str() + "\""; return false; }
+    return a->parse(tree, c, err) && a->check(c, err);
+  }
   json_raw(js, "arch", c.arch);
+  if (model_arch(c.arch)) { err = "unsupported architecture: " + c.arch + " has another configuration form"; return false; }
   c.hidden = (int)jint(js, "hidden", 0);
   c.layers = (int)jint(js, "text_layers", 0);
   c.vocab = (int)jint(js, "vocab", 0);
@@ -86,37 +116,51 @@ bool ModelConfig::from_json(const std::string &js, ModelConfig &c, std::string &
 
 static bool pow2_between(int v, int lo, int hi) { return v >= lo && v <= hi && (v & (v - 1)) == 0; }
 
-bool ModelConfig::check(std::string &err) const {
+static bool int4_check(const ModelConfig &c, std::string &err) {
   auto bad = [&](const std::string &m) { err = "unsupported architecture: " + m; return false; };
-  if (layers <= 0 || (int)layer_types.size() != layers) return bad("layer_types/text_layers mismatch");
-  for (char c : layer_types)
-    if (c != 'L' && c != 'A') return bad("layer_types may hold only L and A");
-  if (!pow2_between(hidden, 256, 4096)) return bad("hidden must be a power of two in [256, 4096]");
-  if (vocab <= 0) return bad("vocab");
-  if (head_dim != 256) return bad("head_dim must be 256");
-  if (rotary_dim != 64) return bad("rotary_dim must be 64");
-  if (n_attn() || mtp_layers) {
-    if (kv_heads <= 0 || q_heads % kv_heads) return bad("q_heads must be a multiple of kv_heads");
-    int g = q_heads / kv_heads;
+  if (c.layers <= 0 || (int)c.layer_types.size() != c.layers) return bad("layer_types/text_layers mismatch");
+  for (char t : c.layer_types)
+    if (t != 'L' && t != 'A') return bad("layer_types may hold only L and A");
+  if (!pow2_between(c.hidden, 256, 4096)) return bad("hidden must be a power of two in [256, 4096]");
+  if (c.vocab <= 0) return bad("vocab");
+  if (c.head_dim != 256) return bad("head_dim must be 256");
+  if (c.rotary_dim != 64) return bad("rotary_dim must be 64");
+  if (c.n_attn() || c.mtp_layers) {
+    if (c.kv_heads <= 0 || c.q_heads % c.kv_heads) return bad("q_heads must be a multiple of kv_heads");
+    int g = c.q_heads / c.kv_heads;
     if (g != 1 && g != 2 && g != 4 && g != 6 && g != 8) return bad("q_heads/kv_heads must be 1, 2, 4, 6 or 8");
-    if (!pow2_between(q_heads * head_dim, 128, 4096)) return bad("q_heads*head_dim must be a power of two <= 4096");
+    if (!pow2_between(c.q_heads * c.head_dim, 128, 4096)) return bad("q_heads*head_dim must be a power of two <= 4096");
   }
-  if (n_lin()) {
-    if (lin_head_dim != 128) return bad("lin_head_dim must be 128");
-    if (conv_kernel != 4) return bad("conv_kernel must be 4");
-    if (lin_k_heads <= 0 || lin_v_heads % lin_k_heads) return bad("lin_v_heads must be a multiple of lin_k_heads");
-    if (!pow2_between(value_dim(), 128, 4096)) return bad("lin_v_heads*128 must be a power of two <= 4096");
+  if (c.n_lin()) {
+    if (c.lin_head_dim != 128) return bad("lin_head_dim must be 128");
+    if (c.conv_kernel != 4) return bad("conv_kernel must be 4");
+    if (c.lin_k_heads <= 0 || c.lin_v_heads % c.lin_k_heads) return bad("lin_v_heads must be a multiple of lin_k_heads");
+    if (!pow2_between(c.value_dim(), 128, 4096)) return bad("lin_v_heads*128 must be a power of two <= 4096");
   }
-  if (experts < 32 || experts > 1024 || experts % 32) return bad("experts must be a multiple of 32 in [32, 1024]");
-  if (top_k <= 0 || top_k > 11 || top_k > experts) return bad("top_k must be in [1, 11]");
-  if (shared_experts != 0 && shared_experts != 1) return bad("shared_experts must be 0 or 1");
-  if (!pow2_between(expert_inter, 128, 1024)) return bad("expert_intermediate must be a power of two in [128, 1024]");
-  if (mtp_layers != 0 && mtp_layers != 1) return bad("mtp_layers must be 0 or 1");
+  if (c.experts < 32 || c.experts > 1024 || c.experts % 32) return bad("experts must be a multiple of 32 in [32, 1024]");
+  if (c.top_k <= 0 || c.top_k > 11 || c.top_k > c.experts) return bad("top_k must be in [1, 11]");
+  if (c.shared_experts != 0 && c.shared_experts != 1) return bad("shared_experts must be 0 or 1");
+  if (!pow2_between(c.expert_inter, 128, 1024)) return bad("expert_intermediate must be a power of two in [128, 1024]");
+  if (c.mtp_layers != 0 && c.mtp_layers != 1) return bad("mtp_layers must be 0 or 1");
+  return true;
+}
+
+static bool read_text(const std::string &path, std::string &out) {
+  FILE *f = fopen(path.c_str(), "rb");
+  if (!f) return false;
+  char buf[65536];
+  size_t n;
+  while ((n = fread(buf, 1, sizeof buf, f)) > 0) out.append(buf, n);
+  fclose(f);
   return true;
 }
 
 bool preset_config(const std::string &name, ModelConfig &c) {
   c = ModelConfig();
+  if (name.rfind("config:", 0) == 0) {
+    std::string js, err;
+    return read_text(name.substr(7), js) && ModelConfig::from_json(js, c, err);
+  }
   if (name == "tiny") {
     c.hidden = 256; c.layers = 2; c.layer_types = "LA"; c.vocab = 512;
     c.q_heads = 2; c.kv_heads = 1; c.lin_k_heads = 2; c.lin_v_heads = 4;
@@ -216,7 +260,7 @@ static void plan_layer(PlanBuilder &pb, const ModelConfig &cfg, const std::strin
   plan_moe(pb, cfg, p);
 }
 
-void build_plan(const ModelConfig &cfg, Container &c, std::vector<SynthSpec> &specs) {
+static void int4_plan(const ModelConfig &cfg, Container &c, std::vector<SynthSpec> &specs) {
   c = Container();
   specs.clear();
   PlanBuilder pb{c, specs};
@@ -361,7 +405,7 @@ static int mirror_small(DeviceModel *m, const std::string &name, float *dst, uin
   return launch_simple(dev, "WidenBf16", {{&dst, 8}, {&in, 8}, {&count, 8}}, groups, err);
 }
 
-int check_directory_shapes(const Container &dir, const ModelConfig &c, std::string &err) {
+static int int4_check_directory(const Container &dir, const ModelConfig &c, std::string &err) {
   const uint64_t H = c.hidden, D = c.head_dim, I = c.expert_inter, V = c.vocab;
   auto need = [&](const std::string &name, uint64_t rows, uint64_t cols, int storage) -> int {
     const TensorEntry *e = dir.find(name);
@@ -474,6 +518,10 @@ static int build_mirrors(DeviceModel *m, std::string &err) {
   return 0;
 }
 
+static const ModelArch kInt4Hybrid = {"int4 hybrid", true,       nullptr,   int4_to_json,
+                                      int4_check,    int4_plan,  int4_check_directory, build_mirrors};
+const ModelArch *int4_hybrid_model_arch() { return &kInt4Hybrid; }
+
 int model_ensure_rope(DeviceModel *m, int max_ctx, std::string &err) {
   if (max_ctx <= m->rope_ctx) return 0;
   ainfer_device_t dev = m->dev;
@@ -570,6 +618,40 @@ static int upload_file(DeviceModel *m, const char *path, std::string &err) {
   return r;
 }
 
+// Uploads the tensors of a SafeTensors source into the arena, each at its directory entry's place.
+static int upload_safetensors(DeviceModel *m, const SafeTensors &src, std::string &err) {
+  ainfer_device_t dev = m->dev;
+  RT_CHECK(ainfer_mem_fill(dev, m->pay_arena, 0, m->pay_bytes));
+  std::vector<uint16_t> tmp;
+  for (const SrcTensor &t : src.tensors) {
+    const TensorEntry *e = m->dir.find(t.name);
+    if (!e) continue;   // not one this architecture reads
+    tmp.resize(e->numel());
+    st_to_bf16(t, tmp.data());
+    RT_CHECK(ainfer_memcpy_h2d(dev, (char *)m->pay_arena + (e->d_off - m->dir.pay_lo), tmp.data(), e->d_bytes));
+  }
+  return 0;
+}
+
+// The directory of a folder's tensors in the architecture's storage order; shapes as the file has them.
+static int directory_from_safetensors(const ModelConfig &cfg, const SafeTensors &src, Container &dir, std::string &err) {
+  std::vector<SynthSpec> specs;
+  build_plan(cfg, dir, specs);
+  std::map<std::string, const SrcTensor *> by_name;
+  for (const SrcTensor &t : src.tensors) by_name[t.name] = &t;
+  for (TensorEntry &e : dir.entries) {
+    auto it = by_name.find(e.name);
+    if (it == by_name.end()) { err = "missing " + e.name; return 1; }
+    const SrcTensor &t = *it->second;
+    const int eb = st_elem_bytes(t.dtype);
+    if (!eb) { err = "unsupported source dtype " + t.dtype + " for " + e.name; return 2; }
+    bool same = t.shape.size() == (size_t)e.ndim && t.bytes == e.numel() * (uint64_t)eb;
+    for (int i = 0; same && i < e.ndim; ++i) same = t.shape[(size_t)i] == e.shape[i];
+    if (!same) { err = "unexpected shape of " + e.name; return 2; }
+  }
+  return 0;
+}
+
 int model_open(ainfer_device_t dev, const char *spec, int validate_level, DeviceModel **out,
                std::string &err) {
   *out = nullptr;
@@ -577,19 +659,29 @@ int model_open(ainfer_device_t dev, const char *spec, int validate_level, Device
   m->dev = dev;
   std::vector<SynthSpec> specs;
   std::string s = spec ? spec : "";
+  SafeTensors files;
+  struct stat fs;
   int r = 0;
   if (s.rfind("synth:", 0) == 0) {
     std::string rest = s.substr(6), preset = rest;
-    size_t c = rest.find(':');
+    size_t c = rest.rfind(":seed=");
     if (c != std::string::npos) {
       preset = rest.substr(0, c);
-      size_t sp = rest.find("seed=");
+      size_t sp = rest.rfind("seed=");
       if (sp != std::string::npos) m->seed = std::strtoull(rest.c_str() + sp + 5, nullptr, 10);
     }
     if (!preset_config(preset, m->cfg)) { err = "unknown synthetic preset: " + preset; delete m; return 2; }
     if (!m->cfg.check(err)) { delete m; return 2; }
     build_plan(m->cfg, m->dir, specs);
     m->synthetic = true;
+  } else if (stat(s.c_str(), &fs) == 0 && S_ISDIR(fs.st_mode)) {
+    std::string js;
+    if (!read_text(s + "/config.json", js)) { err = "cannot open " + s + "/config.json"; delete m; return 2; }
+    if (!ModelConfig::from_json(js, m->cfg, err)) { delete m; return 2; }
+    if (m->cfg.int4_weights()) { err = "usage: convert this architecture's checkpoint to a .binfer file first"; delete m; return 2; }
+    if (!files.open(s.c_str(), err)) { delete m; return 2; }
+    r = directory_from_safetensors(m->cfg, files, m->dir, err);
+    if (r) { delete m; return r; }
   } else {
     r = container_open(s.c_str(), validate_level, m->dir, err);
     if (r) { delete m; return r; }
@@ -613,10 +705,12 @@ int model_open(ainfer_device_t dev, const char *spec, int validate_level, Device
       err = ainfer_last_error(dev); model_close(m); return 1;
     }
     r = fill_synthetic(m, specs, err);
+  } else if (!files.tensors.empty()) {
+    r = upload_safetensors(m, files, err);
   } else {
     r = upload_file(m, s.c_str(), err);
   }
-  if (!r) r = build_mirrors(m, err);
+  if (!r) r = arch_of(m->cfg).prepare(m, err);
   if (r) { model_close(m); return r; }
   *out = m;
   return 0;

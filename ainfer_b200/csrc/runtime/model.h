@@ -7,6 +7,7 @@
 #pragma once
 #include <cstdint>
 #include <map>
+#include <memory>
 #include <string>
 #include <vector>
 
@@ -15,8 +16,17 @@
 
 namespace ainfer {
 
+// One layer of an architecture whose layers carry their own sizes: attention over keys that are also
+// the values, with a short convolution, inside chunks of positions, and a dense feed-forward.
+struct RowLayerConfig {
+  int heads = 0, kv_heads = 0, dim = 0, taps = 1;
+  int chunk = 0;       // positions per chunk (0: one chunk)
+  double scale = 1.0;  // of the scores
+  int ff = 0;          // feed-forward size (0: none)
+};
+
 struct ModelConfig {
-  std::string arch = "qwen3_5_moe";
+  std::string arch = "qwen3_5_moe";   // name in the architecture registry (arch.h)
   int hidden = 0, layers = 0, vocab = 0;
   std::string layer_types;  // one char per layer: 'L' Gated DeltaNet, 'A' gated GQA attention
   int q_heads = 0, kv_heads = 0, head_dim = 256, rotary_dim = 64;
@@ -25,6 +35,11 @@ struct ModelConfig {
   int experts = 0, top_k = 0, shared_experts = 1, expert_inter = 0;
   int mtp_layers = 0;
   double rms_eps = 1e-6;
+  // architectures of residual streams (hidden, layers, vocab and rms_eps are shared)
+  std::vector<RowLayerConfig> row_layers;
+  int streams = 1, max_positions = 0;
+  double embed_scale = 1.0, logit_softcap = 0.0;
+  bool int4_weights() const { return row_layers.empty(); }
   int conv_dim() const { return (2 * lin_k_heads + lin_v_heads) * lin_head_dim; }
   int value_dim() const { return lin_v_heads * lin_head_dim; }
   int n_attn() const { int n = 0; for (char c : layer_types) n += c == 'A'; return n; }
@@ -35,7 +50,7 @@ struct ModelConfig {
   bool check(std::string &err) const;
 };
 
-// Named synthetic shapes: "tiny" (CPU-test sized), "mini" (the CPU-runnable
+// Named synthetic shapes, or a config.json given as "config:<path>" with an "architecture": "tiny" (CPU-test sized), "mini" (the CPU-runnable
 // reference mini-model), "full" (80B-A3B-shaped). Returns false if unknown.
 bool preset_config(const std::string &name, ModelConfig &out);
 
@@ -66,6 +81,8 @@ struct DeviceTensor {
   void *scales = nullptr;  // device address of the scales (INT4) or null
 };
 
+struct RowWeights;   // prepared weights of architectures with a row engine
+
 // Device-resident model.
 struct DeviceModel {
   ainfer_device_t dev = nullptr;
@@ -88,12 +105,14 @@ struct DeviceModel {
   int rope_ctx = 0;
   void *expert_tables = nullptr;                        // [layers(+mtp)][experts+1] ExpertW
   std::vector<int> slot;                                // per layer: index within its type
+  std::shared_ptr<RowWeights> rows;                     // null for the INT4 hybrid
 
   DeviceTensor tensor(const std::string &name) const;
   bool has(const std::string &name) const { return dir.find(name) != nullptr; }
 };
 
-// Opens "synth:<preset>[:seed=N]" (filled on the device) or a .binfer path.
+// Opens "synth:<preset>[:seed=N]" (filled on the device), a folder with config.json (naming its
+// "architecture") and SafeTensors weights, or a .binfer path.
 // Returns 0, or the reference's exit codes: 1 device/API error or missing
 // tensor, 2 bad container / usage.
 int model_open(ainfer_device_t dev, const char *spec, int validate_level, DeviceModel **out,

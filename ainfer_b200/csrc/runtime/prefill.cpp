@@ -22,6 +22,7 @@
 // ones are overwritten before any later position reads them).
 #include <cstring>
 
+#include "arch.h"
 #include "ep.h"
 #include "executor.h"
 #include "row_slabs.h"
@@ -49,6 +50,9 @@ struct Prefill {
   float *Qn = nullptr, *Pm = nullptr, *Pse = nullptr, *Pacc = nullptr;   // per-row attention scratch
   std::map<std::string, ainfer_kernel_t> kernels;
   RowSlabCache slabs;   // problem lists of the GEMMs with few output rows (row_slabs.h)
+  // architectures with a row engine: the rows' sequence (0), its first row (0), and the rows whose logits are wanted
+  int32_t *Seq = nullptr, *First = nullptr, *Want = nullptr;
+  int logits_cap = 0;                            // rows Logits holds
 };
 
 namespace {
@@ -67,11 +71,10 @@ int palloc(Prefill *p, size_t count, T **out) {
   return 0;
 }
 
-struct Launcher {   // immediate launches, or appended to recorded lists; arguments by index in member order
+struct Launcher : KernelCalls {   // immediate launches, or appended to recorded lists
   Prefill *p;
-  int status = 0;
   bool recording = false;
-  ainfer_list_t list = nullptr;
+  explicit Launcher(Prefill *pf) : KernelCalls(pf->s->dev, &pf->kernels, &pf->s->err), p(pf) {}
   // recording: closes the current list (if any) into p->vlists and opens the next one
   void cut(bool open_next) {
     if (status) return;
@@ -82,29 +85,6 @@ struct Launcher {   // immediate launches, or appended to recorded lists; argume
       list = nullptr;
     }
     if (open_next && ainfer_list_create(s->dev, &list) != AINFER_OK) { s->err = ainfer_last_error(s->dev); status = 1; }
-  }
-  template <typename T>
-  void set(ainfer_kernel_t k, uint32_t &idx, const T &v) {
-    if (status) return;
-    if (ainfer_kernel_set_arg(k, idx, sizeof(T), &v) != AINFER_OK) { p->s->err = ainfer_last_error(p->s->dev); status = 1; }
-    ++idx;
-  }
-  template <typename... A>
-  void launch(const char *name, uint32_t groups, const A &...args) {
-    if (status) return;
-    Session *s = p->s;
-    auto it = p->kernels.find(name);
-    ainfer_kernel_t k = nullptr;
-    if (it != p->kernels.end()) k = it->second;
-    else {
-      if (ainfer_kernel_get(s->dev, name, &k) != AINFER_OK) { s->err = std::string("entry ") + name + " not found"; status = 1; return; }
-      p->kernels[name] = k;
-    }
-    uint32_t idx = 0;
-    (set(k, idx, args), ...);
-    if (status) return;
-    const int rc = recording ? ainfer_list_append_launch(list, k, groups ? groups : 1) : ainfer_kernel_launch(s->dev, k, groups ? groups : 1);
-    if (rc != AINFER_OK) { s->err = std::string(name) + ": " + ainfer_last_error(s->dev); status = 1; }
   }
   // Y[rows][N] = X[rows][K] . W^T on the tensor cores
   void gemm(const DeviceTensor &t, const int8_t *XQ, const float *SQ, float *Y, int K, int rows) {
@@ -146,6 +126,16 @@ int prefill_create(Session *s, int rows_cap, bool verify, Prefill **out, int ep_
   Prefill *p = new Prefill;
   p->s = s;
   p->rows_cap = rows_cap;
+  if (s->rows) {
+    p->rows_cap = std::min(rows_cap, s->rows->rows_cap);
+    const size_t n = (size_t)p->rows_cap;
+    if (palloc(p, n * 4, &p->Ctrl) || palloc(p, n, &p->Seq) || palloc(p, n, &p->First) || palloc(p, n, &p->Want)) {
+      prefill_destroy(p);
+      return 1;
+    }
+    *out = p;
+    return 0;
+  }
   const int R = p->rows_cap, H = c.hidden, C = c.conv_dim(), VD = c.value_dim(), nV = c.lin_v_heads;
   const int QN = c.q_heads * 2 * c.head_dim, KN = c.kv_heads * c.head_dim, AK = c.q_heads * c.head_dim;
   const int maxK = std::max(H, std::max(VD, AK));
@@ -191,6 +181,47 @@ void prefill_destroy(Prefill *p) {
 // Advances the session over tokens[0..n) at positions start_pos... predictions (optional, needs a
 // verification object and n <= its rows): every row's greedy next token; the state after every
 // row is then also kept for prefill_rollback.
+// The passes of an architecture with a row engine; want: ascending rows of [0, n) whose logits go to out.
+static int row_passes(Prefill *p, const int *tokens, int n, int start_pos, const int *want, int n_want, float *out) {
+  Session *s = p->s;
+  const size_t V = (size_t)s->m->cfg.vocab;
+  auto failed = [&](int rc) {
+    if (rc != AINFER_OK) s->err = ainfer_last_error(s->dev);
+    return rc != AINFER_OK;
+  };
+  std::vector<int32_t> ctrl((size_t)p->rows_cap * 4), rel;
+  int w = 0;
+  for (int t0 = 0; t0 < n; t0 += p->rows_cap) {
+    const int rows = std::min(p->rows_cap, n - t0);
+    for (int i = 0; i < rows; ++i) {
+      ctrl[4 * i] = tokens[t0 + i];
+      ctrl[4 * i + 1] = start_pos + t0 + i;
+      ctrl[4 * i + 2] = start_pos + t0 + i + 1;
+      ctrl[4 * i + 3] = -1;
+    }
+    if (failed(ainfer_memcpy_h2d(s->dev, p->Ctrl, ctrl.data(), (size_t)rows * 16))) return 1;
+    RowSpan span;
+    span.ctrl = p->Ctrl; span.seq = p->Seq; span.first = p->First;
+    span.rows = rows;
+    rel.clear();
+    const int w0 = w;
+    while (w < n_want && want[w] < t0 + rows) rel.push_back(want[w++] - t0);
+    if (!rel.empty()) {
+      if (failed(ainfer_memcpy_h2d(s->dev, p->Want, rel.data(), rel.size() * 4))) return 1;
+      if (p->logits_cap < (int)rel.size()) {   // grows by whole steps: few reallocations over a session
+        p->logits_cap = std::min(p->rows_cap, ((int)rel.size() + 63) / 64 * 64);
+        if (palloc(p, (size_t)p->logits_cap * V, &p->Logits)) return 1;
+      }
+      span.want = p->Want; span.n_want = (int)rel.size(); span.logits = p->Logits;
+    }
+    Launcher l(p);
+    s->rows->emit(l, span);
+    if (l.status) return l.status;
+    if (!rel.empty() && failed(ainfer_memcpy_d2h(s->dev, out + (size_t)w0 * V, p->Logits, rel.size() * V * 4))) return 1;
+  }
+  return failed(ainfer_sync(s->dev, UINT64_MAX)) ? 1 : 0;
+}
+
 int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predictions) {
   Session *s = p->s;
   DeviceModel *m = s->m;
@@ -199,9 +230,12 @@ int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predic
     s->err = "context overflow: pos " + std::to_string(start_pos + n) + " >= MAXCTX " + std::to_string(s->max_ctx);
     return 3;
   }
+  if (s->rows) {
+    if (predictions) { s->err = "usage: this architecture has no verification pass"; return 2; }
+    return row_passes(p, tokens, n, start_pos, nullptr, 0, nullptr);
+  }
   const int H = c.hidden, C = c.conv_dim(), VD = c.value_dim(), nK = c.lin_k_heads, nV = c.lin_v_heads;
-  const int nQ = c.q_heads, nKV = c.kv_heads, D = c.head_dim;
-  const int QN = nQ * 2 * D, KN = nKV * D, AK = nQ * D;
+  const int nQ = c.q_heads, nKV = c.kv_heads, D = c.head_dim, AK = nQ * D;
   const float eps = (float)c.rms_eps;
   DeviceTensor emb = m->tensor("model.language_model.embed_tokens.weight");
   if (!emb.entry) { s->err = "missing model.language_model.embed_tokens.weight"; return 1; }
@@ -279,7 +313,7 @@ int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predic
   std::vector<int32_t> ctrl((size_t)p->rows_cap * 4);
   const bool use_lists = verify && n == p->rows_cap;
   if (use_lists && p->vlists.empty()) {
-    Launcher rec{p};
+    Launcher rec(p);
     rec.recording = true;
     rec.cut(true);
     int e = pass(rec, n);
@@ -307,7 +341,7 @@ int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predic
       }
       if (ainfer_list_execute(p->vlists[c.layers]) != AINFER_OK) { s->err = ainfer_last_error(s->dev); return 1; }
     } else {
-      Launcher l{p};
+      Launcher l(p);
       int e = pass(l, rows);
       if (e) return e;
     }
@@ -316,6 +350,30 @@ int prefill_run(Prefill *p, const int *tokens, int n, int start_pos, int *predic
     if (ainfer_memcpy_d2h(s->dev, predictions, p->OutT, (size_t)n * 4) != AINFER_OK) { s->err = ainfer_last_error(s->dev); return 1; }
   } else if (ainfer_sync(s->dev, UINT64_MAX) != AINFER_OK) { s->err = ainfer_last_error(s->dev); return 1; }
   return 0;
+}
+
+int prefill_logits(Prefill *p, const int *tokens, int n, int start_pos, const int *want, int n_want, float *out) {
+  Session *s = p->s;
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= n || (i && want[i] <= want[i - 1])) { s->err = "usage: wanted rows must be ascending and inside the call"; return 2; }
+  if (s->rows) {
+    if (n < 0 || start_pos < 0 || start_pos + n > s->max_ctx) {
+      s->err = "context overflow: pos " + std::to_string(start_pos + n) + " >= MAXCTX " + std::to_string(s->max_ctx);
+      return 3;
+    }
+    return row_passes(p, tokens, n, start_pos, want, n_want, out);
+  }
+  // INT4 hybrid: runs of tokens up to each wanted one, whose step (token loop) leaves its logits
+  const size_t V = (size_t)s->m->cfg.vocab;
+  int at = 0;
+  for (int i = 0; i < n_want; ++i) {
+    int e = prefill_run(p, tokens + at, want[i] - at, start_pos + at, nullptr);
+    if (!e) e = session_step(s, tokens[want[i]], start_pos + want[i], nullptr);
+    if (e) return e;
+    if (ainfer_memcpy_d2h(s->dev, out + (size_t)i * V, s->Logits, V * 4) != AINFER_OK) { s->err = ainfer_last_error(s->dev); return 1; }
+    at = want[i] + 1;
+  }
+  return prefill_run(p, tokens + at, n - at, start_pos + at, nullptr);
 }
 
 // Copies row `row`'s final residual of the last verifying pass to dst (H floats, device).

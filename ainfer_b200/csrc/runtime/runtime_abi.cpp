@@ -3,6 +3,7 @@
 #include <string>
 
 #include "../../../include/ainfer_runtime.h"
+#include "arch.h"
 #include "batch.h"
 #include "ep.h"
 #include "executor.h"
@@ -32,7 +33,8 @@ int ainfer_binfer_validate(const char *path, int level) {
   int r = container_open(path, level, c, err);
   if (r == 0) {
     ModelConfig cfg;
-    if (!c.arch_json.empty() && c.arch_json.find("\"text_layers\"") != std::string::npos) {
+    if (!c.arch_json.empty() && (c.arch_json.find("\"text_layers\"") != std::string::npos ||
+                                 c.arch_json.find("\"architecture\"") != std::string::npos)) {
       if (!ModelConfig::from_json(c.arch_json, cfg, err)) r = 2;
       else r = check_directory_shapes(c, cfg, err);
     }
@@ -139,6 +141,8 @@ int ainfer_session_buffer(ainfer_session_t h, const char *which, void **dptr, ui
   Session *s = h->s;
   const ModelConfig &c = s->m->cfg;
   std::string w = which;
+  if (s->rows && s->rows->buffer(w, dptr, bytes)) return 0;
+  if (s->rows && w != "logits" && w != "ctrl" && w != "history") return set_err(2, "unknown session buffer: " + w);
   size_t n_kv = (size_t)(c.n_attn() + c.mtp_layers) * s->max_ctx * c.kv_heads;
   if (w == "conv") { *dptr = s->conv; *bytes = (uint64_t)c.n_lin() * c.conv_dim() * 3 * 4; }
   else if (w == "S") { *dptr = s->S; *bytes = (uint64_t)c.n_lin() * c.lin_v_heads * 128 * 128 * 4; }
@@ -158,9 +162,11 @@ int ainfer_session_buffer(ainfer_session_t h, const char *which, void **dptr, ui
   else return set_err(2, "unknown session buffer: " + w);
   return 0;
 }
-int ainfer_session_prefill(ainfer_session_t h, const int *tokens, int n, int start_pos) {
-  if (!h || (!tokens && n > 0)) return set_err(2, "usage: null argument");
-  Session *s = h->s;
+static int ensure_prefill(Session *s) {
+  if (!s->prefill && s->rows) {
+    int r = prefill_create(s, s->pf_rows > 0 ? s->pf_rows : s->rows->rows_cap, false, &s->prefill);
+    if (r) return set_err(r, s->err);
+  }
   if (!s->prefill) {
     // rows per pass: the planner of the expert-parallel block takes 2048 (row, expert) items over all ranks
     const int topk = s->m->cfg.top_k > 0 ? s->m->cfg.top_k : 1;
@@ -170,7 +176,21 @@ int ainfer_session_prefill(ainfer_session_t h, const int *tokens, int n, int sta
     int r = prefill_create(s, rows, false, &s->prefill, s->pf_rank, s->pf_world, s->pf_id);
     if (r) return set_err(r, s->err);
   }
+  return 0;
+}
+int ainfer_session_prefill(ainfer_session_t h, const int *tokens, int n, int start_pos) {
+  if (!h || (!tokens && n > 0)) return set_err(2, "usage: null argument");
+  Session *s = h->s;
+  if (int e = ensure_prefill(s)) return e;
   int r = prefill_run(s->prefill, tokens, n, start_pos, nullptr);
+  return set_err(r, s->err);
+}
+int ainfer_session_prefill_logits(ainfer_session_t h, const int *tokens, int n, int start_pos, const int *want, int n_want,
+                                  float *out) {
+  if (!h || (!tokens && n > 0) || (n_want > 0 && (!want || !out))) return set_err(2, "usage: null argument");
+  Session *s = h->s;
+  if (int e = ensure_prefill(s)) return e;
+  int r = prefill_logits(s->prefill, tokens, n, start_pos, want, n_want, out);
   return set_err(r, s->err);
 }
 int ainfer_session_prefill_rows(ainfer_session_t h, int rows) {
@@ -183,6 +203,7 @@ int ainfer_session_prefill_rows(ainfer_session_t h, int rows) {
 int ainfer_session_prefill_ep(ainfer_session_t h, const void *id128, int rank, int world) {
   if (!h) return set_err(2, "usage: null argument");
   Session *s = h->s;
+  if (s->rows && world > 1) return set_err(2, "usage: this architecture has no experts to split");
   if (world < 1 || world > 64 || 64 % world || rank < 0 || rank >= world || (world > 1 && !id128))
     return set_err(2, "usage: 0 <= rank < world, world divides 64, and an id for more than one rank");
   if (s->prefill) { prefill_destroy(s->prefill); s->prefill = nullptr; }
@@ -246,6 +267,7 @@ int ainfer_ep_unique_id(void *out128) {
 }
 int ainfer_ep_create(ainfer_model_t m, const void *id128, int rank, int world, int batch, int flags, ainfer_ep_t *out) {
   if (!m || !out) return set_err(2, "usage: null argument");
+  if (m->m->rows) return set_err(2, "usage: this architecture has no experts");
   *out = nullptr;
   ainfer_ep_s *h = new ainfer_ep_s;
   int r = h->e.create(m->m, id128, rank, world, batch, flags);
@@ -317,6 +339,8 @@ int ainfer_batch_buffer(ainfer_batch_t h, const char *which, void **dptr, uint64
   const ModelConfig &c = b.m->cfg;
   const std::string w = which;
   const uint64_t n = (uint64_t)b.n;
+  if (b.rows && b.rows->buffer(w, dptr, bytes)) return 0;
+  if (b.rows && w != "ctrl" && w != "out_tok" && w != "logits") return set_err(2, "unknown buffer: " + w);
   if (w == "ctrl") { *dptr = b.Ctrl; *bytes = n * 16; }
   else if (w == "out_tok") { *dptr = b.OutT; *bytes = n * 4; }
   else if (w == "logits") { *dptr = b.Logits; *bytes = n * c.vocab * 4; }

@@ -45,6 +45,7 @@ SIGNATURES = {
     "ainfer_host_free": (_i, [_vp, _vp]),
     "ainfer_memcpy_h2d_async": (_i, [_vp, _vp, _vp, _sz]),
     "ainfer_memcpy_d2h_async": (_i, [_vp, _vp, _vp, _sz]),
+    "ainfer_tensor_map_bf16": (_i, [_vp, _vp, _vp, _u64, _u64, _u64, _u32]),
     "ainfer_kernel_get": (_i, [_vp, C.c_char_p, _pp]),
     "ainfer_kernel_release": (_i, [_vp]),
     "ainfer_kernel_count": (_i, []),

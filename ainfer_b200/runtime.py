@@ -43,6 +43,7 @@ SIGNATURES = {
     "ainfer_session_buffer": (_i, [_vp, C.c_char_p, _pp, C.POINTER(_u64)]),
     "ainfer_session_step": (_i, [_vp, _i, _i, C.POINTER(_i)]),
     "ainfer_session_prefill": (_i, [_vp, C.POINTER(_i), _i, _i]),
+    "ainfer_session_prefill_logits": (_i, [_vp, _vp, _i, _i, _vp, _i, _vp]),
     "ainfer_session_prefill_ep": (_i, [_vp, C.c_char_p, _i, _i]),
     "ainfer_session_prefill_rows": (_i, [_vp, _i]),
     "ainfer_session_generate": (_i, [_vp, C.POINTER(_i), _i, _i, _i, C.POINTER(_i), C.POINTER(C.c_float)]),
@@ -156,6 +157,7 @@ class Session:
     MULTI_KERNEL = 4
     STAGE_CLOCK = 8
     PERSISTENT = 16
+    F32 = 32
 
     def __init__(self, model, max_ctx, flags=0):
         self.model = model
@@ -216,6 +218,13 @@ class Session:
         """Advances the state over the tokens in passes of up to 192 rows (no logits)."""
         t = np.ascontiguousarray(tokens, np.int32)
         _check(load().ainfer_session_prefill(self.h, t.ctypes.data_as(C.POINTER(C.c_int)), len(t), int(start_pos)))
+
+    def prefill_logits(self, tokens, want, start_pos=0):
+        """prefill that returns the logits [len(want)][V] of the listed rows (ascending indices into tokens)."""
+        t, w = np.ascontiguousarray(tokens, np.int32), np.ascontiguousarray(want, np.int32)
+        out = np.zeros((len(w), self.model.config["vocab"]), np.float32)
+        _check(load().ainfer_session_prefill_logits(self.h, t.ctypes.data, len(t), int(start_pos), w.ctypes.data, len(w), out.ctypes.data))
+        return out
 
     def prefill_rows(self, rows):
         """Rows per pass of the next prefill (rows x world x top-k <= 2048; default the largest multiple of 8 within that, at most 192)."""
@@ -340,6 +349,7 @@ class BatchDecode:
     """Batched decode (ainfer_batch_*): this rank owns batch/world sequences; every step advances
     each of them by one greedy token on the device."""
     ROUTER_BIAS = 1
+    F32 = 32
 
     def __init__(self, model, batch, max_ctx, rank=0, world=1, nccl_id=None, flags=0):
         self.model, self.dev = model, model.dev

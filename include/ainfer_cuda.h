@@ -79,6 +79,14 @@ int ainfer_host_free(ainfer_device_t dev, void *ptr);
 int ainfer_memcpy_h2d_async(ainfer_device_t dev, void *dst, const void *src, size_t bytes);
 int ainfer_memcpy_d2h_async(ainfer_device_t dev, void *dst, const void *src, size_t bytes);
 
+/* A bulk-copy descriptor ("tensor map") of a row-major bf16 matrix [rows][cols] whose rows are
+ * ld elements apart, copied in boxes of box_rows x 64 columns with the 128-byte swizzle (elements
+ * outside the matrix read as zero). map128 receives 128 bytes to pass as a kernel argument. base
+ * must be 16-byte aligned and ld a multiple of 8; 1 <= box_rows <= 256. No counterpart in the
+ * reference. */
+int ainfer_tensor_map_bf16(ainfer_device_t dev, void *map128, const void *base, uint64_t rows, uint64_t cols,
+                           uint64_t ld, uint32_t box_rows);
+
 /* zeModuleCreate + zeKernelCreate by entry name, decode_l0.cpp:376-447. Every
  * call returns a fresh handle with its own argument storage. */
 int ainfer_kernel_get(ainfer_device_t dev, const char *name, ainfer_kernel_t *out);

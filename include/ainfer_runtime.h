@@ -51,8 +51,10 @@ int ainfer_binfer_from_safetensors(const char *src, const char *arch_json, const
 const char *ainfer_preset_config_json(const char *preset);
 
 /* ---- model-loader (decode_l0.cpp:127-374) ---- */
-/* spec: path of a .binfer file, or "synth:<preset>[:seed=N]" to fill the same
- * tensors directly in device memory. */
+/* spec: path of a .binfer file; a folder with config.json, whose "architecture" picks the model
+ * class, and SafeTensors weights (model.safetensors, or shards with their index); or
+ * "synth:<preset>[:seed=N]" to fill the tensors of a named shape directly in device memory
+ * ("synth:config:<path of a config.json>[:seed=N]" takes the shape from a file). */
 int ainfer_model_open(ainfer_device_t dev, const char *spec, int validate_level, ainfer_model_t *out);
 int ainfer_model_close(ainfer_model_t m);
 const char *ainfer_model_config_json(ainfer_model_t m);
@@ -79,12 +81,17 @@ enum {
                                          programmatic dependencies: the default (flag kept for callers) */
   AINFER_SESSION_STAGE_CLOCK = 8,     /* persistent step (implies it): device timestamp after every grid
                                          barrier, read back through the "stage_stamps" buffer (u64 ns) */
-  AINFER_SESSION_PERSISTENT = 16      /* ONE persistent cooperative launch per token (DecodeStep) */
+  AINFER_SESSION_PERSISTENT = 16,     /* ONE persistent cooperative launch per token (DecodeStep); architectures
+                                         without one record a list instead */
+  AINFER_SESSION_F32 = 32             /* activations and cache in 32-bit, no reduced-precision products; code 2 for
+                                         architectures that compute on quantised activations */
 };
 int ainfer_session_create(ainfer_model_t m, int max_ctx, int flags, ainfer_session_t *out);
 int ainfer_session_destroy(ainfer_session_t s);
 int ainfer_session_reset(ainfer_session_t s);
-/* Device buffers of the session, for state upload/download by tests:
+/* Device buffers of the session, for state upload/download by tests (architectures with residual
+ * streams: "shift", "conv", "Kc", all layers of each, "state" for the three together, and the common
+ * "logits", "ctrl", "history"):
  * "conv", "S", "Kc", "Vc", "Ks", "Vs", "logits", "x", "ctrl", "layer_out",
  * "routed", "near_gap", "history", "stage_stamps". */
 int ainfer_session_buffer(ainfer_session_t s, const char *which, void **dptr, uint64_t *bytes);
@@ -99,6 +106,9 @@ int ainfer_session_generate(ainfer_session_t s, const int *prompt, int P, int G,
  * of tools/cmdlist/chunklayer_replay.cpp:366-443). The state afterwards is bit-identical to n calls
  * of ainfer_session_step; follow with ainfer_session_generate(s, &last_prompt_id, 1, G, start_pos + n, ...). */
 int ainfer_session_prefill(ainfer_session_t s, const int *tokens, int n, int start_pos);
+/* The same, returning the logits [n_want][V] (host) of the listed rows: indices into tokens, ascending. */
+int ainfer_session_prefill_logits(ainfer_session_t s, const int *tokens, int n, int start_pos, const int *want, int n_want,
+                                  float *out);
 /* Rows per pass of the next prefill object (1 <= rows, rows x world x top-k <= 2048; default: the
  * largest multiple of 8 within that bound, at most 192). Drops the current prefill object. */
 int ainfer_session_prefill_rows(ainfer_session_t s, int rows);
@@ -169,6 +179,9 @@ int ainfer_ep_moe_stack(ainfer_ep_t ep, int first, int count, float *seg_ms);
  * rest runs on the owner. Per sequence the arithmetic is the single-sequence token loop's
  * (tools/decode/decode_l0.cpp:742-825), so it decodes to the same tokens in a batch as alone. */
 typedef struct ainfer_batch_s *ainfer_batch_t;
+enum { AINFER_BATCH_F32 = 32 /* as AINFER_SESSION_F32; beside AINFER_EP_ROUTER_BIAS in `flags` */ };
+/* A sequence whose control block says position 0 starts anew, whatever its slot held before. (Models
+ * with residual streams; the INT4 hybrid's slots are zeroed by the caller.) */
 int ainfer_batch_create(ainfer_model_t m, const void *id128, int rank, int world, int batch, int max_ctx, int flags,
                         ainfer_batch_t *out);
 int ainfer_batch_destroy(ainfer_batch_t b);
