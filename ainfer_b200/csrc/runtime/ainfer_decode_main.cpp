@@ -5,9 +5,9 @@
 // tools/e2e/run_e2e.py, tools/stress/run_stress.py, tools/sweep/run_sweep.py)
 // can point at this binary instead.
 //
-//   ainfer_decode <model|synth:preset[:seed=N]> <P> <G> [kernel-dir] [report]
+//   ainfer_decode <model|folder|synth:preset[:seed=N]> <P> <G> [kernel-dir] [report]
 //                 [--ids=a,b,..] [--max-new=N] [--temp=T] [--top-k=K] [--top-p=P]
-//                 [--seed=S] [--rep-penalty=R] [--eos=a,b] [--device=N]
+//                 [--seed=S] [--rep-penalty=R] [--eos=a,b] [--device=N] [--dtype=float32]
 //   env: AINFER_MAXCTX, AINFER_PROFILE, AINFER_TOP5, AINFER_DUMP0
 // The fourth positional (the reference's SPIR-V directory) is accepted and
 // ignored: kernels are linked into the library.
@@ -39,6 +39,7 @@ int main(int argc, char **argv) {
   std::vector<int> opt_ids, eos = {248046, 248044};  // the reference's EOS pair, configurable
   int opt_max_new = -1, device = 0;
   SampleParams samp;
+  bool f32 = false;   // activations and cache in 32-bit, where the architecture has that form
   std::vector<const char *> pos;
   for (int i = 1; i < argc; ++i) {
     const char *a = argv[i];
@@ -51,6 +52,8 @@ int main(int argc, char **argv) {
     else if (!std::strncmp(a, "--rep-penalty=", 14)) samp.rep_penalty = (float)atof(a + 14);
     else if (!std::strncmp(a, "--eos=", 6)) eos = parse_ids(a + 6);
     else if (!std::strncmp(a, "--device=", 9)) device = atoi(a + 9);
+    else if (!std::strcmp(a, "--dtype=float32")) f32 = true;
+    else if (!std::strcmp(a, "--dtype=bfloat16")) f32 = false;
     else if (!std::strncmp(a, "--spvdir=", 9)) { /* accepted for compatibility */ }
     else pos.push_back(a);
   }
@@ -88,6 +91,7 @@ int main(int argc, char **argv) {
   int flags = 0;
   if (dump0) flags |= SESSION_DIAG;
   if (prof) flags |= SESSION_PER_LAYER_LISTS;
+  if (f32) flags |= SESSION_F32;
   Session *s = nullptr;
   rc = session_create(model, MAXCTX, flags, &s, err);
   if (rc) { std::fprintf(stderr, "%s\n", err.c_str()); return rc; }

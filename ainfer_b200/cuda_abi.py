@@ -174,6 +174,12 @@ class Device:
     def kernel(self, name):
         return Kernel(self, name)
 
+    def tensor_map_bf16(self, base, rows, cols, ld, box_rows):
+        """128 bytes of a bulk-copy descriptor of a bf16 matrix in device memory (ainfer_tensor_map_bf16)."""
+        buf = C.create_string_buffer(128)
+        self.check(self.L.ainfer_tensor_map_bf16(self.h, buf, base, rows, cols, ld, box_rows))
+        return buf.raw
+
     def sync(self, timeout_ns=2**64 - 1):
         self.check(self.L.ainfer_sync(self.h, timeout_ns))
 
@@ -222,6 +228,10 @@ class Kernel:
         """value: int device address / int / float. kind: 'ptr', 'i32', 'u64', 'f32' (guessed from
         the argument size and the Python type when omitted)."""
         size = self.sizes[index] if index < self.nargs else 0
+        if isinstance(value, bytes):    # a structure passed by value (a tensor map)
+            buf = C.create_string_buffer(value, len(value))
+            self.dev.check(self.dev.L.ainfer_kernel_set_arg(self.h, index, len(value), buf))
+            return
         if kind is None:
             if isinstance(value, float):
                 kind = "f32"

@@ -17,7 +17,7 @@ Without tokenizer assets a prompt is a list of token ids (or a string of ids sep
 and the completion text is the generated ids separated by spaces; with `--tokenizer tokenizer.json`
 (Hugging Face `tokenizers` format) text goes in and out.
 
-Usage: python -m ainfer_b200.server --model model.binfer|synth:<preset> [--port 8010] [--max-ctx 8192]
+Usage: python -m ainfer_b200.server --model model.binfer|folder|synth:<preset> [--port 8010] [--max-ctx 8192]
 """
 import argparse
 import json
@@ -71,15 +71,15 @@ class HfTokenizer:
 class Engine:
     """The persistent worker: one model, one session, one request at a time."""
 
-    def __init__(self, spec, max_ctx=8192, device=0):
+    def __init__(self, spec, max_ctx=8192, device=0, f32=False):
         from . import cuda_abi, runtime
         self.runtime = runtime
         self.dev = cuda_abi.Device(device)
         self.model = runtime.Model(self.dev, spec)
         self.vocab = self.model.config["vocab"]
-        self.max_ctx = max_ctx
-        self.sess = runtime.Session(self.model, max_ctx, runtime.Session.PERSISTENT)
-        self.model_id = spec.split("/")[-1]
+        self.max_ctx = min(max_ctx, self.model.config.get("max_positions", max_ctx))
+        self.sess = runtime.Session(self.model, max_ctx, runtime.Session.PERSISTENT | (runtime.Session.F32 if f32 else 0))
+        self.model_id = spec.rstrip("/").split("/")[-1]
 
     def generate(self, ids, max_new, samp, on_token=None):
         """ids: prompt token ids. Returns (generated ids, wall seconds)."""
@@ -225,12 +225,14 @@ def serve(engine, tokenizer, port=8010, host="127.0.0.1"):
 
 def main(argv=None):
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", required=True, help=".binfer path or synth:<preset>[:seed=N]")
+    ap.add_argument("--model", required=True, help=".binfer path, folder with config.json and SafeTensors weights, or synth:<preset>[:seed=N]")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                    help="activations and cache of models with bf16 weights (the INT4 models compute on INT8 activations)")
     ap.add_argument("--port", type=int, default=8010)
     ap.add_argument("--max-ctx", type=int, default=8192)
     ap.add_argument("--tokenizer", default=None, help="tokenizer.json (Hugging Face tokenizers); default: token ids as text")
     args = ap.parse_args(argv)
-    engine = Engine(args.model, args.max_ctx)
+    engine = Engine(args.model, args.max_ctx, f32=args.dtype == "float32")
     tok = HfTokenizer(args.tokenizer) if args.tokenizer else IdTokenizer(engine.vocab)
     srv = serve(engine, tok, args.port)
     print(f"serving {engine.model_id} on 127.0.0.1:{args.port}", flush=True)
