@@ -109,9 +109,10 @@ __device__ __forceinline__ float block_sum(float v, float *red) {
 __host__ __device__ __forceinline__ bool stream_vec(int S, int W) { return (W & 3) == 0 && S >= 1 && S <= 4; }
 
 template <int ST>
-__device__ __forceinline__ float stream_row(const float *src, const float *y, float *dst, const StreamCoef &c, int W, bool update, float *hs) {
+__device__ __forceinline__ float stream_row(const float *src, const float *y, float *dst, const StreamCoef &c, int W, bool update, float *hs,
+                                            int tid, int nth) {
   float ss = 0.0f;
-  for (int w = threadIdx.x * 4; w < W; w += blockDim.x * 4) {
+  for (int w = tid * 4; w < W; w += nth * 4) {
     float u[4];
     stream_step<ST, 4>(src + w, y + w, dst ? dst + w : nullptr, c, W, update, u);
     *reinterpret_cast<float4 *>(hs + w) = make_float4(u[0], u[1], u[2], u[3]);
@@ -120,17 +121,18 @@ __device__ __forceinline__ float stream_row(const float *src, const float *y, fl
   }
   return ss;
 }
-// One row of W elements: streams -> u in hs[] (each thread its own elements), returns this thread's sum of u^2.
+// One row of W elements over nth threads: streams -> u in hs[] (each thread its own elements); returns
+// this thread's sum of u^2.
 __device__ __forceinline__ float stream_row_any(const float *src, const float *y, float *dst, const StreamCoef &c, int S, int W, bool update,
-                                                float *hs) {
+                                                float *hs, int tid, int nth) {
   if (stream_vec(S, W)) {
-    if (S == 4) return stream_row<4>(src, y, dst, c, W, update, hs);
-    if (S == 3) return stream_row<3>(src, y, dst, c, W, update, hs);
-    if (S == 2) return stream_row<2>(src, y, dst, c, W, update, hs);
-    return stream_row<1>(src, y, dst, c, W, update, hs);
+    if (S == 4) return stream_row<4>(src, y, dst, c, W, update, hs, tid, nth);
+    if (S == 3) return stream_row<3>(src, y, dst, c, W, update, hs, tid, nth);
+    if (S == 2) return stream_row<2>(src, y, dst, c, W, update, hs, tid, nth);
+    return stream_row<1>(src, y, dst, c, W, update, hs, tid, nth);
   }
   float ss = 0.0f;
-  for (int w = threadIdx.x; w < W; w += blockDim.x) {
+  for (int w = tid; w < W; w += nth) {
     const float u = stream_step_n(src + w, y + w, dst ? dst + w : nullptr, c, S, W, update);
     hs[w] = u;
     ss = fmaf(u, u, ss);

@@ -40,9 +40,63 @@ struct ShortConvRowsArgs {
   int64_t kv_stride;
   int32_t rows, C, Qc, taps, cap, ldu, per;   // per: rows of a block
 };
-// grid = ceil(rows / per) x ceil(C / 256)
+// Four channels per thread, TAPS known, the last TAPS - 1 projections in registers.
+template <typename T>
+__device__ __forceinline__ void store4(T *p, const float4 v);
+template <>
+__device__ __forceinline__ void store4<float>(float *p, const float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+template <>
+__device__ __forceinline__ void store4<uint16_t>(uint16_t *p, const float4 v) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2((uint32_t)f32_to_bf16(v.x) | ((uint32_t)f32_to_bf16(v.y) << 16),
+                                             (uint32_t)f32_to_bf16(v.z) | ((uint32_t)f32_to_bf16(v.w) << 16));
+}
+template <typename T, int TAPS>
+__device__ __forceinline__ void short_conv4_body(const ShortConvRowsArgs &a) {
+  const int cb = (a.C + 1023) / 1024;
+  const int c = ((blockIdx.x % cb) * 256 + threadIdx.x) * 4, r0 = blockIdx.x / cb * a.per;
+  if (c >= a.C) return;
+  const int r1 = min(a.rows, r0 + a.per), Kn = a.C - a.Qc;
+  auto ld4 = [](const float *p) { return *reinterpret_cast<const float4 *>(p); };
+  float4 w[TAPS], win[TAPS];   // win[j]: the projection that tap j meets
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) w[j] = ld4(a.CW + (size_t)j * a.C + c);
+  int first = -1;
+  for (int r = r0; r < r1; ++r) {
+    const int pos = a.Ctrl[4 * r + CTRL_POS], seq = a.Seq[r], f = a.First[r];
+    if (f != first) {   // (re)load the history before row r
+      first = f;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int back = TAPS - 1 - j, p = pos - back;
+        win[j + 1] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (r - back >= f) win[j + 1] = ld4(a.U + (size_t)(r - back) * a.ldu + c);
+        else if (p >= 0) win[j + 1] = ld4(a.State + ((size_t)seq * TAPS + p % TAPS) * a.C + c);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
+    win[TAPS - 1] = ld4(a.U + (size_t)r * a.ldu + c);
+    float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      y.x = fmaf(w[j].x, win[j].x, y.x); y.y = fmaf(w[j].y, win[j].y, y.y);
+      y.z = fmaf(w[j].z, win[j].z, y.z); y.w = fmaf(w[j].w, win[j].w, y.w);
+    }
+    if (TAPS > 1 && (r + TAPS - 1 >= a.rows || a.First[r + TAPS - 1] != f))   // among the sequence's last TAPS - 1 rows
+      *reinterpret_cast<float4 *>(a.Pend + ((size_t)seq * TAPS + pos % TAPS) * a.C + c) = win[TAPS - 1];
+    if (c < a.Qc) store4(reinterpret_cast<T *>(a.Q) + (size_t)r * a.Qc + c, y);
+    else store4(reinterpret_cast<T *>(a.Kc) + (size_t)seq * a.kv_stride + (size_t)(pos % a.cap) * Kn + (c - a.Qc), y);
+  }
+}
+// grid = ceil(rows / per) x ceil(C / 1024) with whole quads of channels and 2..4 taps, else x ceil(C / 256)
 template <typename T>
 __device__ __forceinline__ void short_conv_body(const ShortConvRowsArgs &a) {
+  if ((a.C & 3) == 0 && (a.Qc & 3) == 0 && (a.ldu & 3) == 0 && a.taps >= 2 && a.taps <= 4) {
+    if (a.taps == 4) short_conv4_body<T, 4>(a);
+    else if (a.taps == 3) short_conv4_body<T, 3>(a);
+    else short_conv4_body<T, 2>(a);
+    return;
+  }
   const int cb = (a.C + 255) / 256;
   const int c = (blockIdx.x % cb) * 256 + threadIdx.x, r0 = blockIdx.x / cb * a.per;
   if (c >= a.C) return;

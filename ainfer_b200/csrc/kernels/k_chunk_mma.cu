@@ -1,0 +1,491 @@
+// Chunk-local shared-key attention (see k_chunk_attn.cu) in bf16 on the tensor cores, for head sizes
+// that are multiples of 8 up to 256. One tile of keys in shared memory serves both products: read
+// plainly it is the B operand of q . k, read transposed it is the B operand of weights . values.
+// Scores, the distance penalty, maxima, weights and sums are fp32; the weights are rounded to bf16
+// for the second product only.
+//
+//   ChunkAttnMma       rows of one sequence: a block takes 64 rows of one query head, a warp 16 rows
+//   ChunkAttnStepMma   a decode step of every sequence (up to 16 query heads per key head): the heads
+//                      are the 16 rows of the products, a warp takes 16 keys of every tile of 64
+#include <cuda_bf16.h>
+
+#include "hyper_core.cuh"
+
+namespace ainfer {
+
+constexpr int kCmKeys = 64;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ uint32_t cm_smem(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a) : "memory");
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(a)
+               : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack2(float lo, float hi) {
+  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<uint32_t *>(&v);
+}
+__device__ __forceinline__ void cpa16(uint32_t dst, const void *src, bool in) {   // out of range: zero fill
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cpa_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cpa_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// 64 keys [slot, slot + 64) of one key head into a tile of rows of DP + 8 values.
+template <int DP, int THREADS>
+__device__ __forceinline__ void load_keys(uint32_t dst, const uint16_t *K, int slot, int KW, int D) {
+  constexpr int P = DP / 8;
+  for (int i = threadIdx.x; i < kCmKeys * P; i += THREADS) {
+    const int r = i / P, c = i % P;
+    const bool in = c * 8 < D;
+    cpa16(dst + (uint32_t)(r * (DP + 8) + c * 8) * 2, K + (size_t)(slot + r) * KW + (in ? c * 8 : 0), in);
+  }
+}
+
+// One warp, 16 rows against NK keys of a tile at `kt`: s[n] = products with keys 8n .. 8n+7.
+template <int DP, int NK>
+__device__ __forceinline__ void scores(float (&s)[NK / 8][4], const uint32_t (&q)[DP / 16][4], uint32_t kt, int lane) {
+#pragma unroll
+  for (int n = 0; n < NK / 8; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) s[n][i] = 0.0f;
+  const uint32_t a = kt + (uint32_t)(((lane & 7) + ((lane >> 4) & 1) * 8) * (DP + 8) + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+  for (int kk = 0; kk < DP / 16; ++kk)
+#pragma unroll
+    for (int n = 0; n < NK / 16; ++n) {
+      uint32_t b[4];
+      ldm4(b, a + (uint32_t)(n * 16 * (DP + 8) + kk * 16) * 2);
+      mma16816(s[2 * n], q[kk], b[0], b[1]);
+      mma16816(s[2 * n + 1], q[kk], b[2], b[3]);
+    }
+}
+// o += weights (as the score fragments hold them) . keys of the tile
+template <int DP, int NK>
+__device__ __forceinline__ void values(float (&o)[DP / 8][4], const float (&p)[NK / 8][4], uint32_t kt, int lane) {
+  const uint32_t a = kt + (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * (DP + 8) + ((lane >> 4) & 1) * 8) * 2;
+#pragma unroll
+  for (int j = 0; j < NK / 16; ++j) {
+    const uint32_t w[4] = {pack2(p[2 * j][0], p[2 * j][1]), pack2(p[2 * j][2], p[2 * j][3]), pack2(p[2 * j + 1][0], p[2 * j + 1][1]),
+                           pack2(p[2 * j + 1][2], p[2 * j + 1][3])};
+#pragma unroll
+    for (int d = 0; d < DP / 16; ++d) {
+      uint32_t b[4];
+      ldm4t(b, a + (uint32_t)(j * 16 * (DP + 8) + d * 16) * 2);
+      mma16816(o[2 * d], w, b[0], b[1]);
+      mma16816(o[2 * d + 1], w, b[2], b[3]);
+    }
+  }
+}
+__device__ __forceinline__ float quad_max(float v) {
+  v = fmaxf(v, __shfl_xor_sync(kFull, v, 1));
+  return fmaxf(v, __shfl_xor_sync(kFull, v, 2));
+}
+__device__ __forceinline__ float quad_sum(float v) {
+  v = v + __shfl_xor_sync(kFull, v, 1);
+  return v + __shfl_xor_sync(kFull, v, 2);
+}
+
+// ------------------------------------------------------- ChunkAttnMma ---
+struct ChunkAttnMmaArgs {
+  const uint16_t *Q;       // [rows][H D]
+  const uint16_t *Kc;      // [cap][G D], cap a multiple of 64
+  const float *LB;         // [H][lb_len]
+  const float *Temp;       // [H]
+  const int32_t *Ctrl;     // [rows][4]
+  uint16_t *O;             // [rows][ldo]
+  int32_t rows, H, G, D, cap, chunk, lb_len, ldo;
+  float scale;
+};
+constexpr int kCmRows = 64;
+template <int DP>
+__device__ __forceinline__ void chunk_attn_mma_body(const ChunkAttnMmaArgs &a) {
+  extern __shared__ __align__(128) unsigned char cm_raw[];
+  constexpr int LD = DP + 8;
+  uint16_t *Qs = reinterpret_cast<uint16_t *>(cm_raw);
+  uint16_t *Ks = Qs + kCmRows * LD;                                   // [2][64][LD]
+  float *lbw = reinterpret_cast<float *>(Ks + 2 * kCmKeys * LD);      // [2][128] penalty by row - key + 63
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int tiles = (a.rows + kCmRows - 1) / kCmRows;
+  const int h = blockIdx.x % a.H, r0 = (tiles - 1 - blockIdx.x / a.H) * kCmRows, g = h / (a.H / a.G);   // long rows first
+  const int nr = min(kCmRows, a.rows - r0), KW = a.G * a.D;
+  const uint32_t qa = cm_smem(Qs), ka = cm_smem(Ks);
+  {
+    constexpr int P = DP / 8;
+    for (int i = tid; i < kCmRows * P; i += 128) {
+      const int r = i / P, c = i % P;
+      const bool in = r < nr && c * 8 < a.D;
+      cpa16(qa + (uint32_t)(r * LD + c * 8) * 2, a.Q + (in ? (size_t)(r0 + r) * a.H * a.D + (size_t)h * a.D + c * 8 : 0), in);
+    }
+  }
+  const int p0 = a.Ctrl[4 * r0 + CTRL_POS], p1 = p0 + nr - 1;
+  const int lo = p0 - p0 % a.chunk, kb0 = lo / kCmKeys * kCmKeys;
+  const uint16_t *K = a.Kc + (size_t)g * a.D;
+  const float *lb = a.LB + (size_t)h * a.lb_len;
+  auto fetch = [&](int k0, int b) {
+    load_keys<DP, 128>(ka + (uint32_t)(b * kCmKeys * LD) * 2, K, k0 % a.cap, KW, a.D);
+    const int d = p0 - k0 - 63 + tid;   // distance of entry tid (127 used)
+    lbw[b * 128 + tid] = lb[min(max(d, 0), a.lb_len - 1)] * kLog2e;
+    cpa_commit();
+  };
+  fetch(kb0, 0);
+  const float mul = a.scale * a.Temp[h] * kLog2e;
+  uint32_t q[DP / 16][4];
+  float o[DP / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+#pragma unroll
+  for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o[d][i] = 0.0f;
+  const int rw = warp * 16 + (lane >> 2);                 // this thread's rows rw and rw + 8
+  const int pr[2] = {p0 + rw, p0 + rw + 8};
+  const int cs[2] = {pr[0] - pr[0] % a.chunk, pr[1] - pr[1] % a.chunk};
+  const int cs_last = p1 - p1 % a.chunk;
+  bool first = true;
+  int b = 0;
+  for (int k0 = kb0; k0 <= p1; k0 += kCmKeys) {
+    const bool more = k0 + kCmKeys <= p1;
+    if (more) fetch(k0 + kCmKeys, b ^ 1);
+    if (more) cpa_wait<1>(); else cpa_wait<0>();
+    __syncthreads();
+    if (first) {
+#pragma unroll
+      for (int kk = 0; kk < DP / 16; ++kk) ldm4(q[kk], qa + (uint32_t)((warp * 16 + (lane & 15)) * LD + kk * 16 + (lane >> 4) * 8) * 2);
+      first = false;
+    }
+    float s[kCmKeys / 8][4];
+    const uint32_t kt = ka + (uint32_t)(b * kCmKeys * LD) * 2;
+    scores<DP, kCmKeys>(s, q, kt, lane);
+    const bool whole = k0 + kCmKeys - 1 <= p0 && k0 >= cs_last;   // every row sees every key of the tile
+    const float *lw = lbw + b * 128;
+    float mx[2] = {m[0], m[1]};
+#pragma unroll
+    for (int n = 0; n < kCmKeys / 8; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int x = i >> 1, kc = n * 8 + (lane & 3) * 2 + (i & 1), key = k0 + kc;
+        float v = fmaf(s[n][i], mul, -lw[rw + 8 * x - kc + 63]);
+        if (!whole && (key > pr[x] || key < cs[x])) v = -INFINITY;
+        s[n][i] = v;
+        mx[x] = fmaxf(mx[x], v);
+      }
+    float corr[2], base[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      mx[x] = quad_max(mx[x]);
+      base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
+      corr[x] = exp2f(m[x] - base[x]);
+      m[x] = mx[x];
+    }
+    float sum[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int n = 0; n < kCmKeys / 8; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        s[n][i] = exp2f(s[n][i] - base[i >> 1]);
+        sum[i >> 1] += s[n][i];
+      }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) l[x] = fmaf(l[x], corr[x], sum[x]);
+#pragma unroll
+    for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+    values<DP, kCmKeys>(o, s, kt, lane);
+    __syncthreads();
+    b ^= 1;
+  }
+#pragma unroll
+  for (int x = 0; x < 2; ++x) l[x] = 1.0f / quad_sum(l[x]);
+#pragma unroll
+  for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int r = rw + 8 * x, c = d * 8 + (lane & 3) * 2;
+      if (r < nr && c < a.D) *reinterpret_cast<uint32_t *>(a.O + (size_t)(r0 + r) * a.ldo + (size_t)h * a.D + c) = pack2(o[d][2 * x] * l[x], o[d][2 * x + 1] * l[x]);
+    }
+}
+__host__ __device__ inline int cm_pad(int D) { return D <= 32 ? 32 : D <= 64 ? 64 : D <= 96 ? 96 : D <= 128 ? 128 : D <= 192 ? 192 : 256; }
+#define CHUNK_MMA(DP, BLOCKS)                                                                             \
+  __global__ void __launch_bounds__(128, BLOCKS) ChunkAttnMma##DP(const __grid_constant__ ChunkAttnMmaArgs a) { \
+    pdl_launch_dependents();                                                                              \
+    pdl_wait();                                                                                           \
+    chunk_attn_mma_body<DP>(a);                                                                           \
+  }                                                                                                       \
+  static uint32_t chunk_mma_smem##DP(const void *) { return (kCmRows + 2 * kCmKeys) * (DP + 8) * 2 + 2 * 128 * 4; }
+CHUNK_MMA(32, 4)
+CHUNK_MMA(64, 4)
+CHUNK_MMA(96, 3)
+CHUNK_MMA(128, 3)
+CHUNK_MMA(192, 2)
+CHUNK_MMA(256, 2)
+#define F(f) AINFER_ARG(ChunkAttnMmaArgs, f)
+#define CM_FIELDS F(Q), F(Kc), F(LB), F(Temp), F(Ctrl), F(O), F(rows), F(H), F(G), F(D), F(cap), F(chunk), F(lb_len), F(ldo), F(scale)
+#define CM_REGISTER(DP) AINFER_REGISTER(ChunkAttnMma##DP, ChunkAttnMmaArgs, 128, 0, 0, chunk_mma_smem##DP, CM_FIELDS); AINFER_EARLY_LAUNCH(ChunkAttnMma##DP)
+CM_REGISTER(32);
+CM_REGISTER(64);
+CM_REGISTER(96);
+CM_REGISTER(128);
+CM_REGISTER(192);
+CM_REGISTER(256);
+#undef F
+
+// --------------------------------------------------- ChunkAttnStepMma ---
+struct ChunkAttnStepMmaArgs {
+  const float *U;          // [seq][ldu]
+  const float *CW;         // [taps][C]
+  float *State;            // [seq][taps][C]
+  const int32_t *Ctrl;     // [seq][4]
+  uint16_t *Kc;
+  int64_t kv_stride;
+  const float *LB;         // [H][lb_len]
+  const float *Temp;       // [H]
+  float *Part;             // [seq][G][splits][HG (D + 2)]
+  uint32_t *Count;         // [seq][G], zero between launches
+  void *O;                 // [seq][ldo]
+  int32_t nseq, H, G, D, taps, cap, chunk, lb_len, splits, ldu, ldo, out16;
+  float scale;
+};
+constexpr int kSmStages = 3;
+template <int DP>
+__device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &a) {
+  extern __shared__ __align__(128) unsigned char sm_raw[];
+  __shared__ float wm[4][16], wl[4][16];
+  __shared__ int s_last;
+  constexpr int LD = DP + 8;
+  uint16_t *Qs = reinterpret_cast<uint16_t *>(sm_raw);                // [16][LD]
+  uint16_t *kn = Qs + 16 * LD;                                        // the new key [DP]
+  uint16_t *Ks = kn + LD;                                             // [stages][64][LD]
+  const int D = a.D, HG = a.H / a.G, C = (a.H + a.G) * D, Qc = a.H * D, KW = a.G * D;
+  const int split = blockIdx.x % a.splits, g = blockIdx.x / a.splits % a.G, seq = blockIdx.x / (a.splits * a.G);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int pos = a.Ctrl[4 * seq + CTRL_POS], lo = pos - pos % a.chunk;
+  const int t_lo = lo / kCmKeys, t_hi = pos / kCmKeys, nt = t_hi - t_lo + 1;
+  const int per = (nt + a.splits - 1) / a.splits, active = (nt + per - 1) / per;
+  if (split >= active) return;
+  const int t0 = t_lo + split * per, t1 = min(t_hi, t0 + per - 1);
+  uint16_t *K = a.Kc + (size_t)seq * a.kv_stride + (size_t)g * D;
+  const uint32_t ka = cm_smem(Ks);
+  auto fetch = [&](int t) {
+    if (t <= t1) load_keys<DP, 128>(ka + (uint32_t)(((t - t0) % kSmStages) * kCmKeys * LD) * 2, K, t * kCmKeys % a.cap, KW, D);
+    cpa_commit();
+  };
+  for (int i = 0; i < kSmStages - 1; ++i) fetch(t0 + i);
+  // ---- convolution of this key head's channels (its query heads, then the key) ----
+  for (int i = tid; i < 16 * LD; i += 128) Qs[i] = 0;
+  __syncthreads();
+  float *st = a.State + (size_t)seq * a.taps * C;
+  const float *u0 = a.U + (size_t)seq * a.ldu;
+  for (int i = tid; i < (HG + 1) * D; i += 128) {
+    const bool isk = i >= HG * D;
+    const int c = isk ? Qc + g * D + (i - HG * D) : g * HG * D + i;
+    float y = 0.0f;
+    for (int j = 0; j < a.taps - 1; ++j) {
+      const int p = pos - (a.taps - 1 - j);
+      if (p >= 0) y = fmaf(a.CW[(size_t)j * C + c], st[(size_t)(p % a.taps) * C + c], y);
+    }
+    const float u = u0[c];
+    y = fmaf(a.CW[(size_t)(a.taps - 1) * C + c], u, y);
+    if (split == 0) st[(size_t)(pos % a.taps) * C + c] = u;
+    const uint16_t v = f32_to_bf16(y);
+    if (isk) kn[i - HG * D] = v;
+    else Qs[(i / D) * LD + i % D] = v;
+  }
+  __syncthreads();
+  uint32_t q[DP / 16][4];
+#pragma unroll
+  for (int kk = 0; kk < DP / 16; ++kk) ldm4(q[kk], cm_smem(Qs) + (uint32_t)((lane & 15) * LD + kk * 16 + (lane >> 4) * 8) * 2);
+  float o[DP / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, mul[2];
+  const float *lb[2];
+#pragma unroll
+  for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o[d][i] = 0.0f;
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int h = g * HG + min((lane >> 2) + 8 * x, HG - 1);   // rows past the head count repeat the last head
+    mul[x] = a.scale * a.Temp[h] * kLog2e;
+    lb[x] = a.LB + (size_t)h * a.lb_len;
+  }
+  for (int t = t0; t <= t1; ++t) {
+    const int k0 = t * kCmKeys + warp * 16;
+    float pen[2][2][2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) pen[x][n][e] = __ldg(lb[x] + min(max(pos - (k0 + n * 8 + (lane & 3) * 2 + e), 0), a.lb_len - 1));
+    cpa_wait<kSmStages - 2>();
+    __syncthreads();
+    if (t == t_hi) {   // the step's own key: into the tile and the cache
+      uint16_t *row = Ks + ((t - t0) % kSmStages) * kCmKeys * LD + (pos % kCmKeys) * LD;
+      for (int i = tid; i < D; i += 128) {
+        row[i] = kn[i];
+        K[(size_t)(pos % a.cap) * KW + i] = kn[i];
+      }
+      __syncthreads();
+    }
+    fetch(t + kSmStages - 1);
+    const uint32_t kt = ka + (uint32_t)((((t - t0) % kSmStages) * kCmKeys + warp * 16) * LD) * 2;
+    float s[2][4];
+    scores<DP, 16>(s, q, kt, lane);
+    float mx[2] = {m[0], m[1]};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int x = i >> 1, key = k0 + n * 8 + (lane & 3) * 2 + (i & 1);
+        float v = fmaf(s[n][i], mul[x], -pen[x][n][i & 1] * kLog2e);
+        if (key > pos || key < lo) v = -INFINITY;
+        s[n][i] = v;
+        mx[x] = fmaxf(mx[x], v);
+      }
+    float corr[2], sum[2] = {0.0f, 0.0f}, base[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      mx[x] = quad_max(mx[x]);
+      base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
+      corr[x] = exp2f(m[x] - base[x]);
+      m[x] = mx[x];
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        s[n][i] = exp2f(s[n][i] - base[i >> 1]);
+        sum[i >> 1] += s[n][i];
+      }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) l[x] = fmaf(l[x], corr[x], sum[x]);
+#pragma unroll
+    for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+    values<DP, 16>(o, s, kt, lane);
+  }
+  cpa_wait<0>();
+  // ---- the four warps' shares of this block ----
+  float *os = reinterpret_cast<float *>(Ks);   // [4][16][DP], in the key tiles' place
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int r = (lane >> 2) + 8 * x;
+    l[x] = quad_sum(l[x]);
+    if ((lane & 3) == 0) { wm[warp][r] = m[x]; wl[warp][r] = l[x]; }
+    if (r < HG)
+#pragma unroll
+      for (int d = 0; d < DP / 8; ++d) *reinterpret_cast<float2 *>(os + (warp * 16 + r) * DP + d * 8 + (lane & 3) * 2) = make_float2(o[d][2 * x], o[d][2 * x + 1]);
+  }
+  __syncthreads();
+  auto put = [&](int h, int d, float v) {
+    const size_t at = (size_t)seq * a.ldo + (size_t)h * D + d;
+    if (a.out16) reinterpret_cast<uint16_t *>(a.O)[at] = f32_to_bf16(v);
+    else reinterpret_cast<float *>(a.O)[at] = v;
+  };
+  const int per_head = D + 2;
+  float *base_p = a.Part + ((size_t)seq * a.G + g) * a.splits * HG * per_head;
+  float *mine = base_p + (size_t)split * HG * per_head;
+  for (int i = tid; i < HG * D; i += 128) {
+    const int hh = i / D, d = i - hh * D;
+    const float M = fmaxf(fmaxf(wm[0][hh], wm[1][hh]), fmaxf(wm[2][hh], wm[3][hh]));
+    float v = 0.0f, L = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = exp2f(wm[w][hh] - M);
+      v = fmaf(os[(w * 16 + hh) * DP + d], f, v);
+      L = fmaf(wl[w][hh], f, L);
+    }
+    if (active == 1) {
+      put(g * HG + hh, d, v / L);
+    } else {
+      __stcg(mine + (size_t)hh * per_head + 2 + d, v);
+      if (d == 0) { __stcg(mine + (size_t)hh * per_head, M); __stcg(mine + (size_t)hh * per_head + 1, L); }
+    }
+  }
+  if (active == 1) return;
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    const uint32_t n = atomicAdd(a.Count + (size_t)seq * a.G + g, 1u);
+    s_last = n + 1 == (uint32_t)active;
+    if (s_last) a.Count[(size_t)seq * a.G + g] = 0;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  // split factors of every head, then the sums: loads of all splits are independent
+  float *fac = os;   // [HG][active] exp2(m_s - M), then [HG] 1 / L behind them
+  for (int hh = warp; hh < HG; hh += 4) {
+    float M = -INFINITY;
+    for (int s = lane; s < active; s += 32) M = fmaxf(M, __ldcg(base_p + ((size_t)s * HG + hh) * per_head));
+    M = warp_max(M);
+    float L = 0.0f;
+    for (int s = lane; s < active; s += 32) {
+      const float *p = base_p + ((size_t)s * HG + hh) * per_head;
+      const float f = exp2f(__ldcg(p) - M);
+      fac[hh * active + s] = f;
+      L = fmaf(__ldcg(p + 1), f, L);
+    }
+    L = warp_tree_sum(L);
+    if (lane == 0) wm[hh & 3][hh >> 2] = 1.0f / L;
+  }
+  __syncthreads();
+  for (int i = tid; i < HG * D; i += 128) {
+    const int hh = i / D, d = i - hh * D;
+    const float *p = base_p + (size_t)hh * per_head + 2 + d, *f = fac + hh * active;
+    const size_t stride = (size_t)HG * per_head;
+    float v = 0.0f;
+    int s = 0;
+    for (; s + 8 <= active; s += 8) {
+      float x[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[k] = __ldcg(p + (size_t)(s + k) * stride);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v = fmaf(x[k], f[s + k], v);
+    }
+    for (; s < active; ++s) v = fmaf(__ldcg(p + (size_t)s * stride), f[s], v);
+    put(g * HG + hh, d, v * wm[hh & 3][hh >> 2]);
+  }
+}
+#define CHUNK_STEP(DP)                                                                                                  \
+  __global__ void __launch_bounds__(128) ChunkAttnStepMma##DP(const __grid_constant__ ChunkAttnStepMmaArgs a) {         \
+    pdl_launch_dependents();                                                                                            \
+    pdl_wait();                                                                                                         \
+    chunk_step_mma_body<DP>(a);                                                                                         \
+  }                                                                                                                     \
+  static uint32_t chunk_step_smem##DP(const void *) {                                                                   \
+    return (16 + 1 + kSmStages * kCmKeys) * (DP + 8) * 2;                                                               \
+  }                                                                                                                     \
+  static_assert(kSmStages * kCmKeys * (DP + 8) * 2 >= 4 * 16 * DP * 4 && 16 * 64 <= 4 * 16 * DP, "merge buffers lie in the key tiles' place");
+CHUNK_STEP(32)
+CHUNK_STEP(64)
+CHUNK_STEP(96)
+CHUNK_STEP(128)
+CHUNK_STEP(192)
+CHUNK_STEP(256)
+#define F(f) AINFER_ARG(ChunkAttnStepMmaArgs, f)
+#define CS_FIELDS                                                                                                                  \
+  F(U), F(CW), F(State), F(Ctrl), F(Kc), F(kv_stride), F(LB), F(Temp), F(Part), F(Count), F(O), F(nseq), F(H), F(G), F(D), F(taps), \
+      F(cap), F(chunk), F(lb_len), F(splits), F(ldu), F(ldo), F(out16), F(scale)
+#define CS_REGISTER(DP) \
+  AINFER_REGISTER(ChunkAttnStepMma##DP, ChunkAttnStepMmaArgs, 128, 0, 0, chunk_step_smem##DP, CS_FIELDS); AINFER_EARLY_LAUNCH(ChunkAttnStepMma##DP)
+CS_REGISTER(32);
+CS_REGISTER(64);
+CS_REGISTER(96);
+CS_REGISTER(128);
+CS_REGISTER(192);
+CS_REGISTER(256);
+#undef F
+
+}  // namespace ainfer

@@ -79,7 +79,7 @@ __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
     if (a.Idx) r = a.Idx[r];
     const float *src = a.Xin + (size_t)r * a.S * W;
     float *dst = own && a.Xout ? a.Xout + (size_t)r * a.S * W : nullptr;
-    const float ss = stream_row_any(src, a.Y + (update ? (size_t)r * W : 0), dst, coef, a.S, W, update, hs);
+    const float ss = stream_row_any(src, a.Y + (update ? (size_t)r * W : 0), dst, coef, a.S, W, update, hs, tid, 256);
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)W + a.eps);
     // every thread touches only the elements it wrote
     if (vec) {

@@ -7,6 +7,7 @@
 //                     makes the row for itself; block 0 stores the updated streams and the shift row)
 // act: 0 none, 1 relu squared, 2 cap tanh(v / cap).
 #include "hyper_core.cuh"
+#include "weight_ring.cuh"
 
 namespace ainfer {
 
@@ -72,21 +73,51 @@ AINFER_REGISTER(LinearRows, LinearRowsArgs, 256, 0, 0, nullptr, F(X), F(W), F(Bi
 #undef F
 
 // ---------------------------------------------------------- StreamGemv ---
-constexpr int kSgThreads = 512, kSgWarps = kSgThreads / 32;
-constexpr int kSgPre = 2;   // 16-byte pieces of each of a warp's two rows fetched before the dependency wait
-
+// The block's rows are one contiguous range of bytes: a producer warp brings them in tiles of whole rows
+// (about 16 KB) through a ring of shared-memory stages with bulk copies, which start before the kernel's
+// dependency wait (weights do not depend on it); 16 consumer warps multiply. Per tile a row is shared
+// by wpr warps; the partial sums of all rows stay in shared memory until the block's last tile.
+constexpr int kSgWarps = 16, kSgThreads = kSgWarps * 32 + 32, kSgRing = 65536;
+constexpr uint32_t kSgSpin = 1u << 22;
+struct GemvDims { int tile_rows, stage_bytes, nst, wpr; };
+__host__ __device__ inline GemvDims gemv_dims(int ldw) {
+  GemvDims d;
+  d.tile_rows = 16384 / (ldw * 2);
+  if (d.tile_rows < 1) d.tile_rows = 1;
+  if (d.tile_rows > 64) d.tile_rows = 64;
+  d.stage_bytes = d.tile_rows * ldw * 2;
+  d.nst = kSgRing / d.stage_bytes;
+  if (d.nst < 2) d.nst = 2;
+  if (d.nst > 8) d.nst = 8;
+  d.wpr = 1;
+  while (d.wpr * 2 * d.tile_rows <= kSgWarps && d.wpr * 256 < ldw) d.wpr *= 2;
+  return d;
+}
 // The vector in shared memory, split so that a lane's eight values come from two conflict-free
 // 16-byte reads: element k of piece k / 8 lies in half (k / 4) % 2 at (k / 8) * 4 + k % 4.
 __device__ __forceinline__ void sg_put(float *lo, float *hi, int k, float v) { ((k & 4) ? hi : lo)[(k >> 3) * 4 + (k & 3)] = v; }
-__host__ __device__ inline uint32_t sg_half(uint32_t ldw) { return ldw / 2; }
 
 struct GemvShape {
   const uint16_t *W;
   const float *Bias;
   float *Y;
-  int32_t N, ldw, wpr, act;   // wpr: warps that share a pair of rows (1, 2, 4 or 8)
+  int32_t N, ldw, rows_pb, act;   // rows_pb: rows of a block
   float cap;
 };
+struct GemvShared {
+  unsigned long long full[8], empty[8];
+  uint32_t fail;
+};
+__device__ __forceinline__ bool sg_wait(GemvShared *s, unsigned long long *b, uint32_t parity) {
+  if (mbar_try(b, parity)) return true;
+  for (uint32_t i = 0; i < kSgSpin; ++i) {
+    if (mbar_try(b, parity)) return true;
+    if (*reinterpret_cast<volatile uint32_t *>(&s->fail)) return false;
+  }
+  *reinterpret_cast<volatile uint32_t *>(&s->fail) = 1;
+  if (g_stream_fault_word) *reinterpret_cast<volatile unsigned int *>(g_stream_fault_word) = 1;
+  return false;
+}
 __device__ __forceinline__ float dot8(const uint4 w, const float4 a, const float4 b, float s) {
   s = fmaf(u2f(w.x << 16), a.x, s); s = fmaf(u2f(w.x & 0xFFFF0000u), a.y, s);
   s = fmaf(u2f(w.y << 16), a.z, s); s = fmaf(u2f(w.y & 0xFFFF0000u), a.w, s);
@@ -94,66 +125,80 @@ __device__ __forceinline__ float dot8(const uint4 w, const float4 a, const float
   s = fmaf(u2f(w.w << 16), b.z, s); s = fmaf(u2f(w.w & 0xFFFF0000u), b.w, s);
   return s;
 }
-struct GemvFirst { uint4 w[2][kSgPre]; };
-// This warp's first pair of rows and its first pieces of them.
-__device__ __forceinline__ void gemv_prefetch(const GemvShape &c, GemvFirst &f) {
+__device__ __forceinline__ void gemv_init(GemvShared *sh, int nst) {
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < nst; ++i) { mbar_init(&sh->full[i], 1); mbar_init(&sh->empty[i], kSgWarps); }
+    sh->fail = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+}
+// The producer warp's whole work; then it waits at the block's last barrier like everyone.
+__device__ __forceinline__ void gemv_produce(const GemvShape &c, const GemvDims &d, GemvShared *sh, unsigned char *ring) {
+  if ((threadIdx.x & 31) == 0) {
+    const int n0 = blockIdx.x * c.rows_pb, n1 = min(c.N, n0 + c.rows_pb);
+    uint32_t st = 0, ph = 1, issued = 0;
+    for (int n = n0; n < n1; n += d.tile_rows) {
+      if (!sg_wait(sh, &sh->empty[st], ph)) break;
+      const uint32_t bytes = (uint32_t)min(d.tile_rows, n1 - n) * (uint32_t)c.ldw * 2u;
+      mbar_arrive_expect(&sh->full[st], bytes);
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                       smem_addr(ring + (size_t)st * d.stage_bytes)),
+                   "l"(c.W + (size_t)n * c.ldw), "r"(bytes), "r"(smem_addr(&sh->full[st]))
+                   : "memory");
+      ++issued;
+      if (++st == (uint32_t)d.nst) { st = 0; ph ^= 1; }
+    }
+    if (*reinterpret_cast<volatile uint32_t *>(&sh->fail))   // copies in flight land before the block may end
+      for (int i = 0; i < d.nst && (uint32_t)i < issued; ++i) {
+        const uint32_t uses = (issued - (uint32_t)i + (uint32_t)d.nst - 1) / (uint32_t)d.nst;
+        for (uint32_t s = 0; s < kSgSpin && !mbar_try(&sh->full[i], (uses - 1) & 1); ++s) {}
+      }
+  }
+  __syncwarp();
+}
+__device__ __forceinline__ void gemv_consume(const GemvShape &c, const GemvDims &d, GemvShared *sh, const unsigned char *ring, const float *lo,
+                                             const float *hi, float *part) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pieces = c.ldw >> 3;
-  const int pair = blockIdx.x * (kSgWarps / c.wpr) + warp / c.wpr, part = warp % c.wpr;
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int n = min(2 * pair + i, c.N - 1);
-    const uint4 *row = reinterpret_cast<const uint4 *>(c.W + (size_t)n * c.ldw);
-#pragma unroll
-    for (int j = 0; j < kSgPre; ++j) f.w[i][j] = __ldg(row + min(part * 32 + lane + 32 * c.wpr * j, pieces - 1));
+  const int n0 = blockIdx.x * c.rows_pb, n1 = min(c.N, n0 + c.rows_pb), mine = warp % d.wpr, r_step = kSgWarps / d.wpr;
+  uint32_t st = 0, ph = 0;
+  for (int n = n0; n < n1; n += d.tile_rows) {
+    const int nr = min(d.tile_rows, n1 - n);
+    sg_wait(sh, &sh->full[st], ph);
+    __syncwarp();
+    const unsigned char *tile = ring + (size_t)st * d.stage_bytes;
+    for (int r = warp / d.wpr; r < nr; r += r_step) {
+      const uint4 *row = reinterpret_cast<const uint4 *>(tile + (size_t)r * c.ldw * 2);
+      float s0 = 0.0f, s1 = 0.0f;
+      int i = mine * 32 + lane;
+      const int step = 32 * d.wpr;
+      for (; i + step < pieces; i += 2 * step) {
+        s0 = dot8(row[i], *reinterpret_cast<const float4 *>(lo + 4 * i), *reinterpret_cast<const float4 *>(hi + 4 * i), s0);
+        const int k = i + step;
+        s1 = dot8(row[k], *reinterpret_cast<const float4 *>(lo + 4 * k), *reinterpret_cast<const float4 *>(hi + 4 * k), s1);
+      }
+      if (i < pieces) s0 = dot8(row[i], *reinterpret_cast<const float4 *>(lo + 4 * i), *reinterpret_cast<const float4 *>(hi + 4 * i), s0);
+      s0 = warp_tree_sum(s0 + s1);
+      if (lane == 0) part[(n - n0 + r) * d.wpr + mine] = s0;
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&sh->empty[st]);
+    if (++st == (uint32_t)d.nst) { st = 0; ph ^= 1; }
   }
 }
-__device__ __forceinline__ void gemv_body(const GemvShape &c, const float *lo, const float *hi, float *part_sum, const GemvFirst &f) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pieces = c.ldw >> 3;
-  const int gpb = kSgWarps / c.wpr, pairs = (c.N + 1) / 2, part = warp % c.wpr, step = 32 * c.wpr;
-  bool first = true;
-  for (int p0 = blockIdx.x * gpb; p0 < pairs; p0 += gridDim.x * gpb) {
-    const int pair = p0 + warp / c.wpr;
-    float s0 = 0.0f, s1 = 0.0f;
-    if (pair < pairs) {
-      const int n0 = 2 * pair, n1 = min(2 * pair + 1, c.N - 1);
-      const uint4 *r0 = reinterpret_cast<const uint4 *>(c.W + (size_t)n0 * c.ldw), *r1 = reinterpret_cast<const uint4 *>(c.W + (size_t)n1 * c.ldw);
-      int i = part * 32 + lane;
-      if (first) {
-#pragma unroll
-        for (int j = 0; j < kSgPre; ++j) {
-          if (i < pieces) {
-            const float4 a = *reinterpret_cast<const float4 *>(lo + 4 * i), b = *reinterpret_cast<const float4 *>(hi + 4 * i);
-            s0 = dot8(f.w[0][j], a, b, s0);
-            s1 = dot8(f.w[1][j], a, b, s1);
-          }
-          i += step;
-        }
-      }
-#pragma unroll 4
-      for (; i < pieces; i += step) {
-        const uint4 w0 = __ldg(r0 + i), w1 = __ldg(r1 + i);
-        const float4 a = *reinterpret_cast<const float4 *>(lo + 4 * i), b = *reinterpret_cast<const float4 *>(hi + 4 * i);
-        s0 = dot8(w0, a, b, s0);
-        s1 = dot8(w1, a, b, s1);
-      }
-    }
-    first = false;
-    s0 = warp_tree_sum(s0);
-    s1 = warp_tree_sum(s1);
-    if (c.wpr > 1) {
-      if (lane == 0) { part_sum[2 * warp] = s0; part_sum[2 * warp + 1] = s1; }
-      __syncthreads();
-      if (part == 0) {
-        s0 = s1 = 0.0f;
-        for (int i = 0; i < c.wpr; ++i) { s0 += part_sum[2 * (warp + i)]; s1 += part_sum[2 * (warp + i) + 1]; }
-      }
-      __syncthreads();
-    }
-    if (part == 0 && lane < 2 && pair < pairs) {
-      const int n = 2 * pair + lane;
-      if (n < c.N) c.Y[n] = apply_act((lane ? s1 : s0) + (c.Bias ? c.Bias[n] : 0.0f), c.act, c.cap);
-    }
+// After the block's last barrier: one thread per row.
+__device__ __forceinline__ void gemv_store(const GemvShape &c, const GemvDims &d, const float *part) {
+  const int n0 = blockIdx.x * c.rows_pb, n1 = min(c.N, n0 + c.rows_pb);
+  for (int n = n0 + threadIdx.x; n < n1; n += kSgThreads) {
+    float v = 0.0f;
+    for (int i = 0; i < d.wpr; ++i) v += part[(n - n0) * d.wpr + i];
+    c.Y[n] = apply_act(v + (c.Bias ? c.Bias[n] : 0.0f), c.act, c.cap);
   }
+}
+// shared memory: ring, vector halves, then `extra` floats, then the partial sums
+__host__ __device__ inline uint32_t gemv_smem(int ldw, int rows_pb, int extra) {
+  const GemvDims d = gemv_dims(ldw);
+  return (uint32_t)(d.nst * d.stage_bytes) + 4u * (uint32_t)(ldw + extra + rows_pb * d.wpr);
 }
 
 struct StreamGemvArgs {
@@ -161,26 +206,35 @@ struct StreamGemvArgs {
   const uint16_t *W;
   const float *Bias;     // [N] or null
   float *Y;              // [N]
-  int32_t N, K, ldw, wpr, act;
+  int32_t N, K, ldw, rows_pb, act;
   float cap;
 };
+extern __shared__ __align__(128) unsigned char sg_smem[];
 __global__ void __launch_bounds__(kSgThreads, 2) StreamGemv(const StreamGemvArgs a) {
-  extern __shared__ __align__(16) float sg_smem[];
-  __shared__ float part_sum[2 * kSgWarps];
+  __shared__ GemvShared sh;
   pdl_launch_dependents();
-  const GemvShape c{a.W, a.Bias, a.Y, a.N, a.ldw, a.wpr, a.act, a.cap};
-  GemvFirst f;
-  gemv_prefetch(c, f);
-  pdl_wait();
-  float *lo = sg_smem, *hi = sg_smem + sg_half((uint32_t)a.ldw);
-  for (int k = threadIdx.x; k < a.ldw; k += kSgThreads) sg_put(lo, hi, k, k < a.K ? a.X[k] : 0.0f);
+  const GemvDims d = gemv_dims(a.ldw);
+  const GemvShape c{a.W, a.Bias, a.Y, a.N, a.ldw, a.rows_pb, a.act, a.cap};
+  float *lo = reinterpret_cast<float *>(sg_smem + d.nst * d.stage_bytes), *hi = lo + a.ldw / 2, *part = hi + a.ldw / 2;
+  gemv_init(&sh, d.nst);
+  if (threadIdx.x >= kSgWarps * 32) {
+    gemv_produce(c, d, &sh, sg_smem);
+  } else {
+    pdl_wait();
+    for (int k = threadIdx.x; k < a.ldw; k += kSgWarps * 32) sg_put(lo, hi, k, k < a.K ? a.X[k] : 0.0f);
+    asm volatile("bar.sync 1, 512;" ::: "memory");
+    gemv_consume(c, d, &sh, sg_smem, lo, hi, part);
+  }
   __syncthreads();
-  gemv_body(c, lo, hi, part_sum, f);
+  gemv_store(c, d, part);
 }
-static uint32_t stream_gemv_smem(const void *args) { return 4u * (uint32_t)((const StreamGemvArgs *)args)->ldw; }
+static uint32_t stream_gemv_smem(const void *args) {
+  const StreamGemvArgs *a = (const StreamGemvArgs *)args;
+  return gemv_smem(a->ldw, a->rows_pb, 0);
+}
 #define F(f) AINFER_ARG(StreamGemvArgs, f)
-AINFER_REGISTER(StreamGemv, StreamGemvArgs, kSgThreads, 0, 0, stream_gemv_smem, F(X), F(W), F(Bias), F(Y), F(N), F(K), F(ldw), F(wpr), F(act),
-                F(cap));
+AINFER_REGISTER(StreamGemv, StreamGemvArgs, kSgThreads, 0, 0, stream_gemv_smem, F(X), F(W), F(Bias), F(Y), F(N), F(K), F(ldw), F(rows_pb),
+                F(act), F(cap));
 #undef F
 
 struct HyperStreamGemvArgs {
@@ -196,51 +250,60 @@ struct HyperStreamGemvArgs {
   const uint16_t *W;
   const float *Bias;
   float *Y;
-  int32_t S, N, K, ldw, wpr, act;
+  int32_t S, N, K, ldw, rows_pb, act;
   float eps, cap;
 };
 __global__ void __launch_bounds__(kSgThreads, 2) HyperStreamGemv(const HyperStreamGemvArgs a) {
-  extern __shared__ __align__(16) float hg_smem[];
-  __shared__ float part_sum[2 * kSgWarps];
+  __shared__ GemvShared sh;
   __shared__ StreamCoef coef;
   __shared__ float red[33];
   pdl_launch_dependents();
-  const GemvShape c{a.W, a.Bias, a.Y, a.N, a.ldw, a.wpr, a.act, a.cap};
-  GemvFirst f;
-  gemv_prefetch(c, f);
+  const GemvDims d = gemv_dims(a.ldw);
+  const GemvShape c{a.W, a.Bias, a.Y, a.N, a.ldw, a.rows_pb, a.act, a.cap};
+  const int K = a.K, tid = threadIdx.x, nth = kSgWarps * 32;
+  float *lo = reinterpret_cast<float *>(sg_smem + d.nst * d.stage_bytes), *hi = lo + a.ldw / 2, *us = hi + a.ldw / 2,
+        *part = us + ((K + 3) & ~3);
   load_stream_coef(coef, a.Mix, a.Out, a.In, a.S);
-  pdl_wait();
-  __syncthreads();
-  const int K = a.K, tid = threadIdx.x;
-  float *lo = hg_smem, *hi = lo + sg_half((uint32_t)a.ldw), *us = hi + sg_half((uint32_t)a.ldw);
-  const float ss = stream_row_any(a.Xin, a.Yp, blockIdx.x == 0 ? a.Xout : nullptr, coef, a.S, K, a.Yp != nullptr, us);
-  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)K + a.eps);
-  const int pos = a.Shift ? a.Ctrl[CTRL_POS] : 0;
-  const float *prev = a.Shift ? a.State + (size_t)((pos - 1) & 1) * K : nullptr;
-  float *next = a.Shift && blockIdx.x == 0 ? a.State + (size_t)(pos & 1) * K : nullptr;
-  // the block_sum's barriers made every thread's u visible
-  for (int k = tid; k < a.ldw; k += kSgThreads) {
-    float v = 0.0f;
-    if (k < K) {
-      v = us[k] * inv * a.NormW[k];
-      if (a.Shift) {
-        const float pv = pos > 0 ? prev[k] : 0.0f;
-        if (next) next[k] = v;
-        v = fmaf(pv - v, a.Shift[k], v);
+  gemv_init(&sh, d.nst);
+  if (tid >= nth) {
+    gemv_produce(c, d, &sh, sg_smem);
+  } else {
+    const int lane = tid & 31, warp = tid >> 5;
+    pdl_wait();
+    float ss = stream_row_any(a.Xin, a.Yp, blockIdx.x == 0 ? a.Xout : nullptr, coef, a.S, K, a.Yp != nullptr, us, tid, nth);
+    ss = warp_tree_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    asm volatile("bar.sync 1, 512;" ::: "memory");   // also: every thread's u is visible
+    ss = warp_tree_sum(lane < kSgWarps ? red[lane] : 0.0f);
+    const float inv = 1.0f / sqrtf(ss / (float)K + a.eps);
+    const int pos = a.Shift ? a.Ctrl[CTRL_POS] : 0;
+    const float *prev = a.Shift ? a.State + (size_t)((pos - 1) & 1) * K : nullptr;
+    float *next = a.Shift && blockIdx.x == 0 ? a.State + (size_t)(pos & 1) * K : nullptr;
+    for (int k = tid; k < a.ldw; k += nth) {
+      float v = 0.0f;
+      if (k < K) {
+        v = us[k] * inv * a.NormW[k];
+        if (a.Shift) {
+          const float pv = pos > 0 ? prev[k] : 0.0f;
+          if (next) next[k] = v;
+          v = fmaf(pv - v, a.Shift[k], v);
+        }
       }
+      sg_put(lo, hi, k, v);
     }
-    sg_put(lo, hi, k, v);
+    asm volatile("bar.sync 1, 512;" ::: "memory");
+    gemv_consume(c, d, &sh, sg_smem, lo, hi, part);
   }
   __syncthreads();
-  gemv_body(c, lo, hi, part_sum, f);
+  gemv_store(c, d, part);
 }
 static uint32_t hyper_gemv_smem(const void *args) {
   const HyperStreamGemvArgs *a = (const HyperStreamGemvArgs *)args;
-  return 4u * ((uint32_t)a->ldw + (uint32_t)((a->K + 3) & ~3));
+  return gemv_smem(a->ldw, a->rows_pb, (a->K + 3) & ~3);
 }
 #define F(f) AINFER_ARG(HyperStreamGemvArgs, f)
 AINFER_REGISTER(HyperStreamGemv, HyperStreamGemvArgs, kSgThreads, 0, 0, hyper_gemv_smem, F(Xin), F(Yp), F(Mix), F(Out), F(Xout), F(In),
-                F(NormW), F(Shift), F(State), F(Ctrl), F(W), F(Bias), F(Y), F(S), F(N), F(K), F(ldw), F(wpr), F(act), F(eps), F(cap));
+                F(NormW), F(Shift), F(State), F(Ctrl), F(W), F(Bias), F(Y), F(S), F(N), F(K), F(ldw), F(rows_pb), F(act), F(eps), F(cap));
 #undef F
 
 // Copies [N][K] bf16 rows to rows of ld values, zero padded.

@@ -4,10 +4,13 @@
 // activation rows as the N operand (`nt` of them, 16..256), accumulators in tensor memory, two buffers,
 // so that a tile's epilogue overlaps the next tile's products.
 //
-// One block per SM walks (tile, split) units. Roles: warp 0 lane 0 issues the copies, warp 1 lane 0 the
+// LinearTc: one block per SM walks tiles. Roles: warp 0 lane 0 issues the copies, warp 1 lane 0 the
 // products, warps 4..7 read the accumulators (a lane = one output feature, so a warp stores 32
-// consecutive features of a row at a time). With splits > 1 a unit covers a share of K: it leaves fp32
-// partials, and the last unit of a tile to finish adds them in split order and applies the epilogue.
+// consecutive features of a row at a time).
+//
+// LinearTcSplit2 / 4 / 8, for few tiles: a cluster of that many blocks shares one tile (nt <= 128), each
+// block a part of K. The blocks exchange their fp32 partials through distributed shared memory, every
+// block summing its share of the rows in block order.
 //
 // Every wait is bounded: one that runs out stores a code in the host-visible fault word, after which
 // the block's other waits return at once and the kernel ends (copies in flight awaited, tensor memory
@@ -23,9 +26,7 @@ struct LinearTcArgs {
   CUtensorMap Xm;        // [rows][K], box 64 x nt
   const float *Bias;     // [N] or null
   void *Y;               // [rows][ldy]
-  float *Part;           // [splits][tiles][nt][128] when splits > 1
-  uint32_t *Count;       // [tiles], zero between launches
-  int32_t rows, N, K, nt, ldy, act, out16, splits;
+  int32_t rows, N, K, nt, ldy, act, out16;
   float cap;
 };
 
@@ -66,7 +67,7 @@ __device__ __forceinline__ void lt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
 
 struct LtShared {
   unsigned long long full[8], empty[8], acc_full[2], acc_empty[2], drain;
-  uint32_t tmem, fail, last;
+  uint32_t tmem, fail;
 };
 __device__ __forceinline__ bool lt_wait(LtShared *s, unsigned long long *b, uint32_t parity) {
   if (mbar_try(b, parity)) return true;
@@ -94,7 +95,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
   const int nt = a.nt, nst = (int)lt_stages(nt);
   const uint32_t stage_bytes = lt_stage_bytes(nt);
   const int n_tiles = (a.N + 127) / 128, r_tiles = (a.rows + nt - 1) / nt, tiles = n_tiles * r_tiles;
-  const int units = tiles * a.splits, kb = (a.K + 63) / 64;
+  const int kb = (a.K + 63) / 64;
   uint32_t cols = 32;
   while (cols < 2u * (uint32_t)nt) cols <<= 1;
   if (tid == 0) {
@@ -119,11 +120,9 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
   if (warp == 0 && lane == 0) {
     // ---- copies ----
     uint32_t st = 0, ph = 1, issued = 0;
-    for (int u = blockIdx.x; u < units; u += gridDim.x) {
-      const int tile = u % tiles, sp = u / tiles;
-      const int n0 = (tile % n_tiles) * 128, r0 = (tile / n_tiles) * nt;
-      const int k_lo = kb * sp / a.splits, k_hi = kb * (sp + 1) / a.splits;
-      for (int k = k_lo; k < k_hi; ++k) {
+    for (int u = blockIdx.x; u < tiles; u += gridDim.x) {
+      const int n0 = (u % n_tiles) * 128, r0 = (u / n_tiles) * nt;
+      for (int k = 0; k < kb; ++k) {
         if (!lt_wait(&sh, &sh.empty[st], ph)) break;
         const uint32_t dst = base + st * stage_bytes, bar = smem_addr(&sh.full[st]);
         mbar_arrive_expect(&sh.full[st], stage_bytes);
@@ -145,20 +144,18 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
     // ---- products ----
     const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nt >> 3) << 17) | ((128u >> 4) << 24);
     uint32_t st = 0, ph = 0, buf = 0, aph = 1;
-    for (int u = blockIdx.x; u < units; u += gridDim.x) {
-      const int sp = u / tiles;
-      const int k_lo = kb * sp / a.splits, k_hi = kb * (sp + 1) / a.splits;
+    for (int u = blockIdx.x; u < tiles; u += gridDim.x) {
       if (!lt_wait(&sh, &sh.acc_empty[buf], aph)) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t d = tmem + buf * (uint32_t)nt;
       bool ok = true;
-      for (int k = k_lo; k < k_hi; ++k) {
+      for (int k = 0; k < kb; ++k) {
         ok = lt_wait(&sh, &sh.full[st], ph);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const uint64_t da = lt_desc(base + st * stage_bytes), db = lt_desc(base + st * stage_bytes + 128u * 128u);
 #pragma unroll
-        for (int q = 0; q < 4; ++q) lt_mma(d, da + (uint64_t)(2 * q), db + (uint64_t)(2 * q), idesc, k > k_lo || q > 0 ? 1u : 0u);
+        for (int q = 0; q < 4; ++q) lt_mma(d, da + (uint64_t)(2 * q), db + (uint64_t)(2 * q), idesc, k > 0 || q > 0 ? 1u : 0u);
         lt_commit(smem_addr(&sh.empty[st]));
         if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
       }
@@ -174,11 +171,9 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
     // ---- epilogue ----
     const int lw = (warp & 3) * 32 + lane;
     uint32_t buf = 0, ph = 0;
-    for (int u = blockIdx.x; u < units; u += gridDim.x) {
-      const int tile = u % tiles, sp = u / tiles;
-      const int n = (tile % n_tiles) * 128 + lw, r0 = (tile / n_tiles) * nt, nr = min(nt, a.rows - r0);
+    for (int u = blockIdx.x; u < tiles; u += gridDim.x) {
+      const int n = (u % n_tiles) * 128 + lw, r0 = (u / n_tiles) * nt, nr = min(nt, a.rows - r0);
       const float bias = a.Bias && n < a.N ? a.Bias[n] : 0.0f;
-      // after a failed wait the unit's values are garbage, but the four warps still meet at their barriers
       lt_wait(&sh, &sh.acc_full[buf], ph);
       __syncwarp();
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -190,45 +185,17 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
         if (a.out16) reinterpret_cast<uint16_t *>(a.Y)[o] = f32_to_bf16(v);
         else reinterpret_cast<float *>(a.Y)[o] = v;
       };
-      float *part = a.splits > 1 ? a.Part + ((size_t)sp * tiles + tile) * nt * 128 + lw : nullptr;
-      for (int c = 0; c < nt; c += 16) {
-        if (c >= nr) break;
+      for (int c = 0; c < nr; c += 16) {
         uint32_t v[16];
         lt_ld16(taddr + (uint32_t)c, v);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-        if (part) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            if (c + i < nr) __stcg(part + (size_t)(c + i) * 128, __uint_as_float(v[i]));
-        } else {
-#pragma unroll
-          for (int i = 0; i < 16; ++i)
-            if (c + i < nr) emit(c + i, __uint_as_float(v[i]));
-        }
+        for (int i = 0; i < 16; ++i)
+          if (c + i < nr) emit(c + i, __uint_as_float(v[i]));
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       mbar_arrive(&sh.acc_empty[buf]);
       if (++buf == 2) { buf = 0; ph ^= 1; }
-      if (part) {
-        __threadfence();
-        asm volatile("bar.sync 1, 128;" ::: "memory");
-        if (tid == 128) {
-          const uint32_t c = atomicAdd(a.Count + tile, 1u);
-          sh.last = c + 1 == (uint32_t)a.splits;
-          if (sh.last) a.Count[tile] = 0;
-        }
-        asm volatile("bar.sync 1, 128;" ::: "memory");
-        if (sh.last) {
-          __threadfence();
-          const float *p0 = a.Part + (size_t)tile * nt * 128 + lw;
-          const size_t stride = (size_t)tiles * nt * 128;
-          for (int r = 0; r < nr; ++r) {
-            float v = 0.0f;
-            for (int s = 0; s < a.splits; ++s) v += __ldcg(p0 + (size_t)s * stride + (size_t)r * 128);
-            emit(r, v);
-          }
-        }
-      }
     }
   }
   __syncwarp();
@@ -240,11 +207,150 @@ static uint32_t linear_tc_smem(const void *args) {
   const int nt = ((const LinearTcArgs *)args)->nt;
   return lt_stages(nt) * lt_stage_bytes(nt) + 1024;
 }
+
+// ---- K split over a cluster ----
+__host__ __device__ inline uint32_t lts_stages(int nt) {
+  const uint32_t s = ((uint32_t)kLtBudget - (uint32_t)nt * 512u) / lt_stage_bytes(nt);
+  return s > 8 ? 8 : s;
+}
+__device__ __forceinline__ void cluster_sync_all() {
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+template <int CL>
+__device__ __forceinline__ void linear_tc_split(const LinearTcArgs &a) {
+  extern __shared__ __align__(1024) unsigned char lt_smem_raw[];
+  __shared__ LtShared sh;
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t base = (smem_addr(lt_smem_raw) + 1023u) & ~1023u;
+  const int nt = a.nt, nst = (int)lts_stages(nt), rpo = nt / CL;   // rows of the tile that a block sums
+  const uint32_t stage_bytes = lt_stage_bytes(nt), red = base + (uint32_t)nst * stage_bytes;
+  float *red_p = reinterpret_cast<float *>(lt_smem_raw + (red - smem_addr(lt_smem_raw)));   // [CL][rpo][128]
+  const int n_tiles = (a.N + 127) / 128, tile = blockIdx.x / CL, kb = (a.K + 63) / 64;
+  uint32_t rank;
+  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
+  const int n0 = (tile % n_tiles) * 128, r0 = (tile / n_tiles) * nt, nr = min(nt, a.rows - r0);
+  const int k_lo = kb * (int)rank / CL, k_hi = kb * ((int)rank + 1) / CL;
+  uint32_t cols = 32;
+  while (cols < (uint32_t)nt) cols <<= 1;
+  if (tid == 0) {
+    for (int i = 0; i < nst; ++i) { mbar_init(&sh.full[i], 1); mbar_init(&sh.empty[i], 1); }
+    mbar_init(&sh.acc_full[0], 1);
+    mbar_init(&sh.drain, 1);
+    sh.fail = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&a.Wm)) : "memory");
+    asm volatile("prefetch.tensormap [%0];" ::"l"(reinterpret_cast<uint64_t>(&a.Xm)) : "memory");
+  }
+  if (warp == 2) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_addr(&sh.tmem)), "r"(cols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+  const uint32_t tmem = sh.tmem;
+  cluster_sync_all();   // every block of the cluster runs: its shared memory may be written
+  pdl_wait();
+
+  if (warp == 0 && lane == 0) {
+    uint32_t st = 0, ph = 1, issued = 0;
+    for (int k = k_lo; k < k_hi; ++k) {
+      if (!lt_wait(&sh, &sh.empty[st], ph)) break;
+      const uint32_t dst = base + st * stage_bytes, bar = smem_addr(&sh.full[st]);
+      mbar_arrive_expect(&sh.full[st], stage_bytes);
+      lt_tma(dst, &a.Wm, bar, k * 64, n0);
+      lt_tma(dst + 128u * 128u, &a.Xm, bar, k * 64, r0);
+      ++issued;
+      if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
+    }
+    if (*reinterpret_cast<volatile uint32_t *>(&sh.fail)) {
+      for (int i = 0; i < nst && (uint32_t)i < issued; ++i) {
+        const uint32_t uses = (issued - (uint32_t)i + (uint32_t)nst - 1) / (uint32_t)nst;
+        for (uint32_t s = 0; s < kLtSpin && !mbar_try(&sh.full[i], (uses - 1) & 1); ++s) {}
+      }
+    }
+  } else if (warp == 1 && lane == 0) {
+    const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nt >> 3) << 17) | ((128u >> 4) << 24);
+    uint32_t st = 0, ph = 0;
+    bool ok = true;
+    for (int k = k_lo; k < k_hi; ++k) {
+      ok = lt_wait(&sh, &sh.full[st], ph);
+      if (!ok) break;
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const uint64_t da = lt_desc(base + st * stage_bytes), db = lt_desc(base + st * stage_bytes + 128u * 128u);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) lt_mma(tmem, da + (uint64_t)(2 * q), db + (uint64_t)(2 * q), idesc, k > k_lo || q > 0 ? 1u : 0u);
+      lt_commit(smem_addr(&sh.empty[st]));
+      if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
+    }
+    lt_commit(smem_addr(ok ? &sh.acc_full[0] : &sh.drain));
+    if (!ok)
+      for (uint32_t s = 0; s < kLtSpin && !mbar_try(&sh.drain, 0); ++s) {}
+  } else if (warp >= 4) {
+    const int lw = (warp & 3) * 32 + lane;
+    lt_wait(&sh, &sh.acc_full[0], 0);
+    __syncwarp();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t taddr = tmem + ((uint32_t)((warp & 3) * 32) << 16);
+    const uint32_t mine = red + ((uint32_t)rank * (uint32_t)rpo * 128u + (uint32_t)lw) * 4u;
+    for (int c = 0; c < nr; c += 16) {
+      uint32_t v[16];
+      lt_ld16(taddr + (uint32_t)c, v);
+      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const int col = c + i;
+        if (col < nr) {
+          uint32_t peer;
+          asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(peer) : "r"(mine + (uint32_t)(col % rpo) * 512u), "r"(col / rpo));
+          asm volatile("st.shared::cluster.u32 [%0], %1;" ::"r"(peer), "r"(v[i]) : "memory");
+        }
+      }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  }
+  __syncwarp();
+  cluster_sync_all();
+  const int n = n0 + (tid & 127);
+  if (n < a.N) {
+    const float bias = a.Bias ? a.Bias[n] : 0.0f;
+    for (int r = tid >> 7; r < rpo; r += 2) {
+      const int row = (int)rank * rpo + r;
+      if (row >= nr) break;
+      float v = 0.0f;
+#pragma unroll
+      for (int s = 0; s < CL; ++s) v += red_p[(s * rpo + r) * 128 + (tid & 127)];
+      v = lt_act(v + bias, a.act, a.cap);
+      const size_t o = (size_t)(r0 + row) * a.ldy + n;
+      if (a.out16) reinterpret_cast<uint16_t *>(a.Y)[o] = f32_to_bf16(v);
+      else reinterpret_cast<float *>(a.Y)[o] = v;
+    }
+  }
+  asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+  __syncthreads();
+  if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
+}
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit2(const __grid_constant__ LinearTcArgs a) { linear_tc_split<2>(a); }
+__global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit4(const __grid_constant__ LinearTcArgs a) { linear_tc_split<4>(a); }
+__global__ void __cluster_dims__(8, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit8(const __grid_constant__ LinearTcArgs a) { linear_tc_split<8>(a); }
+static uint32_t linear_tc_split_smem(const void *args) {
+  const int nt = ((const LinearTcArgs *)args)->nt;
+  return lts_stages(nt) * lt_stage_bytes(nt) + (uint32_t)nt * 512u + 1024;
+}
+
 #define F(f) AINFER_ARG(LinearTcArgs, f)
-AINFER_REGISTER(LinearTc, LinearTcArgs, kLtThreads, 0, 0, linear_tc_smem, F(Wm), F(Xm), F(Bias), F(Y), F(Part), F(Count), F(rows), F(N), F(K),
-                F(nt), F(ldy), F(act), F(out16), F(splits), F(cap));
+#define LT_FIELDS F(Wm), F(Xm), F(Bias), F(Y), F(rows), F(N), F(K), F(nt), F(ldy), F(act), F(out16), F(cap)
+AINFER_REGISTER(LinearTc, LinearTcArgs, kLtThreads, 0, 0, linear_tc_smem, LT_FIELDS);
+AINFER_REGISTER(LinearTcSplit2, LinearTcArgs, kLtThreads, 2, 0, linear_tc_split_smem, LT_FIELDS);
+AINFER_REGISTER(LinearTcSplit4, LinearTcArgs, kLtThreads, 4, 0, linear_tc_split_smem, LT_FIELDS);
+AINFER_REGISTER(LinearTcSplit8, LinearTcArgs, kLtThreads, 8, 0, linear_tc_split_smem, LT_FIELDS);
 #undef F
 
 AINFER_EARLY_LAUNCH(LinearTc);
+AINFER_EARLY_LAUNCH(LinearTcSplit2);
+AINFER_EARLY_LAUNCH(LinearTcSplit4);
+AINFER_EARLY_LAUNCH(LinearTcSplit8);
 
 }  // namespace ainfer

@@ -6,7 +6,7 @@
 // This file holds what is particular to it: configuration, tensor list, prepared weights, and the
 // sequence of launches of a row pass and of a decode step (RowEngine). The mechanisms are kernels of
 // their own with their constants as arguments: k_hyper.cu, k_chunk_attn.cu, k_linear.cu,
-// k_linear_tc.cu.
+// k_linear_tc.cu, k_chunk_mma.cu.
 #include <algorithm>
 #include <cmath>
 #include <cstring>
@@ -91,7 +91,7 @@ bool check(const ModelConfig &c, std::string &err) {
     if (r.taps < 1 || r.taps > 64) return bad("conv must be in [1, 64] taps");
     if (r.chunk < 0) return bad("mask.size");
     if (!std::isfinite(r.scale)) return bad("mixer.scale");
-    if (r.ff > 49152 || r.heads * r.dim > 49152) return bad("a layer's inner size exceeds 49152");
+    if (r.ff > 24576 || r.heads * r.dim > 24576) return bad("a layer's inner size exceeds 24576");
     // shared memory of the decode step's attention: queries, sums, a tile of keys, scores
     const long hg = r.heads / r.kv_heads;
     if (4 * (2 * hg * r.dim + r.dim + 64L * (r.dim + 1) + 64 * hg + 3 * hg) > 220 * 1024) return bad("too many query heads per key head at this dim");
@@ -339,9 +339,9 @@ struct Engine : RowEngine {
   char *state = nullptr;
   size_t state_bytes = 0, k_off = 0, conv_off = 0;
   // pass buffers
-  float *X[2] = {nullptr, nullptr}, *U = nullptr, *Y = nullptr, *Part = nullptr, *AttPart = nullptr;
+  float *X[2] = {nullptr, nullptr}, *U = nullptr, *Y = nullptr, *AttPart = nullptr;
   char *H = nullptr, *Q = nullptr, *Att = nullptr, *Act = nullptr;
-  uint32_t *Count = nullptr, *AttCount = nullptr;
+  uint32_t *AttCount = nullptr;
   void *tail_rows = nullptr, *tail_steps = nullptr;
   int ldw = 0, ldq = 0, ldf = 0, maxC = 0, att_splits = 1;
   // recording of a decode step
@@ -411,14 +411,11 @@ struct Engine : RowEngine {
       ts.push_back({s.pend_shift, s.shift, nullptr, nullptr, C, 1});   // steps keep their convolution ring themselves
     }
     ldw = round_up((int)W, 8); ldq = round_up(maxQ, 8); ldf = round_up(maxF, 8);
-    att_splits = std::max(1, std::min(64, (2 * sm_count) / std::max(1, std::min(nseq, 2 * sm_count) * maxG)));
+    // blocks of a step's attention: about four per SM over sequences, key heads and splits
+    att_splits = std::max(1, std::min(64, 4 * sm_count / (std::min(nseq, 4 * sm_count) * maxG)));
     for (int i = 0; i < 2; ++i) e |= alloc(R * S * W, &X[i]);
     e |= alloc(R * ldw * esz(), &H); e |= alloc(R * maxC, &U); e |= alloc(R * ldq * esz(), &Q);
     e |= alloc(R * ldq * 4, &Att); e |= alloc(R * W, &Y); e |= alloc(R * ldf * 4, &Act);
-    if (!f32) {
-      e |= alloc((size_t)sm_count * 256 * 128, &Part);
-      e |= alloc((size_t)sm_count, &Count);
-    }
     e |= alloc((size_t)nseq * att_splits * maxHGD, &AttPart);
     e |= alloc((size_t)nseq * maxG, &AttCount);
     TailRecord *d = nullptr;
@@ -458,16 +455,18 @@ struct Engine : RowEngine {
     int nt = rows <= 16 ? 16 : rows <= 32 ? 32 : rows <= 64 ? 64 : rows <= 128 ? 128 : 256;
     if (nt == 256 && n_tiles * ((rows + 255) / 256) < sm_count) nt = 128;
     const int tiles = n_tiles * ((rows + nt - 1) / nt);
-    int splits = 1;
-    if (tiles * 2 <= sm_count) splits = std::max(1, std::min(sm_count / tiles, kb / 4));
+    int splits = 1;   // few tiles: a cluster of blocks per tile, each a part of K
+    while (nt <= 128 && splits < 8 && tiles * splits * 2 <= sm_count && kb >= splits * 4) splits *= 2;
     TensorMap wm, xm;
     if (ainfer_tensor_map_bf16(dev, &wm, mt.w, (uint64_t)mt.N, (uint64_t)mt.K, (uint64_t)mt.ldw, 128) != AINFER_OK ||
         ainfer_tensor_map_bf16(dev, &xm, Xp, (uint64_t)rows, (uint64_t)mt.K, (uint64_t)ldx, (uint32_t)nt) != AINFER_OK) {
       k.fail(1, ainfer_last_error(dev));
       return;
     }
-    k.launch("LinearTc", (uint32_t)std::min(tiles * splits, sm_count), wm, xm, mt.bias, Yp, Part, Count, (int32_t)rows, (int32_t)mt.N,
-             (int32_t)mt.K, (int32_t)nt, (int32_t)ldy, (int32_t)act, (int32_t)(out16 ? 1 : 0), (int32_t)splits, cap);
+    static const char *const names[] = {"LinearTc", "LinearTcSplit2", "LinearTcSplit4", "LinearTcSplit8"};
+    const int which = splits == 8 ? 3 : splits == 4 ? 2 : splits == 2 ? 1 : 0;
+    k.launch(names[which], (uint32_t)(splits > 1 ? tiles * splits : std::min(tiles, sm_count)), wm, xm, mt.bias, Yp, (int32_t)rows, (int32_t)mt.N,
+             (int32_t)mt.K, (int32_t)nt, (int32_t)ldy, (int32_t)act, (int32_t)(out16 ? 1 : 0), cap);
   }
 
   // stream update of the pending sublayer (if any), then the read + norm (+ shift) of the next
@@ -503,12 +502,18 @@ struct Engine : RowEngine {
       linear(k, lw.qk, H, ldw, R, U, C, ACT_NONE, false);
       if (sp.one_sequence) {
         const int per = std::max(1, std::min(16, R / 16));
-        k.launch(f32 ? "ShortConvRowsF32" : "ShortConvRowsB16", (uint32_t)(((R + per - 1) / per) * ((C + 255) / 256)), (const float *)U, lw.conv,
+        const int cblk = C % 4 == 0 && Qc % 4 == 0 && r.taps >= 2 && r.taps <= 4 ? 1024 : 256;   // channels of a block
+        k.launch(f32 ? "ShortConvRowsF32" : "ShortConvRowsB16", (uint32_t)(((R + per - 1) / per) * ((C + cblk - 1) / cblk)), (const float *)U, lw.conv,
                  (const float *)s.conv, s.pend_conv, sp.ctrl, sp.seq, sp.first, (void *)Q, (void *)s.k, kv_stride, (int32_t)R, (int32_t)C,
                  (int32_t)Qc, (int32_t)r.taps, (int32_t)s.cap, (int32_t)C, (int32_t)per);
-        k.launch(f32 ? "ChunkAttnRowsF32" : "ChunkAttnRowsB16", (uint32_t)(((R + 15) / 16) * r.heads), (const void *)Q, (const void *)s.k, lw.lb,
-                 lw.temp, sp.ctrl, (void *)Att, (int32_t)R, (int32_t)r.heads, (int32_t)r.kv_heads, (int32_t)r.dim, (int32_t)s.cap,
-                 (int32_t)s.chunk, (int32_t)lw.lb_len, (int32_t)ldo, (float)r.scale);
+        if (mma_dim(r))
+          k.launch(sized("ChunkAttnMma", r.dim).c_str(), (uint32_t)(((R + 63) / 64) * r.heads), (const uint16_t *)Q, (const uint16_t *)s.k, lw.lb,
+                   lw.temp, sp.ctrl, (uint16_t *)Att, (int32_t)R, (int32_t)r.heads, (int32_t)r.kv_heads, (int32_t)r.dim, (int32_t)s.cap,
+                   (int32_t)s.chunk, (int32_t)lw.lb_len, (int32_t)ldo, (float)r.scale);
+        else
+          k.launch(f32 ? "ChunkAttnRowsF32" : "ChunkAttnRowsB16", (uint32_t)(((R + 15) / 16) * r.heads), (const void *)Q, (const void *)s.k, lw.lb,
+                   lw.temp, sp.ctrl, (void *)Att, (int32_t)R, (int32_t)r.heads, (int32_t)r.kv_heads, (int32_t)r.dim, (int32_t)s.cap,
+                   (int32_t)s.chunk, (int32_t)lw.lb_len, (int32_t)ldo, (float)r.scale);
       } else {
         attn_step(k, r, lw, s, sp.ctrl, R, C, ldo, b16);
       }
@@ -530,38 +535,37 @@ struct Engine : RowEngine {
              (int32_t)c.layers, (int32_t)R, (int32_t)W);
   }
 
+  // head sizes the tensor-core attention takes (bf16), and the name of the instance that holds one
+  bool mma_dim(const RowLayerConfig &r) const { return !f32 && r.dim % 8 == 0 && r.dim <= 256; }
+  static std::string sized(const char *base, int dim) {
+    for (int d : {32, 64, 96, 128, 192})
+      if (dim <= d) return base + std::to_string(d);
+    return base + std::string("256");
+  }
   void attn_step(KernelCalls &k, const RowLayerConfig &r, const RowLayerWeights &lw, const LayerState &s, const int32_t *ctrl, int n, int C, int ldo,
                  bool out16) {
-    k.launch(f32 ? "ChunkAttnStepF32" : "ChunkAttnStepB16", (uint32_t)(n * r.kv_heads * att_splits), (const float *)U, lw.conv, s.conv, ctrl,
+    const std::string name = mma_dim(r) && r.heads / r.kv_heads <= 16 ? sized("ChunkAttnStepMma", r.dim)
+                                                                      : std::string(f32 ? "ChunkAttnStepF32" : "ChunkAttnStepB16");
+    k.launch(name.c_str(), (uint32_t)(n * r.kv_heads * att_splits), (const float *)U, lw.conv, s.conv, ctrl,
              (void *)s.k, (int64_t)s.cap * r.kv_heads * r.dim, lw.lb, lw.temp, AttPart, AttCount, (void *)Att, (int32_t)n, (int32_t)r.heads,
              (int32_t)r.kv_heads, (int32_t)r.dim, (int32_t)r.taps, (int32_t)s.cap, (int32_t)s.chunk, (int32_t)lw.lb_len, (int32_t)att_splits,
              (int32_t)C, (int32_t)ldo, (int32_t)(out16 ? 1 : 0), (float)r.scale);
   }
 
   // ---- one decode step of sequence 0 ----
-  // warps that share two rows, and blocks, of a weight-streaming launch (16 warps a block)
-  void gemv_shape(const RowMatrix &mt, int32_t *wpr, uint32_t *groups) const {
-    const int pairs = (mt.N + 1) / 2, pieces = mt.ldw / 8;
-    *wpr = 1;
-    while (*wpr < 8 && pairs * *wpr * 2 <= sm_count * 16 && pieces >= 64 * *wpr) *wpr *= 2;
-    *groups = (uint32_t)std::min((pairs + 16 / *wpr - 1) / (16 / *wpr), sm_count);
-  }
   void gemv(KernelCalls &k, const RowMatrix &mt, const float *x, float *y, int act) {
-    int32_t wpr;
-    uint32_t groups;
-    gemv_shape(mt, &wpr, &groups);
-    k.launch("StreamGemv", groups, x, mt.w, mt.bias, y, (int32_t)mt.N, (int32_t)mt.K, (int32_t)mt.ldw, wpr, (int32_t)act, 0.0f);
+    const int rows_pb = (mt.N + sm_count - 1) / sm_count;
+    k.launch("StreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), x, mt.w, mt.bias, y, (int32_t)mt.N, (int32_t)mt.K, (int32_t)mt.ldw,
+             (int32_t)rows_pb, (int32_t)act, 0.0f);
   }
   void hyper_gemv(KernelCalls &k, const RowMatrix &mt, const float *in, const float *norm, const float *shift, float *shift_state,
                   const int32_t *ctrl, float *y, int act, float cap) {
     const ModelConfig &c = m->cfg;
-    int32_t wpr;
-    uint32_t groups;
-    gemv_shape(mt, &wpr, &groups);
-    k.launch("HyperStreamGemv", groups, (const float *)X[cur], (const float *)(pending ? Y : nullptr),
+    const int rows_pb = (mt.N + sm_count - 1) / sm_count;
+    k.launch("HyperStreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), (const float *)X[cur], (const float *)(pending ? Y : nullptr),
              (const float *)(pending ? pending->mix : nullptr), (const float *)(pending ? pending->out : nullptr),
              (float *)(pending ? X[cur ^ 1] : nullptr), in, norm, shift, shift_state, ctrl, mt.w, mt.bias, y, (int32_t)c.streams, (int32_t)mt.N,
-             (int32_t)mt.K, (int32_t)mt.ldw, wpr, (int32_t)act, (float)c.rms_eps, cap);
+             (int32_t)mt.K, (int32_t)mt.ldw, (int32_t)rows_pb, (int32_t)act, (float)c.rms_eps, cap);
     if (pending) { cur ^= 1; pending = nullptr; }
   }
   void record_embed(KernelCalls &k, const int32_t *ctrl) override {

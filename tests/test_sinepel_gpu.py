@@ -114,7 +114,7 @@ def test_stream_update_read_norm_and_shift(dev, W, S, per, out):
 
 
 @pytest.mark.parametrize("kind", ["f32", "b16"])
-@pytest.mark.parametrize("taps,Qc,Kn,per", [(4, 24, 8, 1), (1, 300, 20, 3), (2, 16, 16, 2), (7, 20, 12, 5)])
+@pytest.mark.parametrize("taps,Qc,Kn,per", [(4, 24, 8, 1), (1, 300, 20, 3), (2, 16, 16, 2), (7, 20, 12, 5), (3, 1000, 40, 4), (4, 30, 5, 4)])
 def test_short_convolution_over_rows(dev, taps, Qc, Kn, per, kind):
     """Two sequences in a pass, one from position 0 and one continuing; the pending rows are committed."""
     C, cap = Qc + Kn, 16
@@ -132,7 +132,7 @@ def test_short_convolution_over_rows(dev, taps, Qc, Kn, per, kind):
     q, kc = dev.zeros(17 * Qc * 4), dev.zeros(2 * cap * Kn * 4)
     ctl = [dev.upload(ctrl(pos)), dev.upload(np.int32(seq)), dev.upload(np.int32(first))]
     dev.kernel("ShortConvRowsF32" if kind == "f32" else "ShortConvRowsB16")(
-        -(-17 // per) * (-(-C // 256)), dev.upload(f32(U)), dev.upload(f32(cw.T)), dst, pend, *ctl, q, kc, cap * Kn, 17, C, Qc, taps, cap, C, per)
+        -(-17 // per) * (-(-C // (1024 if C % 4 == 0 and Qc % 4 == 0 and 2 <= taps <= 4 else 256))), dev.upload(f32(U)), dev.upload(f32(cw.T)), dst, pend, *ctl, q, kc, cap * Kn, 17, C, Qc, taps, cap, C, per)
     dev.sync()
     dt, tol = (np.float32, 1e-5) if kind == "f32" else (np.uint16, 1e-2)
     val = lambda a: a if kind == "f32" else from_bits(a, a.shape)   # noqa: E731
@@ -184,13 +184,20 @@ def test_distance_table(dev):
 
 
 ATTN = [(70, 4, 2, 16, 24, 128), (33, 3, 3, 20, 1, 64), (90, 8, 2, 64, 50, 128), (40, 5, 1, 33, 1000, 64), (150, 4, 4, 128, 64, 256),
-        (140, 8, 1, 64, 37, 192), (200, 6, 2, 96, 130, 256)]
+        (140, 8, 1, 64, 37, 192), (200, 6, 2, 96, 130, 256), (300, 4, 2, 40, 64, 384), (260, 2, 1, 256, 200, 320), (129, 3, 1, 176, 128, 192),
+        (130, 2, 2, 8, 65, 192)]
 
 
-@pytest.mark.parametrize("kind", ["f32", "b16"])
+def _mma(base, D):
+    return base + str(next(p for p in (32, 64, 96, 128, 192, 256) if D <= p))
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16", "mma"])
 @pytest.mark.parametrize("T,H,G,D,chunk,cap", ATTN)
 def test_chunk_attention_over_rows(dev, T, H, G, D, chunk, cap, kind):
     """Whole and from the middle (the first rows already in the cache)."""
+    if kind == "mma" and D % 8:
+        pytest.skip("head size for the CUDA-core form")
     edge = [(chunk - 1, 0), (chunk, chunk - 1), (2 * chunk, 2 * chunk - 1), (2 * chunk - 1, chunk)] if 2 * chunk < T else None
     q, k, r1, r2, temp = _attn_case(T, H, G, D, chunk, T, edge)
     want = P.shared_kv_attention(q.double(), k.double(), 0.25, temp.double(), r1.double(), r2.double(), chunk).reshape(T, H * D)
@@ -205,8 +212,9 @@ def test_chunk_attention_over_rows(dev, T, H, G, D, chunk, cap, kind):
     for start in (0, T // 3):
         R = T - start
         o = dev.zeros(R * ldo * 4)
-        dev.kernel("ChunkAttnRowsF32" if kind == "f32" else "ChunkAttnRowsB16")(
-            -(-R // 16) * H, dev.upload(conv(q[start:].reshape(R, H * D))), dk, lb, dev.upload(f32(temp)), dev.upload(ctrl(range(start, T))), o, R, H,
+        name, rows = {"f32": ("ChunkAttnRowsF32", 16), "b16": ("ChunkAttnRowsB16", 16), "mma": (_mma("ChunkAttnMma", D), 64)}[kind]
+        dev.kernel(name)(
+            -(-R // rows) * H, dev.upload(conv(q[start:].reshape(R, H * D))), dk, lb, dev.upload(f32(temp)), dev.upload(ctrl(range(start, T))), o, R, H,
             G, D, cap, chunk, n, ldo, 0.25)
         dev.sync()
         raw = dev.download(o, (R, ldo), np.float32 if kind == "f32" else np.uint16)[:, :H * D]
@@ -214,12 +222,14 @@ def test_chunk_attention_over_rows(dev, T, H, G, D, chunk, cap, kind):
         close(got, want[start:], 1e-5 if kind == "f32" else 3e-2)
 
 
-@pytest.mark.parametrize("kind", ["f32", "b16"])
-@pytest.mark.parametrize("H,G,D,chunk,taps,splits", [(4, 2, 16, 24, 3, 1), (6, 2, 20, 100, 1, 5), (8, 1, 64, 150, 4, 2), (3, 3, 33, 1, 2, 3),
+@pytest.mark.parametrize("kind", ["f32", "b16", "mma"])
+@pytest.mark.parametrize("H,G,D,chunk,taps,splits", [(16, 1, 96, 190, 3, 4), (4, 2, 192, 130, 4, 3), (4, 2, 256, 64, 2, 2), (4, 2, 16, 24, 3, 1), (6, 2, 20, 100, 1, 5), (8, 1, 64, 150, 4, 2), (3, 3, 33, 1, 2, 3),
                                                      (4, 4, 128, 90, 4, 8), (12, 2, 40, 200, 5, 16)])
 def test_decode_attention_with_convolution(dev, H, G, D, chunk, taps, splits, kind):
     """Three sequences decode side by side from position 0, at different times, over several chunks; their
     key rings are shorter than the run."""
+    if kind == "mma" and D % 8:
+        pytest.skip("head size for the CUDA-core form")
     T, Q, K, C = 230, H * D, G * D, (H + G) * D
     cap, n = 256 if chunk > 100 else 128, min(chunk, 512)
     g = torch.Generator().manual_seed(D)
@@ -230,7 +240,9 @@ def test_decode_attention_with_convolution(dev, H, G, D, chunk, taps, splits, ki
     want = []
     for s in range(3):
         y = P.short_conv(u[s].double(), cw.double())
-        if kind == "b16":
+        if kind == "mma":       # this form's products take bf16 queries
+            y[:, :Q] = bf16(y[:, :Q]).double()
+        if kind != "f32":
             y[:, Q:] = bf16(y[:, Q:]).double()
         want.append(P.shared_kv_attention(y[:, :Q].reshape(T, H, D), y[:, Q:].reshape(T, G, D), 0.3, temp.double(), r1.double(), r2.double(),
                                           chunk).reshape(T, Q))
@@ -242,7 +254,7 @@ def test_decode_attention_with_convolution(dev, H, G, D, chunk, taps, splits, ki
     kc = dev.upload(f32(torch.randn(3, cap, K, generator=g)) if kind == "f32" else bits(torch.randn(3, cap, K, generator=g)))
     part, cnt = dev.zeros(3 * splits * H * (D + 2) * 4), dev.zeros(3 * G * 4)
     o, du, dc = dev.zeros(3 * Q * 4), dev.zeros(3 * C * 4), dev.zeros(48)
-    k = dev.kernel("ChunkAttnStepF32" if kind == "f32" else "ChunkAttnStepB16")
+    k = dev.kernel({"f32": "ChunkAttnStepF32", "b16": "ChunkAttnStepB16", "mma": _mma("ChunkAttnStepMma", D)}[kind])
     got = np.zeros((3, T, Q), np.float32)
     for t in range(T + 60):
         pos = [min(max(t - lag[s], 0), T - 1) for s in range(3)]
@@ -274,32 +286,34 @@ def test_linear_rows_32bit(dev, R, N, K, act):
 
 @pytest.mark.parametrize("R,N,K,nt,splits,act,out16", [
     (1, 5, 40, 16, 1, 0, 0), (17, 130, 200, 32, 1, 2, 0), (64, 256, 1024, 64, 4, 0, 0), (300, 384, 136, 128, 1, 1, 1), (520, 640, 512, 256, 1, 0, 0),
-    (30, 100, 4096, 16, 7, 1, 1), (1000, 1536, 320, 256, 1, 1, 1), (129, 128, 64, 128, 1, 0, 0)])
+    (30, 100, 4096, 16, 8, 1, 1), (1000, 1536, 320, 256, 1, 1, 1), (129, 128, 64, 128, 1, 0, 0), (5, 300, 520, 16, 2, 0, 0), (100, 260, 2048, 128, 8, 2, 0),
+    (33, 128, 72, 64, 2, 0, 1)])
 def test_linear_tensor_cores(dev, R, N, K, nt, splits, act, out16):
     g = torch.Generator().manual_seed(R)
     x, w, b = bf16(torch.randn(R, K, generator=g)), bf16(torch.randn(N, K, generator=g)), torch.randn(N, generator=g)
     dx, dw = dev.upload(bits(x)), dev.upload(bits(w))
     tiles = -(-N // 128) * (-(-R // nt))
-    y, part, cnt = dev.zeros(R * N * 4), dev.zeros(splits * tiles * nt * 128 * 4), dev.zeros(tiles * 4)
-    k = dev.kernel("LinearTc")
+    y = dev.zeros(R * N * 4)
+    k = dev.kernel("LinearTc" + (f"Split{splits}" if splits > 1 else ""))
     want = ACTS[act](x.double() @ w.double().T + b.double(), 3.0)
-    for _ in range(2):     # the second launch finds the counters as the first left them
-        k(min(tiles * splits, dev.info().sm_count), dev.tensor_map_bf16(dw, N, K, K, 128), dev.tensor_map_bf16(dx, R, K, K, nt), dev.upload(f32(b)), y,
-          part, cnt, R, N, K, nt, N, act, out16, splits, 3.0)
+    for _ in range(2):
+        k(tiles * splits if splits > 1 else min(tiles, 3), dev.tensor_map_bf16(dw, N, K, K, 128), dev.tensor_map_bf16(dx, R, K, K, nt), dev.upload(f32(b)), y,
+          R, N, K, nt, N, act, out16, 3.0)
         dev.sync()
         raw = dev.download(y, (R, N), np.uint16 if out16 else np.float32)
         close(from_bits(raw, (R, N)) if out16 else raw, want, 2e-2 if out16 else 1e-5)
 
 
-@pytest.mark.parametrize("N,K,wpr,act", [(7, 50, 1, 0), (64, 1000, 4, 1), (601, 256, 2, 2), (33, 4096, 8, 0)])
-def test_decode_gemv(dev, N, K, wpr, act):
+@pytest.mark.parametrize("N,K,rows_pb,act", [(7, 50, 3, 0), (64, 1000, 22, 1), (601, 256, 201, 2), (33, 4096, 11, 0), (9, 20000, 5, 0), (500, 2560, 250, 0),
+                                             (3, 8, 1, 0)])
+def test_decode_gemv(dev, N, K, rows_pb, act):
     g = torch.Generator().manual_seed(N)
     x, w, b = torch.randn(K, generator=g), bf16(torch.randn(N, K, generator=g)), torch.randn(N, generator=g)
     ldw = -(-K // 8) * 8
     wp = torch.zeros(N, ldw)
     wp[:, :K] = w.float()
     y = dev.zeros(N * 4)
-    dev.kernel("StreamGemv")(3, dev.upload(f32(x)), dev.upload(bits(wp)), dev.upload(f32(b)), y, N, K, ldw, wpr, act, 3.0)
+    dev.kernel("StreamGemv")(-(-N // rows_pb), dev.upload(f32(x)), dev.upload(bits(wp)), dev.upload(f32(b)), y, N, K, ldw, rows_pb, act, 3.0)
     close(dev.download(y, N, np.float32), ACTS[act](w.double() @ x.double() + b.double(), 3.0), 1e-5)
 
 
@@ -318,8 +332,8 @@ def test_decode_gemv_from_streams(dev, S, K, N, pos, shift):
     hs = h + ((d(st)[(pos - 1) & 1] if pos else 0 * h) - h) * d(sh) if shift else h
     up = lambda t: dev.upload(f32(t))   # noqa: E731
     xo, out, dst = dev.zeros(S * K * 4), dev.zeros(N * 4), up(st)
-    dev.kernel("HyperStreamGemv")(4, up(x), up(y), up(mix), up(o), xo, up(i), up(nw), up(sh) if shift else 0, dst, dev.upload(ctrl([pos])),
-                                  dev.upload(bits(wp)), up(b), out, S, N, K, ldw, 2, 0, 1e-3, 0.0)
+    dev.kernel("HyperStreamGemv")(-(-N // 7), up(x), up(y), up(mix), up(o), xo, up(i), up(nw), up(sh) if shift else 0, dst, dev.upload(ctrl([pos])),
+                                  dev.upload(bits(wp)), up(b), out, S, N, K, ldw, 7, 0, 1e-3, 0.0)
     close(dev.download(out, N, np.float32), hs @ d(w).T + d(b), 1e-5)
     close(dev.download(xo, (S, K), np.float32), xn[0], 1e-5)
     if shift:
