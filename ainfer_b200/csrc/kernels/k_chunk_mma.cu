@@ -250,13 +250,13 @@ struct ChunkAttnStepMmaArgs {
   int64_t kv_stride;
   const float *LB;         // [H][lb_len]
   const float *Temp;       // [H]
-  float *Part;             // [seq][G][splits][HG (D + 2)]
+  float *Part;             // [seq][G] blocks of splits HG (D + 4) floats
   uint32_t *Count;         // [seq][G], zero between launches
   void *O;                 // [seq][ldo]
-  int32_t nseq, H, G, D, taps, cap, chunk, lb_len, splits, ldu, ldo, out16;
+  int32_t nseq, H, G, D, taps, cap, chunk, lb_len, splits, ldu, ldo, out16;   // splits <= 16, ldu a multiple of 4
   float scale;
 };
-constexpr int kSmStages = 3;
+constexpr int kSmStages = 3, kSmMaxSplits = 16;   // at most 16 splits
 template <int DP>
 __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &a) {
   extern __shared__ __align__(128) unsigned char sm_raw[];
@@ -286,20 +286,25 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
   __syncthreads();
   float *st = a.State + (size_t)seq * a.taps * C;
   const float *u0 = a.U + (size_t)seq * a.ldu;
-  for (int i = tid; i < (HG + 1) * D; i += 128) {
+  const int slot = pos % a.taps;
+  for (int i = tid * 4; i < (HG + 1) * D; i += 512) {
     const bool isk = i >= HG * D;
     const int c = isk ? Qc + g * D + (i - HG * D) : g * HG * D + i;
-    float y = 0.0f;
+    const float4 u = *reinterpret_cast<const float4 *>(u0 + c);
+    const float4 wl4 = __ldg(reinterpret_cast<const float4 *>(a.CW + (size_t)(a.taps - 1) * C + c));
+    float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 4
     for (int j = 0; j < a.taps - 1; ++j) {
-      const int p = pos - (a.taps - 1 - j);
-      if (p >= 0) y = fmaf(a.CW[(size_t)j * C + c], st[(size_t)(p % a.taps) * C + c], y);
+      const int back = a.taps - 1 - j, s = slot - back < 0 ? slot - back + a.taps : slot - back;
+      const float4 w = __ldg(reinterpret_cast<const float4 *>(a.CW + (size_t)j * C + c));
+      float4 v = *reinterpret_cast<const float4 *>(st + (size_t)s * C + c);
+      if (pos < back) v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      y.x = fmaf(w.x, v.x, y.x); y.y = fmaf(w.y, v.y, y.y); y.z = fmaf(w.z, v.z, y.z); y.w = fmaf(w.w, v.w, y.w);
     }
-    const float u = u0[c];
-    y = fmaf(a.CW[(size_t)(a.taps - 1) * C + c], u, y);
-    if (split == 0) st[(size_t)(pos % a.taps) * C + c] = u;
-    const uint16_t v = f32_to_bf16(y);
-    if (isk) kn[i - HG * D] = v;
-    else Qs[(i / D) * LD + i % D] = v;
+    y.x = fmaf(wl4.x, u.x, y.x); y.y = fmaf(wl4.y, u.y, y.y); y.z = fmaf(wl4.z, u.z, y.z); y.w = fmaf(wl4.w, u.w, y.w);
+    if (split == 0) *reinterpret_cast<float4 *>(st + (size_t)slot * C + c) = u;
+    const uint2 v = make_uint2(pack2(y.x, y.y), pack2(y.z, y.w));
+    *reinterpret_cast<uint2 *>(isk ? kn + (i - HG * D) : Qs + (i / D) * LD + i % D) = v;
   }
   __syncthreads();
   uint32_t q[DP / 16][4];
@@ -393,9 +398,9 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
     if (a.out16) reinterpret_cast<uint16_t *>(a.O)[at] = f32_to_bf16(v);
     else reinterpret_cast<float *>(a.O)[at] = v;
   };
-  const int per_head = D + 2;
-  float *base_p = a.Part + ((size_t)seq * a.G + g) * a.splits * HG * per_head;
-  float *mine = base_p + (size_t)split * HG * per_head;
+  // partials of a (sequence, key head): sums [splits][HG][D], then (maximum, sum) [splits][HG][2]
+  float *base_p = a.Part + ((size_t)seq * a.G + g) * a.splits * HG * (D + 4);   // D + 4 keeps 16-byte alignment
+  float *base_m = base_p + (size_t)a.splits * HG * D;
   for (int i = tid; i < HG * D; i += 128) {
     const int hh = i / D, d = i - hh * D;
     const float M = fmaxf(fmaxf(wm[0][hh], wm[1][hh]), fmaxf(wm[2][hh], wm[3][hh]));
@@ -409,8 +414,8 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
     if (active == 1) {
       put(g * HG + hh, d, v / L);
     } else {
-      __stcg(mine + (size_t)hh * per_head + 2 + d, v);
-      if (d == 0) { __stcg(mine + (size_t)hh * per_head, M); __stcg(mine + (size_t)hh * per_head + 1, L); }
+      __stcg(base_p + (size_t)split * HG * D + i, v);
+      if (d == 0) __stcg(reinterpret_cast<float2 *>(base_m) + split * HG + hh, make_float2(M, L));
     }
   }
   if (active == 1) return;
@@ -424,38 +429,26 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  // split factors of every head, then the sums: loads of all splits are independent
-  float *fac = os;   // [HG][active] exp2(m_s - M), then [HG] 1 / L behind them
+  // every split's factor exp2(m_s - M) / L, then the sums with the loads of all splits in flight
+  float *fac = os;   // [HG][kSmMaxSplits]
   for (int hh = warp; hh < HG; hh += 4) {
-    float M = -INFINITY;
-    for (int s = lane; s < active; s += 32) M = fmaxf(M, __ldcg(base_p + ((size_t)s * HG + hh) * per_head));
-    M = warp_max(M);
-    float L = 0.0f;
-    for (int s = lane; s < active; s += 32) {
-      const float *p = base_p + ((size_t)s * HG + hh) * per_head;
-      const float f = exp2f(__ldcg(p) - M);
-      fac[hh * active + s] = f;
-      L = fmaf(__ldcg(p + 1), f, L);
-    }
-    L = warp_tree_sum(L);
-    if (lane == 0) wm[hh & 3][hh >> 2] = 1.0f / L;
+    const float2 ml = lane < active ? __ldcg(reinterpret_cast<const float2 *>(base_m) + lane * HG + hh) : make_float2(-INFINITY, 0.0f);
+    const float M = warp_max(ml.x), f = exp2f(ml.x - M), L = warp_tree_sum(ml.y * f);
+    if (lane < kSmMaxSplits) fac[hh * kSmMaxSplits + lane] = lane < active ? f / L : 0.0f;
   }
   __syncthreads();
-  for (int i = tid; i < HG * D; i += 128) {
-    const int hh = i / D, d = i - hh * D;
-    const float *p = base_p + (size_t)hh * per_head + 2 + d, *f = fac + hh * active;
-    const size_t stride = (size_t)HG * per_head;
-    float v = 0.0f;
-    int s = 0;
-    for (; s + 8 <= active; s += 8) {
-      float x[8];
+  for (int i = tid * 4; i < HG * D; i += 512) {
+    const int hh = i / D;
+    const float *p = base_p + i, *f = fac + hh * kSmMaxSplits;
+    float4 x[kSmMaxSplits], v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) x[k] = __ldcg(p + (size_t)(s + k) * stride);
+    for (int s = 0; s < kSmMaxSplits; ++s) x[s] = __ldcg(reinterpret_cast<const float4 *>(p + (size_t)min(s, active - 1) * HG * D));
 #pragma unroll
-      for (int k = 0; k < 8; ++k) v = fmaf(x[k], f[s + k], v);
+    for (int s = 0; s < kSmMaxSplits; ++s) {
+      const float w = f[s];
+      v.x = fmaf(x[s].x, w, v.x); v.y = fmaf(x[s].y, w, v.y); v.z = fmaf(x[s].z, w, v.z); v.w = fmaf(x[s].w, w, v.w);
     }
-    for (; s < active; ++s) v = fmaf(__ldcg(p + (size_t)s * stride), f[s], v);
-    put(g * HG + hh, d, v * wm[hh & 3][hh >> 2]);
+    put(g * HG + hh, i % D, v.x); put(g * HG + hh, i % D + 1, v.y); put(g * HG + hh, i % D + 2, v.z); put(g * HG + hh, i % D + 3, v.w);
   }
 }
 #define CHUNK_STEP(DP)                                                                                                  \
@@ -467,7 +460,7 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
   static uint32_t chunk_step_smem##DP(const void *) {                                                                   \
     return (16 + 1 + kSmStages * kCmKeys) * (DP + 8) * 2;                                                               \
   }                                                                                                                     \
-  static_assert(kSmStages * kCmKeys * (DP + 8) * 2 >= 4 * 16 * DP * 4 && 16 * 64 <= 4 * 16 * DP, "merge buffers lie in the key tiles' place");
+  static_assert(kSmStages * kCmKeys * (DP + 8) * 2 >= 4 * 16 * DP * 4 && 16 * kSmMaxSplits <= 4 * 16 * DP, "merge buffers lie in the key tiles' place");
 CHUNK_STEP(32)
 CHUNK_STEP(64)
 CHUNK_STEP(96)

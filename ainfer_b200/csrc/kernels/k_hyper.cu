@@ -68,7 +68,8 @@ __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
   __shared__ StreamCoef coef;
   __shared__ float red[33];
   const int W = a.W, Wp = (W + 3) & ~3, tid = threadIdx.x;
-  load_stream_coef(coef, a.Mix, a.Out, a.In, a.S);
+  load_stream_coef(coef, a.Mix, a.Out, a.In, a.S);   // weights: they do not depend on the predecessor
+  pdl_wait();
   __syncthreads();
   const bool update = a.Y != nullptr;
   const int r0 = blockIdx.x * a.per, r1 = min(a.rows, r0 + a.per);
@@ -105,20 +106,23 @@ __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
     have_prev = true;
   }
   for (int r = r0; r < r1; ++r) {
+    int seq = 0, pos = 0, fr = 0, fn = 0;
+    if (a.Shift) {
+      seq = a.Seq[r]; pos = a.Ctrl[4 * r + CTRL_POS]; fr = a.First[r];
+      fn = r + 1 == a.rows ? r + 1 : a.First[r + 1];
+    }
     norm_row(r, true, cur);
     T *h = H + (size_t)r * a.ldh;
     if (!a.Shift) {
       each([&](int w) { store_val(h + w, cur[w]); });
       continue;
     }
-    const int seq = a.Seq[r], pos = a.Ctrl[4 * r + CTRL_POS];
-    const bool first = a.First[r] == r;
-    if (first || !have_prev) {
+    if (fr == r || !have_prev) {
       const float *st = a.State + ((size_t)seq * 2 + ((pos - 1) & 1)) * W;
       each([&](int w) { prev[w] = pos > 0 ? st[w] : 0.0f; });
     }
     each([&](int w) { store_val(h + w, fmaf(prev[w] - cur[w], a.Shift[w], cur[w])); });
-    if (r + 1 == a.rows || a.First[r + 1] == r + 1) {
+    if (fn == r + 1) {
       float *pd = a.Pend + (size_t)seq * W;
       each([&](int w) { pd[w] = cur[w]; });
     }
@@ -128,12 +132,10 @@ __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
 }
 __global__ void __launch_bounds__(256) HyperNormRowsF32(const HyperNormRowsArgs a) {
   pdl_launch_dependents();
-  pdl_wait();
   hyper_norm_body<float>(a);
 }
 __global__ void __launch_bounds__(256) HyperNormRowsB16(const HyperNormRowsArgs a) {
   pdl_launch_dependents();
-  pdl_wait();
   hyper_norm_body<uint16_t>(a);
 }
 static uint32_t hyper_norm_smem_fn(const void *args) { return 2u * 4u * (uint32_t)((((const HyperNormRowsArgs *)args)->W + 3) & ~3); }
@@ -147,8 +149,8 @@ AINFER_REGISTER(HyperNormRowsB16, HyperNormRowsArgs, 256, 0, 0, hyper_norm_smem_
 
 // Moves a pass's last rows of every sequence into its state, all layers in one launch: the shift row
 // of the sequence's last position q into slot q & 1, and the projections of the last taps - 1
-// positions (as far as the pass holds them) into slots position % taps. One block per (layer, row);
-// rows that are not their sequence's last do nothing.
+// positions (as far as the pass holds them) into slots position % taps. One block per (layer, row from
+// row0 on); rows that are not their sequence's last do nothing.
 struct SeqTailLayer {
   const float *pend_shift;   // [seq][W]
   float *shift;              // [seq][2][W]
@@ -159,12 +161,12 @@ struct SeqTailLayer {
 struct SeqTailCommitArgs {
   const SeqTailLayer *L;
   const int32_t *Ctrl, *Seq, *First;
-  int32_t layers, rows, W;
+  int32_t layers, rows, W, row0;
 };
 __global__ void __launch_bounds__(256) SeqTailCommit(const SeqTailCommitArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int l = blockIdx.x / a.rows, r = blockIdx.x % a.rows;
+  const int n_rows = a.rows - a.row0, l = blockIdx.x / n_rows, r = a.row0 + blockIdx.x % n_rows;
   if (l >= a.layers) return;
   if (r + 1 < a.rows && a.First[r + 1] != r + 1) return;
   const SeqTailLayer L = a.L[l];
@@ -176,7 +178,7 @@ __global__ void __launch_bounds__(256) SeqTailCommit(const SeqTailCommitArgs a) 
   }
 }
 #define F(f) AINFER_ARG(SeqTailCommitArgs, f)
-AINFER_REGISTER(SeqTailCommit, SeqTailCommitArgs, 256, 1, 0, nullptr, F(L), F(Ctrl), F(Seq), F(First), F(layers), F(rows), F(W));
+AINFER_REGISTER(SeqTailCommit, SeqTailCommitArgs, 256, 1, 0, nullptr, F(L), F(Ctrl), F(Seq), F(First), F(layers), F(rows), F(W), F(row0));
 #undef F
 
 AINFER_EARLY_LAUNCH(EmbedPosRows);

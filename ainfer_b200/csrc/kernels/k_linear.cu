@@ -75,9 +75,10 @@ AINFER_REGISTER(LinearRows, LinearRowsArgs, 256, 0, 0, nullptr, F(X), F(W), F(Bi
 // ---------------------------------------------------------- StreamGemv ---
 // The block's rows are one contiguous range of bytes: a producer warp brings them in tiles of whole rows
 // (about 16 KB) through a ring of shared-memory stages with bulk copies, which start before the kernel's
-// dependency wait (weights do not depend on it); 16 consumer warps multiply. Per tile a row is shared
+// dependency wait (weights do not depend on it); 8 consumer warps multiply. Two blocks per SM: one
+// block's copies complete at a rate that fills about half of an SM's share of the HBM bandwidth. Per tile a row is shared
 // by wpr warps; the partial sums of all rows stay in shared memory until the block's last tile.
-constexpr int kSgWarps = 16, kSgThreads = kSgWarps * 32 + 32, kSgRing = 65536;
+constexpr int kSgWarps = 8, kSgThreads = kSgWarps * 32 + 32, kSgRing = 65536;
 constexpr uint32_t kSgSpin = 1u << 22;
 struct GemvDims { int tile_rows, stage_bytes, nst, wpr; };
 __host__ __device__ inline GemvDims gemv_dims(int ldw) {
@@ -210,7 +211,7 @@ struct StreamGemvArgs {
   float cap;
 };
 extern __shared__ __align__(128) unsigned char sg_smem[];
-__global__ void __launch_bounds__(kSgThreads, 2) StreamGemv(const StreamGemvArgs a) {
+__global__ void __launch_bounds__(kSgThreads, 4) StreamGemv(const StreamGemvArgs a) {
   __shared__ GemvShared sh;
   pdl_launch_dependents();
   const GemvDims d = gemv_dims(a.ldw);
@@ -222,7 +223,7 @@ __global__ void __launch_bounds__(kSgThreads, 2) StreamGemv(const StreamGemvArgs
   } else {
     pdl_wait();
     for (int k = threadIdx.x; k < a.ldw; k += kSgWarps * 32) sg_put(lo, hi, k, k < a.K ? a.X[k] : 0.0f);
-    asm volatile("bar.sync 1, 512;" ::: "memory");
+    asm volatile("bar.sync 1, 256;" ::: "memory");
     gemv_consume(c, d, &sh, sg_smem, lo, hi, part);
   }
   __syncthreads();
@@ -253,7 +254,7 @@ struct HyperStreamGemvArgs {
   int32_t S, N, K, ldw, rows_pb, act;
   float eps, cap;
 };
-__global__ void __launch_bounds__(kSgThreads, 2) HyperStreamGemv(const HyperStreamGemvArgs a) {
+__global__ void __launch_bounds__(kSgThreads, 4) HyperStreamGemv(const HyperStreamGemvArgs a) {
   __shared__ GemvShared sh;
   __shared__ StreamCoef coef;
   __shared__ float red[33];
@@ -273,7 +274,7 @@ __global__ void __launch_bounds__(kSgThreads, 2) HyperStreamGemv(const HyperStre
     float ss = stream_row_any(a.Xin, a.Yp, blockIdx.x == 0 ? a.Xout : nullptr, coef, a.S, K, a.Yp != nullptr, us, tid, nth);
     ss = warp_tree_sum(ss);
     if (lane == 0) red[warp] = ss;
-    asm volatile("bar.sync 1, 512;" ::: "memory");   // also: every thread's u is visible
+    asm volatile("bar.sync 1, 256;" ::: "memory");   // also: every thread's u is visible
     ss = warp_tree_sum(lane < kSgWarps ? red[lane] : 0.0f);
     const float inv = 1.0f / sqrtf(ss / (float)K + a.eps);
     const int pos = a.Shift ? a.Ctrl[CTRL_POS] : 0;
@@ -291,7 +292,7 @@ __global__ void __launch_bounds__(kSgThreads, 2) HyperStreamGemv(const HyperStre
       }
       sg_put(lo, hi, k, v);
     }
-    asm volatile("bar.sync 1, 512;" ::: "memory");
+    asm volatile("bar.sync 1, 256;" ::: "memory");
     gemv_consume(c, d, &sh, sg_smem, lo, hi, part);
   }
   __syncthreads();

@@ -209,8 +209,9 @@ static uint32_t linear_tc_smem(const void *args) {
 }
 
 // ---- K split over a cluster ----
+// Half of an SM's shared memory, so that the next launch's blocks (or a second one of this) fit beside.
 __host__ __device__ inline uint32_t lts_stages(int nt) {
-  const uint32_t s = ((uint32_t)kLtBudget - (uint32_t)nt * 512u) / lt_stage_bytes(nt);
+  const uint32_t s = ((uint32_t)kLtBudget / 2 + 8192 - (uint32_t)nt * 512u) / lt_stage_bytes(nt);
   return s > 8 ? 8 : s;
 }
 __device__ __forceinline__ void cluster_sync_all() {
@@ -252,15 +253,23 @@ __device__ __forceinline__ void linear_tc_split(const LinearTcArgs &a) {
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const uint32_t tmem = sh.tmem;
   cluster_sync_all();   // every block of the cluster runs: its shared memory may be written
+  int pre = 0;          // stages whose weights travel before the dependency wait (they do not depend on it)
+  if (warp == 0 && lane == 0)
+    for (; pre < nst && k_lo + pre < k_hi; ++pre) {
+      mbar_arrive_expect(&sh.full[pre], stage_bytes);
+      lt_tma(base + (uint32_t)pre * stage_bytes, &a.Wm, smem_addr(&sh.full[pre]), (k_lo + pre) * 64, n0);
+    }
   pdl_wait();
 
   if (warp == 0 && lane == 0) {
     uint32_t st = 0, ph = 1, issued = 0;
     for (int k = k_lo; k < k_hi; ++k) {
-      if (!lt_wait(&sh, &sh.empty[st], ph)) break;
       const uint32_t dst = base + st * stage_bytes, bar = smem_addr(&sh.full[st]);
-      mbar_arrive_expect(&sh.full[st], stage_bytes);
-      lt_tma(dst, &a.Wm, bar, k * 64, n0);
+      if (k - k_lo >= pre) {
+        if (!lt_wait(&sh, &sh.empty[st], ph)) break;
+        mbar_arrive_expect(&sh.full[st], stage_bytes);
+        lt_tma(dst, &a.Wm, bar, k * 64, n0);
+      }
       lt_tma(dst + 128u * 128u, &a.Xm, bar, k * 64, r0);
       ++issued;
       if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
@@ -332,9 +341,9 @@ __device__ __forceinline__ void linear_tc_split(const LinearTcArgs &a) {
   __syncthreads();
   if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
 }
-__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit2(const __grid_constant__ LinearTcArgs a) { linear_tc_split<2>(a); }
-__global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit4(const __grid_constant__ LinearTcArgs a) { linear_tc_split<4>(a); }
-__global__ void __cluster_dims__(8, 1, 1) __launch_bounds__(kLtThreads, 1) LinearTcSplit8(const __grid_constant__ LinearTcArgs a) { linear_tc_split<8>(a); }
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kLtThreads, 2) LinearTcSplit2(const __grid_constant__ LinearTcArgs a) { linear_tc_split<2>(a); }
+__global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(kLtThreads, 2) LinearTcSplit4(const __grid_constant__ LinearTcArgs a) { linear_tc_split<4>(a); }
+__global__ void __cluster_dims__(8, 1, 1) __launch_bounds__(kLtThreads, 2) LinearTcSplit8(const __grid_constant__ LinearTcArgs a) { linear_tc_split<8>(a); }
 static uint32_t linear_tc_split_smem(const void *args) {
   const int nt = ((const LinearTcArgs *)args)->nt;
   return lts_stages(nt) * lt_stage_bytes(nt) + (uint32_t)nt * 512u + 1024;

@@ -393,7 +393,7 @@ struct Engine : RowEngine {
       maxF = std::max(maxF, r.ff);
       maxC = std::max(maxC, (r.heads + r.kv_heads) * r.dim);
       maxG = std::max(maxG, r.kv_heads);
-      maxHGD = std::max(maxHGD, r.heads * (r.dim + 2));
+      maxHGD = std::max(maxHGD, r.heads * (r.dim + 4));
     }
     state_bytes = off;
     int e = alloc(state_bytes, &state);
@@ -411,8 +411,8 @@ struct Engine : RowEngine {
       ts.push_back({s.pend_shift, s.shift, nullptr, nullptr, C, 1});   // steps keep their convolution ring themselves
     }
     ldw = round_up((int)W, 8); ldq = round_up(maxQ, 8); ldf = round_up(maxF, 8);
-    // blocks of a step's attention: about four per SM over sequences, key heads and splits
-    att_splits = std::max(1, std::min(64, 4 * sm_count / (std::min(nseq, 4 * sm_count) * maxG)));
+    // blocks of a step's attention over sequences, key heads and splits: few tiles each when there are many sequences
+    att_splits = nseq == 1 ? std::max(1, std::min(16, 2 * sm_count / maxG)) : std::max(1, std::min(16, 8 * sm_count / (std::min(nseq, 8 * sm_count) * maxG)));
     for (int i = 0; i < 2; ++i) e |= alloc(R * S * W, &X[i]);
     e |= alloc(R * ldw * esz(), &H); e |= alloc(R * maxC, &U); e |= alloc(R * ldq * esz(), &Q);
     e |= alloc(R * ldq * 4, &Att); e |= alloc(R * W, &Y); e |= alloc(R * ldf * 4, &Act);
@@ -531,8 +531,9 @@ struct Engine : RowEngine {
       hyper(k, sp, nullptr, w->final_norm, nullptr, nullptr, sp.n_want, sp.want, false);
       linear(k, w->head, H, ldw, sp.n_want, sp.logits, c.vocab, c.logit_softcap > 0 ? ACT_SOFTCAP : ACT_NONE, false, (float)c.logit_softcap);
     }
-    k.launch("SeqTailCommit", (uint32_t)(c.layers * R), (const void *)(sp.one_sequence ? tail_rows : tail_steps), sp.ctrl, sp.seq, sp.first,
-             (int32_t)c.layers, (int32_t)R, (int32_t)W);
+    const int row0 = sp.one_sequence ? R - 1 : 0;   // the first row that may be its sequence's last
+    k.launch("SeqTailCommit", (uint32_t)(c.layers * (R - row0)), (const void *)(sp.one_sequence ? tail_rows : tail_steps), sp.ctrl, sp.seq, sp.first,
+             (int32_t)c.layers, (int32_t)R, (int32_t)W, (int32_t)row0);
   }
 
   // head sizes the tensor-core attention takes (bf16), and the name of the instance that holds one
@@ -554,14 +555,14 @@ struct Engine : RowEngine {
 
   // ---- one decode step of sequence 0 ----
   void gemv(KernelCalls &k, const RowMatrix &mt, const float *x, float *y, int act) {
-    const int rows_pb = (mt.N + sm_count - 1) / sm_count;
+    const int rows_pb = (mt.N + 2 * sm_count - 1) / (2 * sm_count);
     k.launch("StreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), x, mt.w, mt.bias, y, (int32_t)mt.N, (int32_t)mt.K, (int32_t)mt.ldw,
              (int32_t)rows_pb, (int32_t)act, 0.0f);
   }
   void hyper_gemv(KernelCalls &k, const RowMatrix &mt, const float *in, const float *norm, const float *shift, float *shift_state,
                   const int32_t *ctrl, float *y, int act, float cap) {
     const ModelConfig &c = m->cfg;
-    const int rows_pb = (mt.N + sm_count - 1) / sm_count;
+    const int rows_pb = (mt.N + 2 * sm_count - 1) / (2 * sm_count);
     k.launch("HyperStreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), (const float *)X[cur], (const float *)(pending ? Y : nullptr),
              (const float *)(pending ? pending->mix : nullptr), (const float *)(pending ? pending->out : nullptr),
              (float *)(pending ? X[cur ^ 1] : nullptr), in, norm, shift, shift_state, ctrl, mt.w, mt.bias, y, (int32_t)c.streams, (int32_t)mt.N,

@@ -148,7 +148,7 @@ def test_short_convolution_over_rows(dev, taps, Qc, Kn, per, kind):
     W = 6
     psh, sh = dev.upload(np.arange(2 * W, dtype=np.float32)), dev.zeros(2 * 2 * W * 4)
     rec[0] = (psh, sh, pend, dst, C, taps)
-    dev.kernel("SeqTailCommit")(17, dev.upload(rec.view(np.uint8)), *ctl, 1, 17, W)
+    dev.kernel("SeqTailCommit")(17, dev.upload(rec.view(np.uint8)), *ctl, 1, 17, W, 0)
     dev.sync()
     ring, shift = dev.download(dst, (2, taps, C), np.float32), dev.download(sh, (2, 2, W), np.float32)
     for s, last in ((0, 8), (1, 20)):
@@ -252,7 +252,7 @@ def test_decode_attention_with_convolution(dev, H, G, D, chunk, taps, splits, ki
     # slots hold leftovers of earlier sequences
     st = dev.upload(rng.standard_normal((3, taps, C)).astype(np.float32))
     kc = dev.upload(f32(torch.randn(3, cap, K, generator=g)) if kind == "f32" else bits(torch.randn(3, cap, K, generator=g)))
-    part, cnt = dev.zeros(3 * splits * H * (D + 2) * 4), dev.zeros(3 * G * 4)
+    part, cnt = dev.zeros(3 * splits * H * (D + 4) * 4), dev.zeros(3 * G * 4)
     o, du, dc = dev.zeros(3 * Q * 4), dev.zeros(3 * C * 4), dev.zeros(48)
     k = dev.kernel({"f32": "ChunkAttnStepF32", "b16": "ChunkAttnStepB16", "mma": _mma("ChunkAttnStepMma", D)}[kind])
     got = np.zeros((3, T, Q), np.float32)
