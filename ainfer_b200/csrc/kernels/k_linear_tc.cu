@@ -16,6 +16,7 @@
 // the block's other waits return at once and the kernel ends (copies in flight awaited, tensor memory
 // freed).
 #include <cuda.h>
+#include <cuda_bf16.h>
 
 #include "weight_ring.cuh"
 
@@ -64,6 +65,41 @@ __device__ __forceinline__ void lt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
       : "r"(taddr)
       : "memory");
 }
+__device__ __forceinline__ void lt_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ float lt_act(float v, int act, float cap) {
+  if (act == 1) { v = v > 0.0f ? v : 0.0f; return v * v; }
+  if (act == 2) return cap * tanhf(v / cap);
+  return v;
+}
+// One accumulator lane (an output feature) over nr rows: y points at the feature in the tile's first
+// row. No branch depends on data, so the columns of a load overlap; the next columns' load is in flight
+// while these are stored.
+template <int ACT, typename T>
+__device__ __forceinline__ void lt_store16(const uint32_t (&v)[16], T *y, size_t ldy, float bias, float cap, bool in, int left) {
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    const float r = lt_act(__uint_as_float(v[i]) + bias, ACT, cap);
+    if (in && i < left) {
+      if constexpr (sizeof(T) == 2) y[i * ldy] = __float2bfloat16_rn(r);
+      else y[i * ldy] = r;
+    }
+  }
+}
+template <int ACT, typename T>
+__device__ __forceinline__ void lt_epilogue(uint32_t taddr, int nr, T *y, int ld, float bias, float cap, bool in) {
+  const size_t ldy = (size_t)ld;
+  uint32_t a[16], b[16];
+  lt_ld16(taddr, a);
+  for (int c = 0; c < nr; c += 32) {
+    lt_ld_wait();
+    if (c + 16 < nr) lt_ld16(taddr + (uint32_t)c + 16u, b);
+    lt_store16<ACT, T>(a, y + (size_t)c * ldy, ldy, bias, cap, in, nr - c);
+    if (c + 16 >= nr) break;
+    lt_ld_wait();
+    if (c + 32 < nr) lt_ld16(taddr + (uint32_t)c + 32u, a);
+    lt_store16<ACT, T>(b, y + (size_t)(c + 16) * ldy, ldy, bias, cap, in, nr - c - 16);
+  }
+}
 
 struct LtShared {
   unsigned long long full[8], empty[8], acc_full[2], acc_empty[2], drain;
@@ -78,12 +114,6 @@ __device__ __forceinline__ bool lt_wait(LtShared *s, unsigned long long *b, uint
   *reinterpret_cast<volatile uint32_t *>(&s->fail) = 1;
   if (g_stream_fault_word) *reinterpret_cast<volatile unsigned int *>(g_stream_fault_word) = 1;
   return false;
-}
-
-__device__ __forceinline__ float lt_act(float v, int act, float cap) {
-  if (act == 1) { v = v > 0.0f ? v : 0.0f; return v * v; }
-  if (act == 2) return cap * tanhf(v / cap);
-  return v;
 }
 
 __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant__ LinearTcArgs a) {
@@ -178,20 +208,18 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
       __syncwarp();
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t taddr = tmem + buf * (uint32_t)nt + ((uint32_t)((warp & 3) * 32) << 16);
-      auto emit = [&](int r, float v) {
-        if (n >= a.N) return;
-        v = lt_act(v + bias, a.act, a.cap);
-        const size_t o = (size_t)(r0 + r) * a.ldy + n;
-        if (a.out16) reinterpret_cast<uint16_t *>(a.Y)[o] = f32_to_bf16(v);
-        else reinterpret_cast<float *>(a.Y)[o] = v;
-      };
-      for (int c = 0; c < nr; c += 16) {
-        uint32_t v[16];
-        lt_ld16(taddr + (uint32_t)c, v);
-        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-        for (int i = 0; i < 16; ++i)
-          if (c + i < nr) emit(c + i, __uint_as_float(v[i]));
+      const bool in = n < a.N;
+      const size_t o = (size_t)r0 * a.ldy + n;
+      if (a.out16) {
+        __nv_bfloat16 *y = reinterpret_cast<__nv_bfloat16 *>(a.Y) + o;
+        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, a.cap, in);
+      } else {
+        float *y = reinterpret_cast<float *>(a.Y) + o;
+        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, a.cap, in);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       mbar_arrive(&sh.acc_empty[buf]);
@@ -304,6 +332,7 @@ __device__ __forceinline__ void linear_tc_split(const LinearTcArgs &a) {
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t taddr = tmem + ((uint32_t)((warp & 3) * 32) << 16);
     const uint32_t mine = red + ((uint32_t)rank * (uint32_t)rpo * 128u + (uint32_t)lw) * 4u;
+    const int lg = 31 - __clz(rpo);   // nt and the cluster size are powers of two
     for (int c = 0; c < nr; c += 16) {
       uint32_t v[16];
       lt_ld16(taddr + (uint32_t)c, v);
@@ -313,7 +342,7 @@ __device__ __forceinline__ void linear_tc_split(const LinearTcArgs &a) {
         const int col = c + i;
         if (col < nr) {
           uint32_t peer;
-          asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(peer) : "r"(mine + (uint32_t)(col % rpo) * 512u), "r"(col / rpo));
+          asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(peer) : "r"(mine + (uint32_t)(col & (rpo - 1)) * 512u), "r"(col >> lg));
           asm volatile("st.shared::cluster.u32 [%0], %1;" ::"r"(peer), "r"(v[i]) : "memory");
         }
       }

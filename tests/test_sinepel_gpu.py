@@ -287,7 +287,7 @@ def test_linear_rows_32bit(dev, R, N, K, act):
 @pytest.mark.parametrize("R,N,K,nt,splits,act,out16", [
     (1, 5, 40, 16, 1, 0, 0), (17, 130, 200, 32, 1, 2, 0), (64, 256, 1024, 64, 4, 0, 0), (300, 384, 136, 128, 1, 1, 1), (520, 640, 512, 256, 1, 0, 0),
     (30, 100, 4096, 16, 8, 1, 1), (1000, 1536, 320, 256, 1, 1, 1), (129, 128, 64, 128, 1, 0, 0), (5, 300, 520, 16, 2, 0, 0), (100, 260, 2048, 128, 8, 2, 0),
-    (33, 128, 72, 64, 2, 0, 1)])
+    (33, 128, 72, 64, 2, 0, 1), (401, 200, 264, 176, 1, 1, 0), (97, 128, 64, 96, 1, 2, 1)])
 def test_linear_tensor_cores(dev, R, N, K, nt, splits, act, out16):
     g = torch.Generator().manual_seed(R)
     x, w, b = bf16(torch.randn(R, K, generator=g)), bf16(torch.randn(N, K, generator=g)), torch.randn(N, generator=g)
