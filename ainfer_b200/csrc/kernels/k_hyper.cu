@@ -147,6 +147,26 @@ AINFER_REGISTER(HyperNormRowsF32, HyperNormRowsArgs, 256, 0, 0, hyper_norm_smem_
 AINFER_REGISTER(HyperNormRowsB16, HyperNormRowsArgs, 256, 0, 0, hyper_norm_smem_fn, HYPER_FIELDS);
 #undef F
 
+// Dst[row] = sum of the row's streams after a pending update (diagnostics: the residual a layer leaves).
+struct StreamSumRowsArgs {
+  const float *X, *Y, *Mix, *Out;   // Y null: no pending update
+  float *Dst;                       // [rows][W]
+  int32_t W, S;
+};
+__global__ void __launch_bounds__(256) StreamSumRows(const StreamSumRowsArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ StreamCoef coef;
+  load_stream_coef(coef, a.Mix, a.Out, nullptr, a.S);
+  __syncthreads();
+  const size_t row = blockIdx.x;
+  for (int w = threadIdx.x; w < a.W; w += 256)
+    a.Dst[row * a.W + w] = stream_step_n(a.X + row * a.S * a.W + w, a.Y + (a.Y ? row * a.W + w : 0), nullptr, coef, a.S, a.W, a.Y != nullptr);
+}
+#define F(f) AINFER_ARG(StreamSumRowsArgs, f)
+AINFER_REGISTER(StreamSumRows, StreamSumRowsArgs, 256, 1, 0, nullptr, F(X), F(Y), F(Mix), F(Out), F(Dst), F(W), F(S));
+#undef F
+
 // Moves a pass's last rows of every sequence into its state, all layers in one launch: the shift row
 // of the sequence's last position q into slot q & 1, and the projections of the last taps - 1
 // positions (as far as the pass holds them) into slots position % taps. One block per (layer, row from
@@ -185,5 +205,6 @@ AINFER_EARLY_LAUNCH(EmbedPosRows);
 AINFER_EARLY_LAUNCH(HyperNormRowsF32);
 AINFER_EARLY_LAUNCH(HyperNormRowsB16);
 AINFER_EARLY_LAUNCH(SeqTailCommit);
+AINFER_EARLY_LAUNCH(StreamSumRows);
 
 }  // namespace ainfer

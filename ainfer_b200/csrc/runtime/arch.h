@@ -44,6 +44,7 @@ struct RowEngine {                // state of `nseq` sequences plus the buffers 
   // one decode step of sequence 0 as recorded launches: embedding, one layer, final norm + head
   virtual void record_embed(KernelCalls &k, const int32_t *ctrl) = 0;
   virtual void record_layer(KernelCalls &k, int layer, const int32_t *ctrl) = 0;
+  virtual void record_residual(KernelCalls &k, float *dst) = 0;   // after a layer: the residual it leaves [hidden]
   virtual void record_head(KernelCalls &k, float *logits) = 0;
   int rows_cap = 0;
 };
@@ -51,6 +52,7 @@ struct RowEngine {                // state of `nseq` sequences plus the buffers 
 // f32: activations and cache in 32-bit. Returns 0, 1 (device) or 2 (usage).
 int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err);
 
+bool sinepel_preset(const std::string &name, ModelConfig &c);   // "sinepel-tiny", "sinepel-small"
 const ModelArch *sinepel_model_arch();
 const ModelArch *int4_hybrid_model_arch();
 

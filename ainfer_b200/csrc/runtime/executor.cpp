@@ -206,6 +206,7 @@ void record_attn_layer(Recorder &r, int L, const std::string &p) {
 void record_layer(Recorder &r, int L) {
   if (r.s->rows) {
     r.s->rows->record_layer(r, L, r.s->ctrl);
+    if (r.s->layer_out) r.s->rows->record_residual(r, r.s->layer_out + (size_t)L * r.s->m->cfg.hidden);
     return;
   }
   if (r.s->m->cfg.layer_types[L] == 'A') record_attn_layer(r, L, layer_prefix(L));
@@ -481,7 +482,7 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
   if (row_arch) {
     // learned positions bound the context; the persistent step is the INT4 hybrid's, here a token is always a recorded list
     s->max_ctx = max_ctx = std::min(max_ctx, c.max_positions);
-    s->flags = flags &= ~(SESSION_PERSISTENT | SESSION_STAGE_CLOCK | SESSION_DIAG);
+    s->flags = flags &= ~(SESSION_PERSISTENT | SESSION_STAGE_CLOCK);
     const int e = row_engine_create(m, 1, max_ctx, std::min(max_ctx, kRowEnginePassRows), (flags & SESSION_F32) != 0, &s->rows, s->err);
     if (e) return fail(e);
   } else if (flags & SESSION_F32) {
@@ -501,6 +502,7 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
   r |= salloc(s, (size_t)c.vocab, &s->Logits);
   r |= salloc(s, (size_t)s->argmax_parts, &s->PV);
   r |= salloc(s, (size_t)s->argmax_parts, &s->PI);
+  if (flags & SESSION_DIAG) r |= salloc(s, (size_t)c.layers * H, &s->layer_out);
   if (!row_arch) {
     if (model_ensure_rope(m, max_ctx, s->err)) return fail(1);
     size_t n_kv = (size_t)n_kv_layers * max_ctx * nKV;
@@ -545,7 +547,6 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
       r |= salloc(s, 1, &s->out_tok_m);
     }
     if (flags & SESSION_DIAG) {
-      r |= salloc(s, (size_t)c.layers * H, &s->layer_out);
       r |= salloc(s, (size_t)c.layers * (c.top_k + 1), &s->routed);
       r |= salloc(s, (size_t)c.layers, &s->near_gap);
     }

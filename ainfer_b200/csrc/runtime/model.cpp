@@ -161,6 +161,8 @@ bool preset_config(const std::string &name, ModelConfig &c) {
     std::string js, err;
     return read_text(name.substr(7), js) && ModelConfig::from_json(js, c, err);
   }
+  if (sinepel_preset(name, c)) return true;
+  c = ModelConfig();
   if (name == "tiny") {
     c.hidden = 256; c.layers = 2; c.layer_types = "LA"; c.vocab = 512;
     c.q_heads = 2; c.kv_heads = 1; c.lin_k_heads = 2; c.lin_v_heads = 4;

@@ -142,7 +142,7 @@ int ainfer_session_buffer(ainfer_session_t h, const char *which, void **dptr, ui
   const ModelConfig &c = s->m->cfg;
   std::string w = which;
   if (s->rows && s->rows->buffer(w, dptr, bytes)) return 0;
-  if (s->rows && w != "logits" && w != "ctrl" && w != "history") return set_err(2, "unknown session buffer: " + w);
+  if (s->rows && w != "logits" && w != "ctrl" && w != "history" && w != "layer_out") return set_err(2, "unknown session buffer: " + w);
   size_t n_kv = (size_t)(c.n_attn() + c.mtp_layers) * s->max_ctx * c.kv_heads;
   if (w == "conv") { *dptr = s->conv; *bytes = (uint64_t)c.n_lin() * c.conv_dim() * 3 * 4; }
   else if (w == "S") { *dptr = s->S; *bytes = (uint64_t)c.n_lin() * c.lin_v_heads * 128 * 128 * 4; }

@@ -599,6 +599,10 @@ struct Engine : RowEngine {
       pending = &lw.sub[1];
     }
   }
+  void record_residual(KernelCalls &k, float *dst) override {
+    k.launch("StreamSumRows", 1, (const float *)X[cur], (const float *)(pending ? Y : nullptr), (const float *)(pending ? pending->mix : nullptr),
+             (const float *)(pending ? pending->out : nullptr), dst, (int32_t)m->cfg.hidden, (int32_t)m->cfg.streams);
+  }
   void record_head(KernelCalls &k, float *logits) override {
     const ModelConfig &c = m->cfg;
     hyper_gemv(k, w->head, nullptr, w->final_norm, nullptr, nullptr, nullptr, logits, c.logit_softcap > 0 ? ACT_SOFTCAP : ACT_NONE,
@@ -609,6 +613,29 @@ struct Engine : RowEngine {
 }  // namespace
 
 const ModelArch *sinepel_model_arch() { return &kModel; }
+
+bool sinepel_preset(const std::string &name, ModelConfig &c) {
+  auto layer = [](int heads, int kv_heads, int dim, int taps, int chunk, int ff) {
+    RowLayerConfig r;
+    r.heads = heads; r.kv_heads = kv_heads; r.dim = dim; r.taps = taps; r.chunk = chunk; r.ff = ff;
+    r.scale = 1.0 / std::sqrt((double)dim);
+    return r;
+  };
+  c = ModelConfig();
+  c.arch = "Sinepel";
+  c.logit_softcap = 30.0;
+  if (name == "sinepel-tiny") {
+    c.hidden = 96; c.vocab = 512; c.streams = 3; c.max_positions = 1024;
+    c.row_layers = {layer(4, 2, 32, 3, 48, 160), layer(6, 2, 16, 2, 100, 0), layer(3, 1, 40, 4, 32, 128)};
+  } else if (name == "sinepel-small") {
+    c.hidden = 2048; c.vocab = 32000; c.streams = 4; c.max_positions = 8192;
+    c.row_layers.assign(4, layer(16, 4, 128, 4, 2048, 8192));
+  } else {
+    return false;
+  }
+  c.layers = (int)c.row_layers.size();
+  return true;
+}
 
 int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err) {
   *out = nullptr;

@@ -37,7 +37,7 @@ const char *ainfer_rt_last_error(void);
  * CRCs and trailing SHA-256 (docs/binfer_spec.md section 11). */
 int ainfer_binfer_validate(const char *path, int level);
 /* Writes a synthetic model of a named shape ("tiny", "mini", "mini-mtp",
- * "small", "full") on the host. Counterpart of tools/binfer.py cmd_quantize
+ * "small", "full", "sinepel-tiny", "sinepel-small") on the host. Counterpart of tools/binfer.py cmd_quantize
  * (:155-353) with seeded N(0, 0.02) weights in place of a checkpoint. */
 int ainfer_synth_write(const char *path, const char *preset, uint64_t seed);
 /* Checkpoint ingestion: a SafeTensors file, or a directory holding model.safetensors.index.json
@@ -91,7 +91,7 @@ int ainfer_session_destroy(ainfer_session_t s);
 int ainfer_session_reset(ainfer_session_t s);
 /* Device buffers of the session, for state upload/download by tests (architectures with residual
  * streams: "shift", "conv", "Kc", all layers of each, "state" for the three together, and the common
- * "logits", "ctrl", "history"):
+ * "logits", "ctrl", "history", "layer_out"):
  * "conv", "S", "Kc", "Vc", "Ks", "Vs", "logits", "x", "ctrl", "layer_out",
  * "routed", "near_gap", "history", "stage_stamps". */
 int ainfer_session_buffer(ainfer_session_t s, const char *which, void **dptr, uint64_t *bytes);

@@ -1,9 +1,7 @@
 """Sinepel without a GPU: the plain restatement's mechanisms against hand-worked cases, the
 configuration reader (round trip, refusals), and the container / SafeTensors paths of the loader."""
-import ctypes as C
 import json
 import math
-import os
 
 import pytest
 import torch
@@ -126,6 +124,13 @@ def test_synthetic_file_and_conversion(rt, tmp_path):
     P.write_model(str(tmp_path / "bad2"), c, bad)
     with pytest.raises(rt.RuntimeError_, match="missing l1.shift"):
         rt.from_safetensors(str(tmp_path / "bad2"), json.dumps(c), str(tmp_path / "x.binfer"))
+
+
+@pytest.mark.parametrize("name", ["sinepel-tiny", "sinepel-small"])
+def test_named_shapes(rt, name):
+    c = json.loads(rt.preset_config_json(name))
+    assert c["architecture"] == "Sinepel" and len(c["layers"]) >= 3
+    assert all(ly["mixer"]["heads"] % ly["mixer"]["kv_heads"] == 0 for ly in c["layers"])
 
 
 def test_plain_reader_and_writer_agree(tmp_path):

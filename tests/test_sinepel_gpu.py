@@ -486,6 +486,19 @@ def test_greedy_generation_everywhere(rt, bundle):
         assert [int(x) for x in line.split()[1:]] == want, spec
 
 
+def test_residual_after_every_layer(rt, bundle):
+    c, plain, model, toks, _, _ = bundle
+    _, layers = plain.forward(toks[:60], want_layers=True)
+    s = rt.Session(model, 96, rt.Session.F32 | rt.Session.DIAG)
+    s.prefill(toks[:50])
+    for i in range(50, 60):
+        s.step(toks[i], i)
+        got = s.read("layer_out", np.float32).reshape(len(c["layers"]), -1)
+        for L in range(len(c["layers"])):
+            close(got[L], layers[L, i], 3e-5)
+    s.close()
+
+
 def test_bf16_generation_follows_the_plain_logits(rt, bundle):
     c, plain, model, toks, _, _ = bundle
     s = rt.Session(model, 96)
@@ -561,6 +574,11 @@ def test_limits_are_refused(dev, rt, tmp_path):
         s.mtp_draft(1, 1)
     s.close()
     model.close()
+    named = rt.Model(dev, "synth:sinepel-tiny:seed=3")
+    s = rt.Session(named, 4096, rt.Session.PERSISTENT)      # no persistent step: a recorded list
+    assert s.launches_per_token() > 1 and len(s.generate([1, 2, 3], 5)) == 5
+    s.close()
+    named.close()
     tiny = rt.Model(dev, "synth:tiny")
     with pytest.raises(rt.RuntimeError_, match="32-bit"):
         rt.Session(tiny, 32, rt.Session.F32)
