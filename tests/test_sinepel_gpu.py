@@ -347,6 +347,8 @@ L = P.make_layer
 MODELS = {
     "mixed": P.make_config(layers=[L(), L(heads=6, kv_heads=3, dim=20, conv=1, chunk=7, ff=None), L(heads=2, kv_heads=2, dim=48, conv=5, chunk=40, ff=33)]),
     "odd": P.make_config(width=50, vocab=77, streams=1, layers=[L(heads=3, kv_heads=1, dim=10, chunk=16, ff=21), L(heads=1, kv_heads=1, dim=9, ff=None)]),
+    "many": P.make_config(width=72, vocab=130, streams=2, layers=[L(heads=20, kv_heads=1, dim=16, conv=3, chunk=30, ff=100),
+                                                                  L(heads=34, kv_heads=2, dim=12, conv=6, chunk=55, ff=40)]),
     "wide": P.make_config(width=128, vocab=320, streams=4, eps=1e-3, embed_scale=0.5, cap=4.0,
                           layers=[L(heads=8, kv_heads=2, dim=32, conv=4, chunk=96, ff=512), L(heads=4, kv_heads=4, dim=64, conv=2, chunk=33, ff=256)]),
     "pairs": P.make_config(width=40, vocab=90, streams=6, layers=[L(heads=4, kv_heads=1, dim=24, conv=4, chunk=1000, ff=64),
