@@ -71,6 +71,27 @@ __device__ __forceinline__ void scores(float (&s)[NK / 8][4], const uint32_t (&q
       mma16816(s[2 * n + 1], q[kk], b[2], b[3]);
     }
 }
+// The same with the query fragments read from shared memory (qa: this lane's address in the warp's 16 rows).
+template <int DP, int NK>
+__device__ __forceinline__ void scores_smem(float (&s)[NK / 8][4], uint32_t qa, uint32_t kt, int lane) {
+#pragma unroll
+  for (int n = 0; n < NK / 8; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) s[n][i] = 0.0f;
+  const uint32_t a = kt + (uint32_t)(((lane & 7) + ((lane >> 4) & 1) * 8) * (DP + 8) + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+  for (int kk = 0; kk < DP / 16; ++kk) {
+    uint32_t q[4];
+    ldm4(q, qa + (uint32_t)(kk * 32));
+#pragma unroll
+    for (int n = 0; n < NK / 16; ++n) {
+      uint32_t b[4];
+      ldm4(b, a + (uint32_t)(n * 16 * (DP + 8) + kk * 16) * 2);
+      mma16816(s[2 * n], q, b[0], b[1]);
+      mma16816(s[2 * n + 1], q, b[2], b[3]);
+    }
+  }
+}
 // o += weights (as the score fragments hold them) . keys of the tile
 template <int DP, int NK>
 __device__ __forceinline__ void values(float (&o)[DP / 8][4], const float (&p)[NK / 8][4], uint32_t kt, int lane) {
@@ -87,6 +108,11 @@ __device__ __forceinline__ void values(float (&o)[DP / 8][4], const float (&p)[N
       mma16816(o[2 * d + 1], w, b[2], b[3]);
     }
   }
+}
+__device__ __forceinline__ float fast_exp2(float x) {   // one instruction, 2 ulp, small results flushed to zero
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 __device__ __forceinline__ float quad_max(float v) {
   v = fmaxf(v, __shfl_xor_sync(kFull, v, 1));
@@ -133,58 +159,68 @@ __device__ __forceinline__ void chunk_attn_mma_body(const ChunkAttnMmaArgs &a) {
   const int lo = p0 - p0 % a.chunk, kb0 = lo / kCmKeys * kCmKeys;
   const uint16_t *K = a.Kc + (size_t)g * a.D;
   const float *lb = a.LB + (size_t)h * a.lb_len;
+  // keys of a tile by asynchronous copies; its penalties (entry tid: distance p0 - k0 - 63 + tid, 127 used) wait
+  // in a register until the tile before is done
+  int slot = kb0 % a.cap;
+  float pen = 0.0f;
   auto fetch = [&](int k0, int b) {
-    load_keys<DP, 128>(ka + (uint32_t)(b * kCmKeys * LD) * 2, K, k0 % a.cap, KW, a.D);
-    const int d = p0 - k0 - 63 + tid;   // distance of entry tid (127 used)
-    lbw[b * 128 + tid] = lb[min(max(d, 0), a.lb_len - 1)] * kLog2e;
+    pen = __ldg(lb + min(max(p0 - k0 - 63 + tid, 0), a.lb_len - 1));
+    load_keys<DP, 128>(ka + (uint32_t)(b * kCmKeys * LD) * 2, K, slot, KW, a.D);
     cpa_commit();
+    slot += kCmKeys;
+    if (slot == a.cap) slot = 0;
   };
   fetch(kb0, 0);
+  lbw[tid] = pen * kLog2e;
   const float mul = a.scale * a.Temp[h] * kLog2e;
-  uint32_t q[DP / 16][4];
   float o[DP / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 #pragma unroll
   for (int d = 0; d < DP / 8; ++d)
 #pragma unroll
     for (int i = 0; i < 4; ++i) o[d][i] = 0.0f;
+  const uint32_t qw = qa + (uint32_t)((warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2;
   const int rw = warp * 16 + (lane >> 2);                 // this thread's rows rw and rw + 8
   const int pr[2] = {p0 + rw, p0 + rw + 8};
   const int cs[2] = {pr[0] - pr[0] % a.chunk, pr[1] - pr[1] % a.chunk};
   const int cs_last = p1 - p1 % a.chunk;
-  bool first = true;
   int b = 0;
   for (int k0 = kb0; k0 <= p1; k0 += kCmKeys) {
     const bool more = k0 + kCmKeys <= p1;
     if (more) fetch(k0 + kCmKeys, b ^ 1);
     if (more) cpa_wait<1>(); else cpa_wait<0>();
     __syncthreads();
-    if (first) {
-#pragma unroll
-      for (int kk = 0; kk < DP / 16; ++kk) ldm4(q[kk], qa + (uint32_t)((warp * 16 + (lane & 15)) * LD + kk * 16 + (lane >> 4) * 8) * 2);
-      first = false;
-    }
     float s[kCmKeys / 8][4];
     const uint32_t kt = ka + (uint32_t)(b * kCmKeys * LD) * 2;
-    scores<DP, kCmKeys>(s, q, kt, lane);
+    scores_smem<DP, kCmKeys>(s, qw, kt, lane);
     const bool whole = k0 + kCmKeys - 1 <= p0 && k0 >= cs_last;   // every row sees every key of the tile
     const float *lw = lbw + b * 128;
     float mx[2] = {m[0], m[1]};
+    const float *lr = lw + rw + 63 - (lane & 3) * 2;   // entry of (row, key): + 8 per row half, - key
+    if (whole) {
 #pragma unroll
-    for (int n = 0; n < kCmKeys / 8; ++n)
+      for (int n = 0; n < kCmKeys / 8; ++n)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int x = i >> 1, kc = n * 8 + (lane & 3) * 2 + (i & 1), key = k0 + kc;
-        float v = fmaf(s[n][i], mul, -lw[rw + 8 * x - kc + 63]);
-        if (!whole && (key > pr[x] || key < cs[x])) v = -INFINITY;
-        s[n][i] = v;
-        mx[x] = fmaxf(mx[x], v);
-      }
+        for (int i = 0; i < 4; ++i) {
+          s[n][i] = fmaf(s[n][i], mul, -lr[8 * (i >> 1) - n * 8 - (i & 1)]);
+          mx[i >> 1] = fmaxf(mx[i >> 1], s[n][i]);
+        }
+    } else {
+#pragma unroll
+      for (int n = 0; n < kCmKeys / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int x = i >> 1, key = k0 + n * 8 + (lane & 3) * 2 + (i & 1);
+          const float v = fmaf(s[n][i], mul, -lr[8 * x - n * 8 - (i & 1)]);
+          s[n][i] = key > pr[x] || key < cs[x] ? -INFINITY : v;
+          mx[x] = fmaxf(mx[x], s[n][i]);
+        }
+    }
     float corr[2], base[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       mx[x] = quad_max(mx[x]);
       base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
-      corr[x] = exp2f(m[x] - base[x]);
+      corr[x] = fast_exp2(m[x] - base[x]);
       m[x] = mx[x];
     }
     float sum[2] = {0.0f, 0.0f};
@@ -192,16 +228,19 @@ __device__ __forceinline__ void chunk_attn_mma_body(const ChunkAttnMmaArgs &a) {
     for (int n = 0; n < kCmKeys / 8; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        s[n][i] = exp2f(s[n][i] - base[i >> 1]);
+        s[n][i] = fast_exp2(s[n][i] - base[i >> 1]);
         sum[i >> 1] += s[n][i];
       }
 #pragma unroll
     for (int x = 0; x < 2; ++x) l[x] = fmaf(l[x], corr[x], sum[x]);
+    if (__any_sync(kFull, corr[0] != 1.0f || corr[1] != 1.0f)) {   // some row's maximum moved
 #pragma unroll
-    for (int d = 0; d < DP / 8; ++d)
+      for (int d = 0; d < DP / 8; ++d)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+        for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+    }
     values<DP, kCmKeys>(o, s, kt, lane);
+    if (more) lbw[(b ^ 1) * 128 + tid] = pen * kLog2e;
     __syncthreads();
     b ^= 1;
   }
@@ -361,14 +400,14 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
     for (int x = 0; x < 2; ++x) {
       mx[x] = quad_max(mx[x]);
       base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
-      corr[x] = exp2f(m[x] - base[x]);
+      corr[x] = fast_exp2(m[x] - base[x]);
       m[x] = mx[x];
     }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        s[n][i] = exp2f(s[n][i] - base[i >> 1]);
+        s[n][i] = fast_exp2(s[n][i] - base[i >> 1]);
         sum[i >> 1] += s[n][i];
       }
 #pragma unroll
@@ -407,7 +446,7 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
     float v = 0.0f, L = 0.0f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float f = exp2f(wm[w][hh] - M);
+      const float f = fast_exp2(wm[w][hh] - M);
       v = fmaf(os[(w * 16 + hh) * DP + d], f, v);
       L = fmaf(wl[w][hh], f, L);
     }
@@ -433,7 +472,7 @@ __device__ __forceinline__ void chunk_step_mma_body(const ChunkAttnStepMmaArgs &
   float *fac = os;   // [HG][kSmMaxSplits]
   for (int hh = warp; hh < HG; hh += 4) {
     const float2 ml = lane < active ? __ldcg(reinterpret_cast<const float2 *>(base_m) + lane * HG + hh) : make_float2(-INFINITY, 0.0f);
-    const float M = warp_max(ml.x), f = exp2f(ml.x - M), L = warp_tree_sum(ml.y * f);
+    const float M = warp_max(ml.x), f = fast_exp2(ml.x - M), L = warp_tree_sum(ml.y * f);
     if (lane < kSmMaxSplits) fac[hh * kSmMaxSplits + lane] = lane < active ? f / L : 0.0f;
   }
   __syncthreads();

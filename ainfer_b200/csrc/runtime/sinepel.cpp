@@ -508,7 +508,7 @@ struct Engine : RowEngine {
       hyper(k, sp, lw.sub[0].in, lw.sub[0].norm, &lw, &s, R, nullptr, true);
       linear(k, lw.qk, H, ldw, R, U, C, ACT_NONE, false);
       if (sp.one_sequence) {
-        const int per = std::max(1, std::min(16, R / 16));
+        const int per = std::max(1, std::min(8, R / 16));
         const int cblk = C % 4 == 0 && Qc % 4 == 0 && r.taps >= 2 && r.taps <= 4 ? 1024 : 256;   // channels of a block
         k.launch(f32 ? "ShortConvRowsF32" : "ShortConvRowsB16", (uint32_t)(((R + per - 1) / per) * ((C + cblk - 1) / cblk)), (const float *)U, lw.conv,
                  (const float *)s.conv, s.pend_conv, sp.ctrl, sp.seq, sp.first, (void *)Q, (void *)s.k, kv_stride, (int32_t)R, (int32_t)C,

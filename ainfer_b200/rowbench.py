@@ -112,3 +112,37 @@ def run(dev, names, hbm_gbs, bf16_tflops, steps=32):
             rows[name]["int4_hybrid_" + preset] = measure(dev, m, ctx, min(prompt, 4096), (16, 64), steps, runtime.Session.PERSISTENT)
             m.close()
     return rows
+
+
+def once(name, what):
+    """A few launches to capture: a prompt pass of 2048 rows, four decode steps at position 2000, or two
+    batched steps (what = the batch) at position 2000."""
+    from . import cuda_abi, runtime
+    dev = cuda_abi.Device(0)
+    m = open_model(dev, name)
+    ids = np.random.default_rng(0).integers(0, m.config["vocab"], 4096).astype(np.int32)
+    dev.sync()
+    if what == "prefill":
+        s = runtime.Session(m, 4096)
+        s.prefill(ids[:2048])
+    elif what == "decode":
+        s = runtime.Session(m, 4096)
+        s.generate(ids[:1], 4, start_pos=2000)
+    else:
+        s = runtime.BatchDecode(m, int(what), 2100)
+        s.set_inputs(ids[:int(what)], np.full(int(what), 2000, np.int32))
+        s.step()
+        s.step()
+    dev.sync()
+    s.close()
+    m.close()
+    dev.close()
+
+
+if __name__ == "__main__":
+    import argparse
+    ap = argparse.ArgumentParser(description=once.__doc__)
+    ap.add_argument("size", choices=sorted(SIZES))
+    ap.add_argument("what", help="prefill, decode or a batch size")
+    a = ap.parse_args()
+    once(a.size, a.what)
