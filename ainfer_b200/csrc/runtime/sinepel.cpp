@@ -211,7 +211,6 @@ int prepare(DeviceModel *m, std::string &err) {
   auto w = std::make_shared<RowWeights>();
   std::map<std::string, ainfer_kernel_t> kernels;
   KernelCalls k(dev, &kernels, &err);
-  const int W = c.hidden, S = c.streams;
   auto alloc = [&](size_t bytes) -> void * {
     void *p = nullptr;
     if (k.status) return nullptr;
@@ -258,7 +257,6 @@ int prepare(DeviceModel *m, std::string &err) {
     if (p && ainfer_memcpy_h2d(dev, p, v.data(), v.size() * 4) != AINFER_OK) k.fail(1, ainfer_last_error(dev));
     return p;
   };
-  (void)S;
   for (int L = 0; L < c.layers && !k.status; ++L) {
     const RowLayerConfig &r = c.row_layers[L];
     const std::string p = layer_name(L), x = p + "mix.";
@@ -307,7 +305,6 @@ int prepare(DeviceModel *m, std::string &err) {
     if (!k.status && ainfer_sync(dev, UINT64_MAX) != AINFER_OK) k.fail(1, ainfer_last_error(dev));
   }
   for (auto &kv : kernels) ainfer_kernel_release(kv.second);
-  (void)W;
   m->rows = w;
   return k.status;
 }
@@ -378,7 +375,7 @@ struct Engine : RowEngine {
     size_t off = 0;
     auto take = [&](size_t bytes) { const size_t o = off; off += (bytes + 255) / 256 * 256; return o; };
     std::vector<size_t> so, co, ko;
-    for (const RowLayerConfig &r : c.row_layers) { (void)r; so.push_back(take((size_t)nseq * 2 * W * 4)); }
+    for (int L = 0; L < c.layers; ++L) so.push_back(take((size_t)nseq * 2 * W * 4));
     conv_off = off;
     for (const RowLayerConfig &r : c.row_layers) co.push_back(take((size_t)nseq * r.taps * (r.heads + r.kv_heads) * r.dim * 4));
     k_off = off;

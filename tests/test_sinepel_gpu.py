@@ -75,7 +75,7 @@ def test_embedding_with_positions(dev, W, S):
 
 
 @pytest.mark.parametrize("out", ["f32", "b16"])
-@pytest.mark.parametrize("W,S,per", [(64, 4, 1), (192, 4, 3), (50, 3, 2), (37, 1, 4), (36, 2, 8), (40, 5, 3)])
+@pytest.mark.parametrize("W,S,per", [(64, 4, 1), (196, 4, 3), (50, 3, 2), (37, 1, 4), (36, 2, 8), (40, 5, 3)])
 def test_stream_update_read_norm_and_shift(dev, W, S, per, out):
     """Three sequences in one pass: rows 0..4 start at position 0, 5..6 continue (even and odd position),
     7 is alone."""
