@@ -1,6 +1,7 @@
 // Scalar arithmetic of the decode path, shared by device kernels and by the
 // host-side synthetic-model writer. Every transcendental is a fixed polynomial
-// over IEEE add/mul/fma, so host and device agree bit for bit. Build rules:
+// over IEEE add/mul/fma (exponential and logarithm: the single-precision polynomials of the Cephes
+// library by S. L. Moshier), so host and device agree bit for bit. Build rules:
 // nvcc -fmad=false and g++ -ffp-contract=off (a fused multiply-add happens only
 // where fmaf is written); no fast-math.
 //
