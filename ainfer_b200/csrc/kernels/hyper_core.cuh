@@ -5,7 +5,7 @@
 // sublayer and the read of the next touch the same elements, so they run as one step per element:
 // the S values are loaded once, updated, stored once, and the next sublayer's u falls out.
 #pragma once
-#include "common.cuh"
+#include "row_types.cuh"
 
 namespace ainfer {
 
@@ -87,22 +87,6 @@ __device__ __forceinline__ float stream_step_n(const float *src, const float *y,
     u = fmaf(c.in[t], a, u);
   }
   return u;
-}
-
-// Block sum in fp32 (any number of warps up to 32); every thread gets the total. red: 33 floats.
-__device__ __forceinline__ float block_sum(float v, float *red) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
-  v = warp_tree_sum(v);
-  __syncthreads();   // earlier readers of red are done
-  if (lane == 0) red[warp] = v;
-  __syncthreads();
-  if (warp == 0) {
-    float t = lane < nw ? red[lane] : 0.0f;
-    t = warp_tree_sum(t);
-    if (lane == 0) red[32] = t;
-  }
-  __syncthreads();
-  return red[32];
 }
 
 // How a row's elements are dealt to threads: four consecutive ones each, or one.

@@ -15,19 +15,6 @@
 
 namespace ainfer {
 
-template <typename T>
-__device__ __forceinline__ float ld_val(const T *p);
-template <>
-__device__ __forceinline__ float ld_val<float>(const float *p) { return *p; }
-template <>
-__device__ __forceinline__ float ld_val<uint16_t>(const uint16_t *p) { return bf16_to_f32(*p); }
-template <typename T>
-__device__ __forceinline__ void st_val(T *p, float v);
-template <>
-__device__ __forceinline__ void st_val<float>(float *p, float v) { *p = v; }
-template <>
-__device__ __forceinline__ void st_val<uint16_t>(uint16_t *p, float v) { *p = f32_to_bf16(v); }
-
 // ------------------------------------------------------- ShortConvRows ---
 struct ShortConvRowsArgs {
   const float *U;          // [rows][ldu] projections (q channels, then k channels)
@@ -41,15 +28,6 @@ struct ShortConvRowsArgs {
   int32_t rows, C, Qc, taps, cap, ldu, per;   // per: rows of a block
 };
 // Four channels per thread, TAPS known, the last TAPS - 1 projections in registers.
-template <typename T>
-__device__ __forceinline__ void store4(T *p, const float4 v);
-template <>
-__device__ __forceinline__ void store4<float>(float *p, const float4 v) { *reinterpret_cast<float4 *>(p) = v; }
-template <>
-__device__ __forceinline__ void store4<uint16_t>(uint16_t *p, const float4 v) {
-  *reinterpret_cast<uint2 *>(p) = make_uint2((uint32_t)f32_to_bf16(v.x) | ((uint32_t)f32_to_bf16(v.y) << 16),
-                                             (uint32_t)f32_to_bf16(v.z) | ((uint32_t)f32_to_bf16(v.w) << 16));
-}
 template <typename T, int TAPS>
 __device__ __forceinline__ void short_conv4_body(const ShortConvRowsArgs &a) {
   const int cb = (a.C + 1023) / 1024;
@@ -84,8 +62,8 @@ __device__ __forceinline__ void short_conv4_body(const ShortConvRowsArgs &a) {
     }
     if (TAPS > 1 && (r + TAPS - 1 >= a.rows || a.First[r + TAPS - 1] != f))   // among the sequence's last TAPS - 1 rows
       *reinterpret_cast<float4 *>(a.Pend + ((size_t)seq * TAPS + pos % TAPS) * a.C + c) = win[TAPS - 1];
-    if (c < a.Qc) store4(reinterpret_cast<T *>(a.Q) + (size_t)r * a.Qc + c, y);
-    else store4(reinterpret_cast<T *>(a.Kc) + (size_t)seq * a.kv_stride + (size_t)(pos % a.cap) * Kn + (c - a.Qc), y);
+    if (c < a.Qc) st_val4(reinterpret_cast<T *>(a.Q) + (size_t)r * a.Qc + c, y);
+    else st_val4(reinterpret_cast<T *>(a.Kc) + (size_t)seq * a.kv_stride + (size_t)(pos % a.cap) * Kn + (c - a.Qc), y);
   }
 }
 // grid = ceil(rows / per) x ceil(C / 1024) with whole quads of channels and 2..4 taps, else x ceil(C / 256)

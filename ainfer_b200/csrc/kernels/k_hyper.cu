@@ -56,13 +56,6 @@ struct HyperNormRowsArgs {
 };
 
 template <typename T>
-__device__ __forceinline__ void store_val(T *p, float v);
-template <>
-__device__ __forceinline__ void store_val<float>(float *p, float v) { *p = v; }
-template <>
-__device__ __forceinline__ void store_val<uint16_t>(uint16_t *p, float v) { *p = f32_to_bf16(v); }
-
-template <typename T>
 __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
   extern __shared__ __align__(16) float hy_smem[];   // [2][W rounded to 4]
   __shared__ StreamCoef coef;
@@ -114,14 +107,14 @@ __device__ __forceinline__ void hyper_norm_body(const HyperNormRowsArgs &a) {
     norm_row(r, true, cur);
     T *h = H + (size_t)r * a.ldh;
     if (!a.Shift) {
-      each([&](int w) { store_val(h + w, cur[w]); });
+      each([&](int w) { st_val(h + w, cur[w]); });
       continue;
     }
     if (fr == r || !have_prev) {
       const float *st = a.State + ((size_t)seq * 2 + ((pos - 1) & 1)) * W;
       each([&](int w) { prev[w] = pos > 0 ? st[w] : 0.0f; });
     }
-    each([&](int w) { store_val(h + w, fmaf(prev[w] - cur[w], a.Shift[w], cur[w])); });
+    each([&](int w) { st_val(h + w, fmaf(prev[w] - cur[w], a.Shift[w], cur[w])); });
     if (fn == r + 1) {
       float *pd = a.Pend + (size_t)seq * W;
       each([&](int w) { pd[w] = cur[w]; });
