@@ -8,6 +8,9 @@
 // products, warps 4..7 read the accumulators (a lane = one output feature, so a warp stores 32
 // consecutive features of a row at a time).
 //
+// LinearTcGrouped: the same over the rows of a mixture's experts, sorted by expert: W [E][N][K] as one
+// map of E N rows, tiles (expert, first row, rows) and their number from memory.
+//
 // LinearTcSplit2 / 4 / 8, for few tiles: a cluster of that many blocks shares one tile (nt <= 128), each
 // block a part of K. The blocks exchange their fp32 partials through distributed shared memory, every
 // block summing its share of the rows in block order.
@@ -29,6 +32,15 @@ struct LinearTcArgs {
   void *Y;               // [rows][ldy]
   int32_t rows, N, K, nt, ldy, act, out16;
   float cap;
+};
+
+struct LinearTcGroupedArgs {
+  CUtensorMap Wm;        // [E N][K], box 64 x 128
+  CUtensorMap Xm;        // [places][K], box 64 x nt
+  void *Y;               // [places][ldy]
+  const int4 *Tiles;     // (expert, first place, places <= nt, 0)
+  const int32_t *Count;  // tiles
+  int32_t N, K, nt, ldy, act, out16;
 };
 
 constexpr int kLtThreads = 256, kLtBudget = 200 * 1024;
@@ -116,7 +128,26 @@ __device__ __forceinline__ bool lt_wait(LtShared *s, unsigned long long *b, uint
   return false;
 }
 
-__global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant__ LinearTcArgs a) {
+// What a tile is: its first row of the weights' map, first output feature, first row and rows.
+struct LtTile { int w0, n0, r0, nr; };
+__device__ __forceinline__ LtTile lt_tile(const LinearTcArgs &a, int u, int n_tiles) {
+  const int n0 = (u % n_tiles) * 128, r0 = (u / n_tiles) * a.nt;
+  return LtTile{n0, n0, r0, min(a.nt, a.rows - r0)};
+}
+__device__ __forceinline__ LtTile lt_tile(const LinearTcGroupedArgs &a, int u, int n_tiles) {
+  const int4 t = a.Tiles[u / n_tiles];
+  const int n0 = (u % n_tiles) * 128;
+  return LtTile{t.x * a.N + n0, n0, t.y, t.z};
+}
+__device__ __forceinline__ int lt_tiles(const LinearTcArgs &a, int n_tiles) { return n_tiles * ((a.rows + a.nt - 1) / a.nt); }
+__device__ __forceinline__ int lt_tiles(const LinearTcGroupedArgs &a, int n_tiles) { return n_tiles * a.Count[0]; }
+__device__ __forceinline__ float lt_bias(const LinearTcArgs &a, int n) { return a.Bias && n < a.N ? a.Bias[n] : 0.0f; }
+__device__ __forceinline__ float lt_bias(const LinearTcGroupedArgs &, int) { return 0.0f; }
+__device__ __forceinline__ float lt_cap(const LinearTcArgs &a) { return a.cap; }
+__device__ __forceinline__ float lt_cap(const LinearTcGroupedArgs &) { return 0.0f; }
+
+template <typename Args>
+__device__ __forceinline__ void linear_tc_body(const Args &a) {
   extern __shared__ __align__(1024) unsigned char lt_smem_raw[];
   __shared__ LtShared sh;
   pdl_launch_dependents();
@@ -124,7 +155,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
   const uint32_t base = (smem_addr(lt_smem_raw) + 1023u) & ~1023u;
   const int nt = a.nt, nst = (int)lt_stages(nt);
   const uint32_t stage_bytes = lt_stage_bytes(nt);
-  const int n_tiles = (a.N + 127) / 128, r_tiles = (a.rows + nt - 1) / nt, tiles = n_tiles * r_tiles;
+  const int n_tiles = (a.N + 127) / 128;
   const int kb = (a.K + 63) / 64;
   uint32_t cols = 32;
   while (cols < 2u * (uint32_t)nt) cols <<= 1;
@@ -146,18 +177,19 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
   const uint32_t tmem = sh.tmem;
   pdl_wait();
+  const int tiles = lt_tiles(a, n_tiles);
 
   if (warp == 0 && lane == 0) {
     // ---- copies ----
     uint32_t st = 0, ph = 1, issued = 0;
     for (int u = blockIdx.x; u < tiles; u += gridDim.x) {
-      const int n0 = (u % n_tiles) * 128, r0 = (u / n_tiles) * nt;
+      const LtTile t = lt_tile(a, u, n_tiles);
       for (int k = 0; k < kb; ++k) {
         if (!lt_wait(&sh, &sh.empty[st], ph)) break;
         const uint32_t dst = base + st * stage_bytes, bar = smem_addr(&sh.full[st]);
         mbar_arrive_expect(&sh.full[st], stage_bytes);
-        lt_tma(dst, &a.Wm, bar, k * 64, n0);
-        lt_tma(dst + 128u * 128u, &a.Xm, bar, k * 64, r0);
+        lt_tma(dst, &a.Wm, bar, k * 64, t.w0);
+        lt_tma(dst + 128u * 128u, &a.Xm, bar, k * 64, t.r0);
         ++issued;
         if (++st == (uint32_t)nst) { st = 0; ph ^= 1; }
       }
@@ -202,24 +234,25 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
     const int lw = (warp & 3) * 32 + lane;
     uint32_t buf = 0, ph = 0;
     for (int u = blockIdx.x; u < tiles; u += gridDim.x) {
-      const int n = (u % n_tiles) * 128 + lw, r0 = (u / n_tiles) * nt, nr = min(nt, a.rows - r0);
-      const float bias = a.Bias && n < a.N ? a.Bias[n] : 0.0f;
+      const LtTile t = lt_tile(a, u, n_tiles);
+      const int n = t.n0 + lw, nr = t.nr;
+      const float bias = lt_bias(a, n), cap = lt_cap(a);
       lt_wait(&sh, &sh.acc_full[buf], ph);
       __syncwarp();
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t taddr = tmem + buf * (uint32_t)nt + ((uint32_t)((warp & 3) * 32) << 16);
       const bool in = n < a.N;
-      const size_t o = (size_t)r0 * a.ldy + n;
+      const size_t o = (size_t)t.r0 * a.ldy + n;
       if (a.out16) {
         __nv_bfloat16 *y = reinterpret_cast<__nv_bfloat16 *>(a.Y) + o;
-        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, a.cap, in);
-        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, a.cap, in);
-        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, cap, in);
+        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, cap, in);
+        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, cap, in);
       } else {
         float *y = reinterpret_cast<float *>(a.Y) + o;
-        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, a.cap, in);
-        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, a.cap, in);
-        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, a.cap, in);
+        if (a.act == 1) lt_epilogue<1>(taddr, nr, y, a.ldy, bias, cap, in);
+        else if (a.act == 2) lt_epilogue<2>(taddr, nr, y, a.ldy, bias, cap, in);
+        else lt_epilogue<0>(taddr, nr, y, a.ldy, bias, cap, in);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       mbar_arrive(&sh.acc_empty[buf]);
@@ -231,8 +264,14 @@ __global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant_
   __syncthreads();
   if (warp == 2) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(cols) : "memory");
 }
+__global__ void __launch_bounds__(kLtThreads, 1) LinearTc(const __grid_constant__ LinearTcArgs a) { linear_tc_body(a); }
+__global__ void __launch_bounds__(kLtThreads, 1) LinearTcGrouped(const __grid_constant__ LinearTcGroupedArgs a) { linear_tc_body(a); }
 static uint32_t linear_tc_smem(const void *args) {
   const int nt = ((const LinearTcArgs *)args)->nt;
+  return lt_stages(nt) * lt_stage_bytes(nt) + 1024;
+}
+static uint32_t linear_tc_grouped_smem(const void *args) {
+  const int nt = ((const LinearTcGroupedArgs *)args)->nt;
   return lt_stages(nt) * lt_stage_bytes(nt) + 1024;
 }
 
@@ -386,6 +425,12 @@ AINFER_REGISTER(LinearTcSplit4, LinearTcArgs, kLtThreads, 4, 0, linear_tc_split_
 AINFER_REGISTER(LinearTcSplit8, LinearTcArgs, kLtThreads, 8, 0, linear_tc_split_smem, LT_FIELDS);
 #undef F
 
+#define F(f) AINFER_ARG(LinearTcGroupedArgs, f)
+AINFER_REGISTER(LinearTcGrouped, LinearTcGroupedArgs, kLtThreads, 0, 0, linear_tc_grouped_smem, F(Wm), F(Xm), F(Y), F(Tiles), F(Count), F(N), F(K),
+                F(nt), F(ldy), F(act), F(out16));
+#undef F
+
+AINFER_EARLY_LAUNCH(LinearTcGrouped);
 AINFER_EARLY_LAUNCH(LinearTc);
 AINFER_EARLY_LAUNCH(LinearTcSplit2);
 AINFER_EARLY_LAUNCH(LinearTcSplit4);

@@ -13,6 +13,7 @@ namespace ainfer {
 
 struct Session;
 struct Json;
+struct RowEngine;
 
 // Configuration and weights.
 struct ModelArch {
@@ -24,6 +25,7 @@ struct ModelArch {
   void (*plan)(const ModelConfig &c, Container &dir, std::vector<SynthSpec> &specs);
   int (*check_directory)(const Container &dir, const ModelConfig &c, std::string &err);
   int (*prepare)(DeviceModel *m, std::string &err);                      // after the weights are on the device
+  RowEngine *(*engine)();                                                // null: the block executor of the INT4 hybrid
 };
 const ModelArch *model_arch(const std::string &name);                    // null: unknown
 
@@ -38,6 +40,8 @@ struct RowSpan {
 };
 struct RowEngine {                // state of `nseq` sequences plus the buffers of a pass of `rows_cap` rows
   virtual ~RowEngine() {}
+  // max_ctx: positions a sequence may reach; f32: activations and cache in 32-bit. 0, 1 (device) or 2 (usage).
+  virtual int create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, std::string &err) = 0;
   virtual void emit(KernelCalls &k, const RowSpan &span) = 0;
   virtual int reset(std::string &err) = 0;
   virtual bool buffer(const std::string &which, void **dptr, uint64_t *bytes) = 0;
@@ -48,12 +52,13 @@ struct RowEngine {                // state of `nseq` sequences plus the buffers 
   virtual void record_head(KernelCalls &k, float *logits) = 0;
   int rows_cap = 0;
 };
-// Creates the row engine of an architecture that has one. max_ctx: positions a sequence may reach;
-// f32: activations and cache in 32-bit. Returns 0, 1 (device) or 2 (usage).
+// Makes and creates the row engine of a model's architecture (usage error where it has none).
 int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err);
 
 bool sinepel_preset(const std::string &name, ModelConfig &c);   // "sinepel-tiny", "sinepel-small"
+bool robopel_preset(const std::string &name, ModelConfig &c);   // "robopel-tiny", "robopel-small"
 const ModelArch *sinepel_model_arch();
+const ModelArch *robopel_model_arch();
 const ModelArch *int4_hybrid_model_arch();
 
 }  // namespace ainfer

@@ -112,7 +112,7 @@ int BatchDecode::create(DeviceModel *model, const void *id128, int rank, int wor
 int BatchDecode::create_rows(int owned, bool f32) {
   const ModelConfig &c = m->cfg;
   n = owned;
-  max_ctx = std::min(max_ctx, c.max_positions);
+  max_ctx = c.positions(max_ctx);
   int r = row_engine_create(m, n, max_ctx, n, f32, &rows, err);
   if (r) return r;
   int32_t *seq = nullptr;   // row = sequence = first row of its sequence = row whose logits are wanted

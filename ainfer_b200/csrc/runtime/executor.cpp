@@ -481,7 +481,7 @@ int session_create(DeviceModel *m, int max_ctx, int flags, Session **out, std::s
   const bool row_arch = m->rows != nullptr;
   if (row_arch) {
     // learned positions bound the context; the persistent step is the INT4 hybrid's, here a token is always a recorded list
-    s->max_ctx = max_ctx = std::min(max_ctx, c.max_positions);
+    s->max_ctx = max_ctx = c.positions(max_ctx);
     s->flags = flags &= ~(SESSION_PERSISTENT | SESSION_STAGE_CLOCK);
     const int e = row_engine_create(m, 1, max_ctx, std::min(max_ctx, kRowEnginePassRows), (flags & SESSION_F32) != 0, &s->rows, s->err);
     if (e) return fail(e);

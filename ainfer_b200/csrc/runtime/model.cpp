@@ -21,7 +21,7 @@ std::string layer_prefix(int L) { return "model.language_model.layers." + std::t
 
 // ----------------------------------------------------------- registry ---
 const ModelArch *model_arch(const std::string &name) {
-  const ModelArch *row[] = {sinepel_model_arch()};
+  const ModelArch *row[] = {sinepel_model_arch(), robopel_model_arch()};
   for (const ModelArch *a : row)
     if (name == a->name) return a;
   return nullptr;
@@ -35,6 +35,17 @@ std::string ModelConfig::to_json() const { return arch_of(*this).to_json(*this);
 bool ModelConfig::check(std::string &err) const { return arch_of(*this).check(*this, err); }
 void build_plan(const ModelConfig &cfg, Container &c, std::vector<SynthSpec> &specs) { arch_of(cfg).plan(cfg, c, specs); }
 int check_directory_shapes(const Container &dir, const ModelConfig &cfg, std::string &err) { return arch_of(cfg).check_directory(dir, cfg, err); }
+
+int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err) {
+  *out = nullptr;
+  const ModelArch &a = arch_of(m->cfg);
+  if (!m->rows || !a.engine) { err = "usage: this architecture has no row engine"; return 2; }
+  RowEngine *e = a.engine();
+  const int r = e->create(m, nseq, max_ctx, rows_cap, f32, err);
+  if (r) { delete e; return r; }
+  *out = e;
+  return 0;
+}
 
 // ------------------------------------------------------------- config ---
 static std::string int4_to_json(const ModelConfig &c) {
@@ -161,7 +172,7 @@ bool preset_config(const std::string &name, ModelConfig &c) {
     std::string js, err;
     return read_text(name.substr(7), js) && ModelConfig::from_json(js, c, err);
   }
-  if (sinepel_preset(name, c)) return true;
+  if (sinepel_preset(name, c) || robopel_preset(name, c)) return true;
   c = ModelConfig();
   if (name == "tiny") {
     c.hidden = 256; c.layers = 2; c.layer_types = "LA"; c.vocab = 512;
@@ -521,7 +532,7 @@ static int build_mirrors(DeviceModel *m, std::string &err) {
 }
 
 static const ModelArch kInt4Hybrid = {"int4 hybrid", true,       nullptr,   int4_to_json,
-                                      int4_check,    int4_plan,  int4_check_directory, build_mirrors};
+                                      int4_check,    int4_plan,  int4_check_directory, build_mirrors, nullptr};
 const ModelArch *int4_hybrid_model_arch() { return &kInt4Hybrid; }
 
 int model_ensure_rope(DeviceModel *m, int max_ctx, std::string &err) {

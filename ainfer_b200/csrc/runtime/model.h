@@ -16,13 +16,34 @@
 
 namespace ainfer {
 
-// One layer of an architecture whose layers carry their own sizes: attention over keys that are also
-// the values, with a short convolution, inside chunks of positions, and a dense feed-forward.
+// Rotary positions: `dims` leading dimensions of a head, in pairs; scaled: long wavelengths slowed by
+// `factor`, with a linear transition between original / high and original / low.
+struct RotaryConfig {
+  int dims = 0;
+  double base = 10000.0;
+  bool scaled = false;
+  double factor = 1.0, low = 1.0, high = 4.0, original = 0.0;
+};
+// One layer of an architecture whose layers carry their own sizes. Each architecture uses the fields of
+// the mechanisms it has.
 struct RowLayerConfig {
-  int heads = 0, kv_heads = 0, dim = 0, taps = 1;
+  enum Mixer { ATTENTION, MINGRU };
+  int mixer = ATTENTION;
+  // attention
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+  int taps = 1;        // short convolution
   int chunk = 0;       // positions per chunk (0: one chunk)
+  int window = 0;      // tokens a row sees (0: all)
+  int pool = 0;        // tokens of a pooled block before the window (0: none)
+  int kv_from = -1;    // the layer whose keys and values this one reads (-1: its own)
   double scale = 1.0;  // of the scores
-  int ff = 0;          // feed-forward size (0: none)
+  double softcap = 0;  // of the scores (0: none)
+  RotaryConfig rot;
+  // recurrence
+  int width = 0;
+  // feed-forward
+  int ff = 0;          // size (0: none), of an expert where there are experts
+  int experts = 0, identity = 0, top = 0;
 };
 
 struct ModelConfig {
@@ -35,9 +56,10 @@ struct ModelConfig {
   int experts = 0, top_k = 0, shared_experts = 1, expert_inter = 0;
   int mtp_layers = 0;
   double rms_eps = 1e-6;
-  // architectures of residual streams (hidden, layers, vocab and rms_eps are shared)
+  // architectures whose layers carry their own sizes (hidden, layers, vocab and rms_eps are shared)
   std::vector<RowLayerConfig> row_layers;
-  int streams = 1, max_positions = 0;
+  int streams = 1, max_positions = 0;   // max_positions 0: no limit
+  int positions(int wanted) const { return max_positions > 0 && max_positions < wanted ? max_positions : wanted; }
   double embed_scale = 1.0, logit_softcap = 0.0;
   bool int4_weights() const { return row_layers.empty(); }
   int conv_dim() const { return (2 * lin_k_heads + lin_v_heads) * lin_head_dim; }
@@ -81,7 +103,9 @@ struct DeviceTensor {
   void *scales = nullptr;  // device address of the scales (INT4) or null
 };
 
-struct RowWeights;   // prepared weights of architectures with a row engine
+struct RowWeights {   // prepared weights of an architecture with a row engine
+  virtual ~RowWeights() {}
+};
 
 // Device-resident model.
 struct DeviceModel {

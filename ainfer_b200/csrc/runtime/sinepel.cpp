@@ -11,8 +11,8 @@
 #include <cmath>
 #include <cstring>
 
-#include "arch.h"
 #include "json.h"
+#include "row_engine.h"
 #include "../common/detmath.h"
 
 namespace ainfer {
@@ -55,27 +55,19 @@ bool parse(const Json &js, ModelConfig &c, std::string &err) {
   return true;
 }
 
-std::string num(double v) {
-  char b[40];
-  std::snprintf(b, sizeof b, "%.17g", v);
-  return b;
-}
-
 std::string to_json(const ModelConfig &c) {
-  std::string s = "{\"architecture\":\"Sinepel\",\"embedding\":{\"scale\":" + num(c.embed_scale) + "},\"layers\":[";
+  std::string s = "{\"architecture\":\"Sinepel\",\"embedding\":{\"scale\":" + json_num(c.embed_scale) + "},\"layers\":[";
   for (size_t i = 0; i < c.row_layers.size(); ++i) {
     const RowLayerConfig &r = c.row_layers[i];
     s += (i ? "," : "") + std::string("{\"mixer\":{\"conv\":") + std::to_string(r.taps) + ",\"dim\":" + std::to_string(r.dim) +
          ",\"heads\":" + std::to_string(r.heads) + ",\"kv_heads\":" + std::to_string(r.kv_heads) + ",\"mask\":{\"size\":" +
-         std::to_string(r.chunk) + "},\"scale\":" + num(r.scale) + ",\"vdim\":" + std::to_string(r.dim) + "},\"mlp\":" +
+         std::to_string(r.chunk) + "},\"scale\":" + json_num(r.scale) + ",\"vdim\":" + std::to_string(r.dim) + "},\"mlp\":" +
          (r.ff ? "{\"ff\":" + std::to_string(r.ff) + ",\"kind\":\"dense\"}" : std::string("null")) + ",\"type\":\"attention\"}";
   }
-  return s + "],\"logit_softcap\":" + num(c.logit_softcap) + ",\"max_positions\":" + std::to_string(c.max_positions) +
-         ",\"norm\":{\"eps\":" + num(c.rms_eps) + "},\"streams\":" + std::to_string(c.streams) + ",\"vocab\":" + std::to_string(c.vocab) +
+  return s + "],\"logit_softcap\":" + json_num(c.logit_softcap) + ",\"max_positions\":" + std::to_string(c.max_positions) +
+         ",\"norm\":{\"eps\":" + json_num(c.rms_eps) + "},\"streams\":" + std::to_string(c.streams) + ",\"vocab\":" + std::to_string(c.vocab) +
          ",\"width\":" + std::to_string(c.hidden) + "}";
 }
-
-int round_up(int v, int m) { return (v + m - 1) / m * m; }
 
 bool check(const ModelConfig &c, std::string &err) {
   auto bad = [&](const std::string &m) { err = "unsupported architecture: " + m; return false; };
@@ -99,12 +91,9 @@ bool check(const ModelConfig &c, std::string &err) {
   return true;
 }
 
-std::string layer_name(int L) { return "l" + std::to_string(L) + "."; }
-
 // Every tensor with its shape, in storage order (q directly before k: one matrix when rows align).
-struct Named { std::string name; std::vector<uint64_t> shape; float std_, constant; };
-std::vector<Named> tensors(const ModelConfig &c) {
-  std::vector<Named> t;
+std::vector<RowTensor> tensors(const ModelConfig &c) {
+  std::vector<RowTensor> t;
   const uint64_t W = c.hidden, S = c.streams, V = c.vocab;
   auto add = [&](const std::string &n, std::vector<uint64_t> sh, float sd, float cst) { t.push_back({n, sh, sd, cst}); };
   add("embed", {V, W}, 0.5f, 0);
@@ -143,52 +132,12 @@ std::vector<Named> tensors(const ModelConfig &c) {
   return t;
 }
 
-void plan(const ModelConfig &c, Container &dir, std::vector<SynthSpec> &specs) {
-  dir = Container();
-  specs.clear();
-  for (const Named &n : tensors(c)) {
-    TensorEntry e;
-    e.name = n.name;
-    e.ndim = (int)n.shape.size();
-    for (int i = 0; i < e.ndim; ++i) e.shape[i] = n.shape[i];
-    e.logical = e.storage = DT_BF16;
-    e.d_bytes = e.numel() * 2;
-    dir.index[e.name] = dir.entries.size();
-    dir.entries.push_back(e);
-    SynthSpec sp;
-    sp.std_ = n.std_;
-    sp.constant = n.constant;
-    specs.push_back(sp);
-  }
-  dir.identity_json =
-      "{\"converter\":\"ainfer_b200 synthetic writer\",\"converter_version\":\"1.0\",\"created_date\":\"1970-01-01\",\"source_repo\":"
-      "\"synthetic\",\"source_revision\":\"0000000000000000000000000000000000000000\",\"source_total_bytes\":0}";
-  dir.arch_json = to_json(c);
-  dir.tokenizer_json = "{\"format\":\"none\",\"vocab_size\":" + std::to_string(c.vocab) + "}";
-  dir.policy_json = "{\"default\":\"BF16\"}";
-  container_layout(dir);
-}
-
-int check_directory(const Container &dir, const ModelConfig &c, std::string &err) {
-  for (const Named &n : tensors(c)) {
-    const TensorEntry *e = dir.find(n.name);
-    if (!e) { err = "missing " + n.name; return 1; }
-    if (e->storage != DT_BF16) { err = "unexpected storage of " + n.name; return 2; }
-    bool same = e->ndim == (int)n.shape.size();
-    for (int i = 0; same && i < e->ndim; ++i) same = e->shape[i] == n.shape[i];
-    if (!same) { err = "unexpected shape of " + n.name; return 2; }
-  }
-  return 0;
-}
+void plan(const ModelConfig &c, Container &dir, std::vector<SynthSpec> &specs) { plan_row_tensors(tensors(c), to_json(c), c.vocab, dir, specs); }
+int check_directory(const Container &dir, const ModelConfig &c, std::string &err) { return check_row_tensors(dir, tensors(c), err); }
 
 }  // namespace
 
 // ------------------------------------------------------------- prepared weights ---
-struct RowMatrix {           // bf16 rows of ldw values (ldw a multiple of 8, zero padding)
-  const uint16_t *w = nullptr;
-  const float *bias = nullptr;
-  int N = 0, K = 0, ldw = 0;
-};
 struct RowSublayer { const float *in, *out, *mix, *norm; };
 struct RowLayerWeights {
   RowMatrix qk, o, up, down;
@@ -196,7 +145,7 @@ struct RowLayerWeights {
   const float *shift, *conv /* [taps][C] */, *temp, *lb /* [H][lb_len] */;
   int lb_len;
 };
-struct RowWeights {
+struct SinepelWeights : RowWeights {
   std::vector<RowLayerWeights> L;
   RowMatrix head;
   const float *final_norm = nullptr;
@@ -207,114 +156,60 @@ namespace {
 
 int prepare(DeviceModel *m, std::string &err) {
   const ModelConfig &c = m->cfg;
-  ainfer_device_t dev = m->dev;
-  auto w = std::make_shared<RowWeights>();
-  std::map<std::string, ainfer_kernel_t> kernels;
-  KernelCalls k(dev, &kernels, &err);
-  auto alloc = [&](size_t bytes) -> void * {
-    void *p = nullptr;
-    if (k.status) return nullptr;
-    if (ainfer_mem_alloc(dev, std::max<size_t>(bytes, 16), 256, &p) != AINFER_OK) { k.fail(1, ainfer_last_error(dev)); return nullptr; }
-    m->owned.push_back(p);
-    return p;
-  };
-  auto widen = [&](const std::string &name) -> const float * {
-    DeviceTensor t = m->tensor(name);
-    const uint64_t n = t.entry->numel();
-    float *p = (float *)alloc(n * 4);
-    if (p) k.launch("WidenBf16", (uint32_t)std::min<uint64_t>((n + 255) / 256, 1024), p, (const void *)t.data, n);
-    return p;
-  };
-  // rows of one or two tensors as one matrix; copied only when rows need padding or the two do not adjoin
-  auto matrix = [&](const std::string &a, const std::string &b) {
-    DeviceTensor ta = m->tensor(a), tb = b.empty() ? DeviceTensor() : m->tensor(b);
-    RowMatrix r;
-    const int Na = (int)ta.entry->shape[0], Nb = b.empty() ? 0 : (int)tb.entry->shape[0];
-    r.K = (int)ta.entry->shape[1];
-    r.N = Na + Nb;
-    r.ldw = round_up(r.K, 8);
-    if (r.ldw == r.K && (b.empty() || (char *)ta.data + (size_t)Na * r.K * 2 == (char *)tb.data)) {
-      r.w = (const uint16_t *)ta.data;
-      return r;
-    }
-    uint16_t *p = (uint16_t *)alloc((size_t)r.N * r.ldw * 2);
-    r.w = p;
-    if (!p) return r;
-    k.launch("PackRowsBf16", (uint32_t)std::min(Na, 4096), p, (const uint16_t *)ta.data, (int32_t)Na, (int32_t)r.K, (int32_t)r.ldw);
-    if (Nb)
-      k.launch("PackRowsBf16", (uint32_t)std::min(Nb, 4096), p + (size_t)Na * r.ldw, (const uint16_t *)tb.data, (int32_t)Nb, (int32_t)r.K,
-               (int32_t)r.ldw);
-    return r;
-  };
-  auto host_bf16 = [&](const std::string &name) {
-    DeviceTensor t = m->tensor(name);
-    std::vector<uint16_t> v(t.entry->numel());
-    if (ainfer_memcpy_d2h(dev, v.data(), t.data, v.size() * 2) != AINFER_OK) k.fail(1, ainfer_last_error(dev));
-    return v;
-  };
-  auto upload = [&](const std::vector<float> &v) -> const float * {
-    float *p = (float *)alloc(v.size() * 4);
-    if (p && ainfer_memcpy_h2d(dev, p, v.data(), v.size() * 4) != AINFER_OK) k.fail(1, ainfer_last_error(dev));
-    return p;
-  };
+  auto w = std::make_shared<SinepelWeights>();
+  RowLoader k(m, &err);
   for (int L = 0; L < c.layers && !k.status; ++L) {
     const RowLayerConfig &r = c.row_layers[L];
     const std::string p = layer_name(L), x = p + "mix.";
     const int Q = r.heads * r.dim, Kn = r.kv_heads * r.dim, C = Q + Kn;
     RowLayerWeights lw{};
-    lw.qk = matrix(x + "q", x + "k");
+    lw.qk = k.stack({x + "q", x + "k"});
     std::vector<float> bias((size_t)C), conv((size_t)C * r.taps);
     int at = 0;
     for (const char *n : {"q", "k"}) {
-      const auto b = host_bf16(x + n + ".b"), cv = host_bf16(x + n + std::string(".conv"));
+      const auto b = k.host(x + n + ".b"), cv = k.host(x + n + std::string(".conv"));
       for (size_t i = 0; i < b.size(); ++i) {
         bias[(size_t)at + i] = bf16_to_f32(b[i]);
         for (int j = 0; j < r.taps; ++j) conv[(size_t)j * C + at + i] = bf16_to_f32(cv[i * r.taps + j]);
       }
       at += (int)b.size();
     }
-    lw.qk.bias = upload(bias);
-    lw.conv = upload(conv);
-    lw.o = matrix(x + "o", "");
-    lw.temp = widen(x + "temp");
+    lw.qk.bias = k.upload(bias);
+    lw.conv = k.upload(conv);
+    lw.o = k.stack({x + "o"});
+    lw.temp = k.widen(x + "temp");
     // distances that occur: below the chunk length and below the number of positions
     lw.lb_len = r.chunk ? std::min(r.chunk, c.max_positions) : c.max_positions;
-    float *lb = (float *)alloc((size_t)r.heads * lw.lb_len * 4);
-    const float *r1 = widen(x + "r1"), *r2 = widen(x + "r2");
+    float *lb = (float *)k.alloc((size_t)r.heads * lw.lb_len * 4);
+    const float *r1 = k.widen(x + "r1"), *r2 = k.widen(x + "r2");
     if (!k.status) k.launch("LogDistanceTable", 1024, lb, r1, r2, (int32_t)r.heads, (int32_t)lw.lb_len);
     lw.lb = lb;
-    lw.shift = widen(p + "shift");
+    lw.shift = k.widen(p + "shift");
     for (int q = 0; q < (r.ff ? 2 : 1); ++q) {
       const std::string h = p + "hc" + std::to_string(q + 1) + ".";
-      lw.sub[q].in = widen(h + "in");
-      lw.sub[q].out = widen(h + "out");
-      lw.sub[q].mix = widen(h + "mix");
-      lw.sub[q].norm = widen(p + (q ? "norm2" : "norm1"));
+      lw.sub[q].in = k.widen(h + "in");
+      lw.sub[q].out = k.widen(h + "out");
+      lw.sub[q].mix = k.widen(h + "mix");
+      lw.sub[q].norm = k.widen(p + (q ? "norm2" : "norm1"));
     }
     if (r.ff) {
-      lw.up = matrix(p + "mlp.up", "");
-      lw.down = matrix(p + "mlp.down", "");
+      lw.up = k.stack({p + "mlp.up"});
+      lw.down = k.stack({p + "mlp.down"});
     }
     w->L.push_back(lw);
   }
   if (!k.status) {
-    w->head = matrix("head", "");
-    w->final_norm = widen("final.norm");
+    w->head = k.stack({"head"});
+    w->final_norm = k.widen("final.norm");
     w->embed = (const uint16_t *)m->tensor("embed").data;
     w->pos = (const uint16_t *)m->tensor("pos").data;
-    if (!k.status && ainfer_sync(dev, UINT64_MAX) != AINFER_OK) k.fail(1, ainfer_last_error(dev));
   }
-  for (auto &kv : kernels) ainfer_kernel_release(kv.second);
+  k.finish();
   m->rows = w;
   return k.status;
 }
 
-const ModelArch kModel = {"Sinepel", false, parse, to_json, check, plan, check_directory, prepare};
-
 // ------------------------------------------------------------------- row engine ---
-struct alignas(64) TensorMap { unsigned char b[128]; };
-enum { ACT_NONE = 0, ACT_RELU2 = 1, ACT_SOFTCAP = 2 };
-
 struct TailRecord {   // SeqTailLayer of k_hyper.cu
   const float *pend_shift;
   float *shift;
@@ -323,14 +218,8 @@ struct TailRecord {   // SeqTailLayer of k_hyper.cu
   int32_t C, taps;
 };
 
-struct Engine : RowEngine {
-  DeviceModel *m;
-  ainfer_device_t dev;
-  const RowWeights *w;
-  int nseq, max_ctx, sm_count = 1;
-  bool f32;
-  std::vector<void *> owned;
-  std::string alloc_err;
+struct Engine : RowEngineBase {
+  const SinepelWeights *w;
   struct LayerState { float *shift, *conv, *pend_shift, *pend_conv; char *k; int cap, chunk; };
   std::vector<LayerState> st;
   char *state = nullptr;
@@ -345,30 +234,10 @@ struct Engine : RowEngine {
   int cur = 0;
   const RowSublayer *pending = nullptr;
 
-  size_t esz() const { return f32 ? 4 : 2; }
-
-  template <typename T>
-  int alloc(size_t count, T **out) {
-    void *p = nullptr;
-    const size_t bytes = std::max<size_t>(count * sizeof(T), 16);
-    if (ainfer_mem_alloc(dev, bytes, 256, &p) != AINFER_OK || ainfer_mem_fill(dev, p, 0, bytes) != AINFER_OK) {
-      alloc_err = ainfer_last_error(dev);
-      return 1;
-    }
-    owned.push_back(p);
-    *out = (T *)p;
-    return 0;
-  }
-
-  int create(DeviceModel *model, int n, int ctx, int cap_rows, bool in_f32, std::string &err) {
-    m = model; dev = m->dev; w = m->rows.get();
-    nseq = n; f32 = in_f32;
+  int create(DeviceModel *model, int n, int ctx, int cap_rows, bool in_f32, std::string &err) override {
+    if (begin(model, n, ctx, cap_rows, in_f32, err)) return 1;
+    w = static_cast<const SinepelWeights *>(m->rows.get());
     const ModelConfig &c = m->cfg;
-    max_ctx = std::min(ctx, c.max_positions);
-    rows_cap = std::max(1, cap_rows);
-    ainfer_device_info info;
-    if (ainfer_device_get_info(dev, &info) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
-    sm_count = info.sm_count;
     const size_t W = c.hidden, S = c.streams, R = rows_cap;
     int maxQ = 1, maxF = 1, maxHGD = 1, maxG = 1;
     // one block of state: shift rows, convolution rings, key rings, layer after layer
@@ -408,8 +277,7 @@ struct Engine : RowEngine {
       ts.push_back({s.pend_shift, s.shift, nullptr, nullptr, C, 1});   // steps keep their convolution ring themselves
     }
     ldw = round_up((int)W, 8); ldq = round_up(maxQ, 8); ldf = round_up(maxF, 8);
-    // blocks of a step's attention over sequences, key heads and splits: few tiles each when there are many sequences
-    att_splits = nseq == 1 ? std::max(1, std::min(16, 2 * sm_count / maxG)) : std::max(1, std::min(16, 8 * sm_count / (std::min(nseq, 8 * sm_count) * maxG)));
+    att_splits = step_splits(maxG);
     for (int i = 0; i < 2; ++i) e |= alloc(R * S * W, &X[i]);
     e |= alloc(R * ldw * esz(), &H); e |= alloc(R * maxC, &U); e |= alloc(R * ldq * esz(), &Q);
     e |= alloc(R * ldq * 4, &Att); e |= alloc(R * W, &Y); e |= alloc(R * ldf * 4, &Act);
@@ -423,10 +291,6 @@ struct Engine : RowEngine {
     if (e) { err = "row engine: " + (alloc_err.empty() ? std::string(ainfer_last_error(dev)) : alloc_err); return 1; }
     return 0;
   }
-  ~Engine() override {
-    ainfer_sync(dev, UINT64_MAX);
-    for (void *p : owned) ainfer_mem_free(dev, p);
-  }
   int reset(std::string &err) override {
     if (ainfer_mem_fill(dev, state, 0, state_bytes) != AINFER_OK) { err = ainfer_last_error(dev); return 1; }
     return 0;
@@ -438,39 +302,6 @@ struct Engine : RowEngine {
     else if (which == "Kc") { *p = state + k_off; *n = state_bytes - k_off; }
     else return false;
     return true;
-  }
-
-  // Y[rows][N] = act(X W^T + bias); X in the activation type, out16: Y bf16 (else fp32)
-  void linear(KernelCalls &k, const RowMatrix &mt, const char *Xp, int ldx, int rows, void *Yp, int ldy, int act, bool out16, float cap = 0.0f) {
-    if (k.status) return;
-    if (f32) {
-      k.launch("LinearRows", (uint32_t)(((mt.N + 63) / 64) * ((rows + 63) / 64)), (const float *)Xp, mt.w, mt.bias, (float *)Yp, (int32_t)rows,
-               (int32_t)mt.N, (int32_t)mt.K, (int32_t)ldx, (int32_t)mt.ldw, (int32_t)ldy, (int32_t)act, cap);
-      return;
-    }
-    const int n_tiles = (mt.N + 127) / 128, kb = (mt.K + 63) / 64;
-    int nt = rows <= 16 ? 16 : rows <= 32 ? 32 : rows <= 64 ? 64 : 128;
-    if (rows > 128) {
-      // rows of a tile: as large as possible (operand traffic), but a launch lasts whole rounds of tiles over the SMs
-      long best = -1;
-      for (int t = 256; t >= 96; t -= 16) {
-        const long rounds = ((long)n_tiles * ((rows + t - 1) / t) + sm_count - 1) / sm_count, cost = rounds * (t + 48);
-        if (best < 0 || cost < best) { best = cost; nt = t; }
-      }
-    }
-    const int tiles = n_tiles * ((rows + nt - 1) / nt);
-    int splits = 1;   // few tiles: a cluster of blocks per tile, each a part of K
-    while (rows <= 128 && splits < 8 && tiles * splits * 2 <= sm_count && kb >= splits * 4) splits *= 2;
-    TensorMap wm, xm;
-    if (ainfer_tensor_map_bf16(dev, &wm, mt.w, (uint64_t)mt.N, (uint64_t)mt.K, (uint64_t)mt.ldw, 128) != AINFER_OK ||
-        ainfer_tensor_map_bf16(dev, &xm, Xp, (uint64_t)rows, (uint64_t)mt.K, (uint64_t)ldx, (uint32_t)nt) != AINFER_OK) {
-      k.fail(1, ainfer_last_error(dev));
-      return;
-    }
-    static const char *const names[] = {"LinearTc", "LinearTcSplit2", "LinearTcSplit4", "LinearTcSplit8"};
-    const int which = splits == 8 ? 3 : splits == 4 ? 2 : splits == 2 ? 1 : 0;
-    k.launch(names[which], (uint32_t)(splits > 1 ? tiles * splits : std::min(tiles, sm_count)), wm, xm, mt.bias, Yp, (int32_t)rows, (int32_t)mt.N,
-             (int32_t)mt.K, (int32_t)nt, (int32_t)ldy, (int32_t)act, (int32_t)(out16 ? 1 : 0), cap);
   }
 
   // stream update of the pending sublayer (if any), then the read + norm (+ shift) of the next
@@ -540,13 +371,8 @@ struct Engine : RowEngine {
              (int32_t)c.layers, (int32_t)R, (int32_t)W, (int32_t)row0);
   }
 
-  // head sizes the tensor-core attention takes (bf16), and the name of the instance that holds one
+  // head sizes the tensor-core attention takes (bf16)
   bool mma_dim(const RowLayerConfig &r) const { return !f32 && r.dim % 8 == 0 && r.dim <= 256; }
-  static std::string sized(const char *base, int dim) {
-    for (int d : {32, 64, 96, 128, 192})
-      if (dim <= d) return base + std::to_string(d);
-    return base + std::string("256");
-  }
   void attn_step(KernelCalls &k, const RowLayerConfig &r, const RowLayerWeights &lw, const LayerState &s, const int32_t *ctrl, int n, int C, int ldo,
                  bool out16) {
     const std::string name = mma_dim(r) && r.heads / r.kv_heads <= 16 ? sized("ChunkAttnStepMma", r.dim)
@@ -558,16 +384,11 @@ struct Engine : RowEngine {
   }
 
   // ---- one decode step of sequence 0 ----
-  void gemv(KernelCalls &k, const RowMatrix &mt, const float *x, float *y, int act) {
-    const int rows_pb = (mt.N + 2 * sm_count - 1) / (2 * sm_count);
-    k.launch("StreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), x, mt.w, mt.bias, y, (int32_t)mt.N, (int32_t)mt.K, (int32_t)mt.ldw,
-             (int32_t)rows_pb, (int32_t)act, 0.0f);
-  }
   void hyper_gemv(KernelCalls &k, const RowMatrix &mt, const float *in, const float *norm, const float *shift, float *shift_state,
                   const int32_t *ctrl, float *y, int act, float cap) {
     const ModelConfig &c = m->cfg;
-    const int rows_pb = (mt.N + 2 * sm_count - 1) / (2 * sm_count);
-    k.launch("HyperStreamGemv", (uint32_t)((mt.N + rows_pb - 1) / rows_pb), (const float *)X[cur], (const float *)(pending ? Y : nullptr),
+    const int rows_pb = gemv_rows(mt.N);
+    k.launch("HyperStreamGemv", gemv_blocks(mt.N), (const float *)X[cur], (const float *)(pending ? Y : nullptr),
              (const float *)(pending ? pending->mix : nullptr), (const float *)(pending ? pending->out : nullptr),
              (float *)(pending ? X[cur ^ 1] : nullptr), in, norm, shift, shift_state, ctrl, mt.w, mt.bias, y, (int32_t)c.streams, (int32_t)mt.N,
              (int32_t)mt.K, (int32_t)mt.ldw, (int32_t)rows_pb, (int32_t)act, (float)c.rms_eps, cap);
@@ -609,7 +430,10 @@ struct Engine : RowEngine {
 
 }  // namespace
 
-const ModelArch *sinepel_model_arch() { return &kModel; }
+const ModelArch *sinepel_model_arch() {
+  static const ModelArch a = {"Sinepel", false, parse, to_json, check, plan, check_directory, prepare, []() -> RowEngine * { return new Engine; }};
+  return &a;
+}
 
 bool sinepel_preset(const std::string &name, ModelConfig &c) {
   auto layer = [](int heads, int kv_heads, int dim, int taps, int chunk, int ff) {
@@ -632,16 +456,6 @@ bool sinepel_preset(const std::string &name, ModelConfig &c) {
   }
   c.layers = (int)c.row_layers.size();
   return true;
-}
-
-int row_engine_create(DeviceModel *m, int nseq, int max_ctx, int rows_cap, bool f32, RowEngine **out, std::string &err) {
-  *out = nullptr;
-  if (!m->rows) { err = "usage: this architecture has no row engine"; return 2; }
-  Engine *e = new Engine;
-  const int r = e->create(m, nseq, max_ctx, rows_cap, f32, err);
-  if (r) { delete e; return r; }
-  *out = e;
-  return 0;
 }
 
 }  // namespace ainfer
