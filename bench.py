@@ -460,14 +460,14 @@ def run_prefill_ep(args, dev, model, rank, world, dist):
 
 
 def run_design(args):
-    """--design sinepel: throughput of that architecture at a few sizes beside the INT4 hybrid (one GPU)."""
+    """--design sinepel | robopel: throughput of that architecture at a few sizes beside the closest other model (one GPU)."""
     from ainfer_b200 import cuda_abi, rowbench
     peak, src = measured_peak()
     p = os.path.join(ROOT, "MEASURED_PEAKS.json")
     tf = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
     dev = cuda_abi.Device(0)
     clocks = ClockSampler(0)
-    rows = rowbench.run(dev, args.design_sizes.split(","), peak, tf)
+    rows = rowbench.run(dev, args.design_sizes.split(","), peak, tf, design=args.design)
     print(json.dumps({"design": args.design, "data": "synthetic", "n_gpus": 1, "hbm_gbs": peak, "bf16_tflops": tf, "peak_source": src,
                       "clocks": clocks.stop(), "sizes": rows}))
     dev.close()
@@ -682,7 +682,7 @@ def main():
     ap.add_argument("--ep-steps", type=int, default=5)
     ap.add_argument("--ep-warmup", type=int, default=2)
     ap.add_argument("--list", action="store_true", help="time the recorded list of stand-alone launches instead of the persistent step")
-    ap.add_argument("--design", default=None, choices=["sinepel"], help="instead of the decode benchmark: prefill, decode and batched decode of this architecture")
+    ap.add_argument("--design", default=None, choices=["sinepel", "robopel"], help="instead of the decode benchmark: prefill, decode and batched decode of this architecture")
     ap.add_argument("--design-sizes", default="w1024,w2048,w4096")
     args = ap.parse_args()
     if args.design:

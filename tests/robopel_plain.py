@@ -8,6 +8,8 @@ import math
 
 import torch
 
+from model_files import read_model, write_model  # noqa: F401
+
 
 # ---------------------------------------------------------------- mechanisms ---
 def rms(x, eps, gain=None):
@@ -116,6 +118,15 @@ def route(h, w, correction, top):
     return idx, s.gather(-1, idx)
 
 
+def choice_margin(h, w, correction, top):
+    """[T]: by how much the last chosen score beats the first one left out."""
+    c = torch.softmax(h @ w.T, -1) + correction
+    if top == c.shape[-1]:
+        return torch.full(c.shape[:1], math.inf, dtype=c.dtype)
+    v = torch.topk(c, top + 1, -1).values
+    return v[:, top - 1] - v[:, top]
+
+
 def relu2_expert(h, up, down):
     return torch.relu(h @ up.T).square() @ down.T
 
@@ -163,12 +174,14 @@ class Plain:
         if f["kind"] == "dense":
             return poly_norm(h @ w[p + "up"].T, w[p + "act"], self.c["norm"]["eps"]) @ w[p + "down"].T
         r = f["router"]
+        self.margin = torch.minimum(self.margin, choice_margin(h, w[p + "router"], w[p + "correction"], r["top"]))
         return mixture(h, w[p + "router"], w[p + "correction"], r["top"], [(w[p + f"e{e}.up"], w[p + f"e{e}.down"]) for e in range(r["experts"])])
 
     def forward(self, tokens, want_layers=False):
         c, w, eps = self.c, self.w, self.c["norm"]["eps"]
         x = w["embed"][torch.as_tensor(list(tokens), dtype=torch.long)] * c["embedding"]["scale"]
         layers, kv = [], {}
+        self.margin = torch.full((len(x),), math.inf, dtype=x.dtype)   # per token, over the layers of the last call
         for i, ly in enumerate(c["layers"]):
             x = after_norm(x, self.mixer(i, x, kv), w[f"l{i}.norm1"], eps)
             if ly["mlp"] is not None:
@@ -183,3 +196,116 @@ class Plain:
             out.append(int(self.forward(ids)[-1].argmax()))
             ids.append(out[-1])
         return out
+
+
+# ------------------------------------------------- random models and files ---
+def make_config(width=48, vocab=96, eps=1e-5, embed_scale=3.0, layers=None):
+    return {"architecture": "Robopel", "embedding": {"scale": embed_scale}, "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def rot(dims=16, base=100.0, scaling=(8.0, 1.0, 4.0, 64)):
+    r = {"base": base, "dims": dims}
+    if scaling:
+        r["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return r
+
+
+def dense(ff):
+    return {"ff": ff, "kind": "dense"}
+
+
+def moe(experts, identity, top, ff):
+    return {"expert": {"ff": ff}, "kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}}
+
+
+def attention(heads=4, kv_heads=2, dim=16, vdim=24, size=20, pool=6, turn=rot(), scale=0.6, softcap=9.0, kv_from=None, mlp=None):
+    m = {"dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"size": size}, "scale": scale, "vdim": vdim}
+    if pool:
+        m["mask"]["pool"] = pool
+    if turn:
+        m["rot"] = turn
+    if softcap:
+        m["softcap"] = softcap
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def mingru(width=56, mlp=None):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": mlp}
+
+
+def tensor_shapes(c):
+    W = c["width"]
+    sh = {"embed": (c["vocab"], W)}
+    for i, ly in enumerate(c["layers"]):
+        m, p, f = ly["mixer"], f"l{i}.", ly["mlp"]
+        sh[p + "norm1"] = (W,)
+        if ly["type"] == "mingru":
+            K = m["width"]
+            sh.update({p + "mix.z": (K, W), p + "mix.x": (K, W), p + "mix.g": (K, W), p + "mix.z.b": (K,), p + "mix.x.b": (K,), p + "mix.o": (W, K)})
+        else:
+            H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            sh.update({p + "mix.q": (H * D, W), p + "mix.q.norm": (D,), p + "mix.sink": (H,), p + "mix.g": (H * E, W), p + "mix.o": (W, H * E)})
+            if "kv_from" not in m:
+                sh.update({p + "mix.k": (G * D, W), p + "mix.v": (G * E, W), p + "mix.k.norm": (D,)})
+        if f is None:
+            continue
+        sh[p + "norm2"] = (W,)
+        if f["kind"] == "dense":
+            sh.update({p + "mlp.up": (f["ff"], W), p + "mlp.down": (W, f["ff"]), p + "mlp.act": (4,)})
+        else:
+            n = f["router"]["experts"] + f["router"]["identity"]
+            sh.update({p + "mlp.router": (n, W), p + "mlp.correction": (n,)})
+            for e in range(f["router"]["experts"]):
+                sh.update({p + f"mlp.e{e}.up": (f["expert"]["ff"], W), p + f"mlp.e{e}.down": (W, f["expert"]["ff"])})
+    sh.update({"final.norm": (W,), "head": (c["vocab"], W)})
+    return sh
+
+
+def make_weights(c, seed=0):
+    """Seeded bf16 weights with every mechanism well away from its neutral value: queries long enough for
+    single keys to stand out, sinks of the size of the scores, recurrences that remember for long."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for n, s in tensor_shapes(c).items():
+        r = torch.randn(s, generator=g)
+        leaf = n.split(".", 1)[-1]
+        if leaf in ("norm1", "norm2") or n == "final.norm":
+            v = 0.25 * r
+        elif leaf == "mix.q.norm":
+            v = 1.8 + 0.2 * r
+        elif leaf == "mix.k.norm":
+            v = 1.0 + 0.2 * r
+        elif leaf == "mix.sink":
+            v = 2.0 + r
+        elif leaf == "mix.z.b":
+            v = -2.0 + r
+        elif leaf == "mix.x.b":
+            v = 0.3 * r
+        elif leaf == "mlp.act":
+            v = torch.tensor([0.7, -0.5, 0.4, 0.3]) + 0.1 * r
+        elif leaf == "mlp.router":
+            v = 1.5 * r / math.sqrt(s[1])
+        elif leaf == "mlp.correction":
+            v = 0.4 * r
+        elif n == "embed":
+            v = 0.5 * r
+        else:
+            v = r / math.sqrt(s[1])
+        out[n] = v.to(torch.bfloat16)
+    return out
+
+
+def steady_tokens(plain, n, seed, margin=0.03, block=3):
+    """n random tokens whose expert choices are not close calls."""
+    g = torch.Generator().manual_seed(seed)
+    ids = []
+    while len(ids) < n:
+        for _ in range(60):
+            more = torch.randint(0, plain.c["vocab"], (min(block, n - len(ids)),), generator=g).tolist()
+            plain.forward(ids + more)
+            if plain.margin[len(ids):].min() > margin:
+                break
+        ids += more
+    return ids

@@ -4,12 +4,11 @@ shares no code with the product and the product never imports it.
 
 Notation: T tokens, W width, S residual streams, H query heads over G key heads of size D.
 """
-import json
 import math
-import struct
 
-import numpy as np
 import torch
+
+from model_files import read_model, write_model  # noqa: F401
 
 
 # ---------------------------------------------------------------- mechanisms ---
@@ -187,35 +186,3 @@ def make_weights(c, seed=0):
             v = r / math.sqrt(s[1])
         out[n] = v.to(torch.bfloat16)
     return out
-
-
-def write_model(folder, config, weights):
-    """config.json and model.safetensors."""
-    import os
-    os.makedirs(folder, exist_ok=True)
-    with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(config, f, indent=1)
-    head, off, blobs = {}, 0, []
-    for n in sorted(weights):
-        b = weights[n].contiguous().view(torch.int16).numpy().tobytes()
-        head[n] = {"dtype": "BF16", "shape": list(weights[n].shape), "data_offsets": [off, off + len(b)]}
-        off += len(b)
-        blobs.append(b)
-    j = json.dumps(head).encode()
-    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
-        f.write(struct.pack("<Q", len(j)) + j + b"".join(blobs))
-
-
-def read_model(folder):
-    import os
-    with open(os.path.join(folder, "config.json")) as f:
-        c = json.load(f)
-    with open(os.path.join(folder, "model.safetensors"), "rb") as f:
-        n = struct.unpack("<Q", f.read(8))[0]
-        head, raw = json.loads(f.read(n)), f.read()
-    w = {}
-    for k, e in head.items():
-        if k != "__metadata__":
-            a, b = e["data_offsets"]
-            w[k] = torch.from_numpy(np.frombuffer(raw[a:b], np.int16).copy()).view(torch.bfloat16).reshape(e["shape"])
-    return c, w

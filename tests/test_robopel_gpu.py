@@ -1,0 +1,792 @@
+"""Robopel on the GPU against the plain restatement (robopel_plain.py): every kernel alone, prompts,
+decoding, portions, batches, reuse of slots, window and block edges, far keys, long decoding, and
+generation through the session, the command line and the server. Small random models; 32-bit sessions
+are held to rounding error, bf16 sessions to bf16 rounding (on tokens whose expert choices are not
+close calls)."""
+import json
+import os
+import subprocess
+import threading
+import urllib.request
+
+import numpy as np
+import pytest
+import torch
+
+import robopel_plain as P
+from robopel_models import MODELS, weights
+
+pytestmark = pytest.mark.gpu
+TOL = {"f32": 3e-5, "b16": 8e-2}   # the plain model with operands rounded to bf16 strays by up to 0.05 at single rows
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+
+@pytest.fixture(scope="module")
+def dev():
+    from ainfer_b200 import cuda_abi
+    d = cuda_abi.Device(0)
+    yield d
+    d.close()
+
+
+@pytest.fixture(scope="module")
+def rt():
+    from ainfer_b200 import runtime
+    return runtime
+
+
+def bf16(x):
+    return torch.as_tensor(x).to(torch.bfloat16)
+
+
+def bits(x):
+    return bf16(x).contiguous().view(torch.int16).numpy()
+
+
+def from_bits(a, shape):
+    return torch.from_numpy(np.ascontiguousarray(a).view(np.int16).copy()).view(torch.bfloat16).float().reshape(shape).numpy()
+
+
+def f32(x):
+    return np.ascontiguousarray(torch.as_tensor(x).float().numpy())
+
+
+def ctrl(positions, tokens=None):
+    c = np.zeros((len(positions), 4), np.int32)
+    c[:, 1], c[:, 2] = positions, np.asarray(positions) + 1
+    if tokens is not None:
+        c[:, 0] = tokens
+    return c
+
+
+def close(got, want, tol):
+    """Every element within tol of its own size plus the array's."""
+    want = np.asarray(want, np.float64)
+    err = (np.abs(np.asarray(got, np.float64) - want) / (np.abs(want) + np.sqrt((want ** 2).mean()) + 1e-30)).max()
+    assert err < tol, err
+
+
+def gen(seed):
+    g = torch.Generator().manual_seed(seed)
+    return lambda *s: torch.randn(*s, generator=g)
+
+
+def padded(w):
+    """Rows of a bf16 matrix padded to a multiple of 8 values."""
+    ld = -(-w.shape[1] // 8) * 8
+    p = torch.zeros(w.shape[0], ld)
+    p[:, :w.shape[1]] = w.float()
+    return bits(p), ld
+
+
+def down(dev, ptr, shape, kind):
+    raw = dev.download(ptr, shape, np.float32 if kind == "f32" else np.uint16)
+    return raw if kind == "f32" else from_bits(raw, shape)
+
+
+# --------------------------------------------------------------- output norm ---
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+@pytest.mark.parametrize("W,top", [(64, 0), (50, 0), (37, 3), (96, 2), (2500, 0), (4100, 4)])
+def test_output_norm_rows(dev, W, top, kind):
+    """Update, stored residual and operand; the experts' rows by place with identities; chosen rows under a
+    second norm."""
+    rn, R, eps, ld = gen(W), 7, 1e-2, W + 4
+    x, g, fg = rn(R, W), rn(W), rn(W)
+    place, pw = torch.full((R, max(top, 1)), -1, dtype=torch.int32), torch.rand(R, max(top, 1))
+    if top:
+        y = rn(R * top, W)
+        perm = torch.randperm(R * top, generator=torch.Generator().manual_seed(1)).int().reshape(R, top)
+        place = torch.where(torch.arange(R * top).reshape(R, top) % 3 == 1, torch.tensor(-1, dtype=torch.int32), perm)
+        rows = torch.where((place >= 0)[..., None], y[place.clamp(min=0).long()], x[:, None, :].expand(R, top, W)).double()
+        yy = (rows * pw[..., None].double()).sum(1)
+    else:
+        y = rn(R, W)
+        yy = y.double()
+    want = x.double() + P.rms(yy, eps, g.double())
+    up = lambda t: dev.upload(f32(t))   # noqa: E731
+    dx, xo, h = up(x), dev.zeros(R * W * 4), dev.zeros(R * ld * 4)
+    k = dev.kernel("PostNormRowsF32" if kind == "f32" else "PostNormRowsB16")
+    tail = [dev.upload(place.numpy()), up(pw)]
+    k(R, dx, up(y), up(g), xo, *tail, 0, 0, h, W, R, top, ld, eps)
+    dev.sync()
+    close(dev.download(xo, (R, W), np.float32), want, 1e-5)
+    close(down(dev, h, (R, ld), kind)[:, :W], want, 1e-5 if kind == "f32" else 1e-2)
+    idx = np.int32([5, 0, 3])
+    k(3, dx, up(y), up(g), 0, *tail, up(fg), dev.upload(idx), h, W, 3, top, ld, eps)
+    dev.sync()
+    close(down(dev, h, (R, ld), kind)[:3, :W], P.rms(want, eps, fg.double())[idx.tolist()], 1e-5 if kind == "f32" else 1e-2)
+    k(R, dx, 0, 0, xo, *tail, 0, 0, h, W, R, 0, ld, eps)          # nothing pending: a copy
+    dev.sync()
+    close(down(dev, h, (R, ld), kind)[:, :W], x, 1e-6 if kind == "f32" else 1e-2)
+
+
+@pytest.mark.parametrize("K,N,act,final", [(64, 33, 0, False), (50, 20, 1, True), (2052, 70, 0, True), (4100, 9, 0, True), (4096, 40, 2, False), (1, 3, 0, True)])
+def test_output_norm_gemv(dev, K, N, act, final):
+    rn, eps = gen(K + N), 1e-2
+    x, y, g, fg, w, b = rn(K), rn(K), rn(K), rn(K), bf16(rn(N, K)), rn(N)
+    wp, ldw = padded(w)
+    acts = [lambda v: v, lambda v: torch.relu(v) ** 2, lambda v: P.softcap(v, 3.0)]
+    up = lambda t: dev.upload(f32(t))   # noqa: E731
+    for pend in (True, False):
+        xn = x.double() + (P.rms(y.double(), eps, g.double()) if pend else 0)
+        h = P.rms(xn, eps, fg.double()) if final else xn
+        out, xo = dev.zeros(N * 4), dev.zeros(K * 4)
+        dev.kernel("PostNormStreamGemv")(-(-N // 7), up(x), up(y) if pend else 0, up(g), xo, up(fg) if final else 0, dev.upload(wp), up(b), out, N, K, ldw, 7, act,
+                                         eps, 3.0)
+        close(dev.download(out, N, np.float32), acts[act](w.double() @ h + b.double()), 1e-5)
+        close(dev.download(xo, K, np.float32), xn, 1e-5)
+
+
+# ------------------------------------------------------------------ PolyNorm ---
+@pytest.mark.parametrize("F", [64, 33, 1, 1000, 9000])
+def test_poly_norm(dev, F):
+    rn, R, eps, ld = gen(F), 5, 1e-2, -(-F // 8) * 8
+    coef, w = torch.tensor([0.7, -0.4, 0.6, 0.2]), bf16(rn(13, F))
+    z = torch.zeros(R, ld)
+    z[:, :F] = rn(R, F)
+    for kind in ("f32", "b16"):
+        zz = z if kind == "f32" else bf16(z).float()
+        want = P.poly_norm(zz[:, :F].double(), coef.double(), eps)
+        o = dev.zeros(R * ld * 4)
+        dev.kernel("PolyNormRowsF32" if kind == "f32" else "PolyNormRowsB16")(R, dev.upload(f32(z) if kind == "f32" else bits(z)), dev.upload(f32(coef)), o, F, ld,
+                                                                              ld, eps)
+        close(down(dev, o, (R, ld), kind)[:, :F], want, 1e-5 if kind == "f32" else 1e-2)
+    wp, ldw = padded(w)
+    y = dev.zeros(13 * 4)
+    dev.kernel("PolyStreamGemv")(4, dev.upload(f32(z[2, :F])), dev.upload(f32(coef)), dev.upload(wp), y, 13, F, ldw, 4, eps)
+    close(dev.download(y, 13, np.float32), w.double() @ P.poly_norm(z[2:3, :F].double(), coef.double(), eps)[0], 2e-5)
+
+
+# -------------------------------------------------------------------- minGRU ---
+def _gru_plain(u, K, state=None):
+    """u [T][3 K] (z, u, g before their functions): output without the projections, and the states."""
+    eye, zero = torch.eye(K, dtype=torch.float64), torch.zeros(K, dtype=torch.float64)
+    z, x, g = (u[:, i * K:(i + 1) * K].double() for i in range(3))
+    pick = lambda i: torch.nn.functional.pad(eye, (i * K, (2 - i) * K))   # noqa: E731  rows that pick a third
+    y = P.min_gru(u.double(), pick(0), zero, pick(1), zero, pick(2), eye, state)
+    s = zero if state is None else state
+    zs = torch.sigmoid(z)
+    for t in range(len(u)):
+        s = (1 - zs[t]) * s + zs[t] * torch.where(x[t] >= 0, x[t] + 0.5, torch.sigmoid(x[t]))
+    return y, s
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+@pytest.mark.parametrize("K", [40, 300, 33])
+def test_recurrence_over_rows_and_steps(dev, K, kind):
+    """Passes of many sizes (chunks of 32 rows inside), each from the state that the one before left; then
+    steps; the slots hold another sequence's leftovers at the start."""
+    rn = gen(K)
+    T, lda = 213, -(-K // 8) * 8
+    u = rn(T, 3 * K) * 2
+    u[:, :K] -= 2.0      # long memory
+    want, last = _gru_plain(u, K)
+    state = dev.upload(f32(rn(2, 2, K) * 50))
+    st1 = state + 2 * K * 4                                  # second sequence's slots
+    pair, tol = dev.zeros(20 * 2 * K * 4), 1e-5 if kind == "f32" else 1e-2
+    sfx, at, got = "F32" if kind == "f32" else "B16", 0, []
+    cb = -(-K // 256)
+    for n in (1, 31, 32, 33, 2, 64, 3, 40):
+        du, dc, a = dev.upload(f32(u[at:at + n])), dev.upload(ctrl(range(at, at + n))), dev.zeros(n * lda * 4)
+        ch = -(-n // 32)
+        dev.kernel("MinGruChunk")(cb * ch, du, st1, dc, pair, n, K)
+        dev.kernel("MinGruScan" + sfx)(cb * ch, du, pair, st1, dc, a, n, K, lda)
+        got.append(down(dev, a, (n, lda), kind)[:, :K])
+        at += n
+    k = dev.kernel("MinGruStepRows" + sfx)
+    while at < T:       # sequence 0 starts now, sequence 1 goes on
+        i = at - 206
+        du, dc, a = dev.upload(f32(torch.stack([u[i], u[at]]))), dev.upload(ctrl([i, at])), dev.zeros(2 * lda * 4)
+        k(2 * cb, du, state, dc, a, 2, K, lda)
+        r = down(dev, a, (2, lda), kind)[:, :K]
+        close(r[0], want[i], tol)
+        got.append(r[1:])
+        at += 1
+    close(np.concatenate(got), want, tol)
+    close(dev.download(st1, (2, K), np.float32)[(T - 1) & 1], last, 1e-5)
+
+
+@pytest.mark.parametrize("K,N", [(40, 21), (33, 5), (2048, 100)])
+def test_recurrence_gemv(dev, K, N):
+    rn = gen(K)
+    u, w = rn(4, 3 * K), bf16(rn(N, K))
+    wp, ldw = padded(w)
+    y, _ = _gru_plain(u, K)
+    st, out = dev.upload(f32(rn(2, K) * 9)), dev.zeros(N * 4)
+    k = dev.kernel("MinGruStreamGemv")
+    for t in range(4):
+        k(-(-N // 6), dev.upload(f32(u[t])), st, dev.upload(ctrl([t])), dev.upload(wp), out, N, K, ldw, 6)
+        close(dev.download(out, N, np.float32), w.double() @ y[t], 1e-5)
+
+
+# ------------------------------------------------------------------- mixture ---
+def _mixture_case(E, I, top, W, F, R):
+    rn = gen(E * W)
+    x, router, corr = bf16(rn(R, W)).float(), rn(E + I, W) * 2 / W ** 0.5, 0.3 * rn(E + I)
+    up, dn = bf16(rn(E, F, W) / W ** 0.5), bf16(rn(E, W, F) / F ** 0.5)
+    logits = (x @ router.T).float()
+    return x, logits, corr, up, dn
+
+
+CASES = [(5, 2, 3, 40, 24, 70), (16, 0, 1, 50, 33, 9), (3, 1, 4, 64, 130, 40), (40, 8, 6, 128, 72, 200), (1, 0, 1, 16, 8, 3), (200, 56, 8, 64, 40, 33)]
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+@pytest.mark.parametrize("E,I,top,W,F,R", CASES)
+def test_mixture_over_rows(dev, E, I, top, W, F, R, kind):
+    x, logits, corr, up, dn = _mixture_case(E, I, top, W, F, R)
+    s = torch.softmax(logits.double(), -1)
+    idx = torch.topk(s + corr.double(), top, -1).indices
+    EI, ldw, ldf = E + I, -(-W // 8) * 8, -(-F // 8) * 8
+    sel, sw, place, rowof = (dev.zeros(R * top * 4) for _ in range(4))
+    dev.kernel("RouterTopRows")(-(-R // 4), dev.upload(f32(logits)), dev.upload(f32(corr)), sel, sw, R, EI, top)
+    gs = dev.download(sel, (R, top), np.int32)
+    assert np.array_equal(gs, idx.numpy())
+    close(dev.download(sw, (R, top), np.float32), s.gather(1, idx), 1e-5)
+    nt, count = (64 if kind == "f32" else 16), dev.zeros(8)
+    tiles = dev.zeros((R * top // 16 + E + 1) * 16)
+    dev.kernel("MoePlanRows")(1, sel, place, rowof, tiles, count, R, top, E, nt)
+    pl, ct = dev.download(place, (R, top), np.int32), dev.download(count, 2, np.int32)
+    real = gs < E
+    assert ct[1] == real.sum() and (pl[~real] == -1).all() and sorted(pl[real]) == list(range(ct[1]))
+    ro, tl = dev.download(rowof, R * top, np.int32), dev.download(tiles, (int(ct[0]), 4), np.int32)
+    seen = 0
+    for e, p0, n, _ in tl:
+        assert p0 == seen and 0 < n <= nt and all(e in gs[ro[p]] for p in range(p0, p0 + n))
+        seen += n
+    assert seen == ct[1]
+    xp = torch.zeros(R, ldw)
+    xp[:, :W] = x
+    es = 4 if kind == "f32" else 2
+    hp, act, y = dev.zeros(R * top * ldw * es), dev.zeros(R * top * ldf * es), dev.zeros(R * top * W * 4)
+    dev.kernel("GatherRows")(5, hp, dev.upload(f32(xp) if kind == "f32" else bits(xp)), rowof, count, ldw * es, ldw * es, ldw * es)
+    wu, ldu = padded(up.reshape(E * F, W))
+    wd, ldd = padded(dn.reshape(E * W, F))
+    du, dd = dev.upload(wu), dev.upload(wd)
+    if kind == "f32":
+        k = dev.kernel("LinearRowsGrouped")
+        k(7, hp, du, act, tiles, count, F, W, ldw, ldu, ldf, 1)
+        k(7, act, dd, y, tiles, count, W, F, ldf, ldd, W, 0)
+    else:
+        k = dev.kernel("LinearTcGrouped")
+        tm = dev.tensor_map_bf16
+        k(7, tm(du, E * F, W, ldu, 128), tm(hp, R * top, W, ldw, nt), act, tiles, count, F, W, nt, ldf, 1, 1)
+        k(7, tm(dd, E * W, F, ldd, 128), tm(act, R * top, F, ldf, nt), y, tiles, count, W, F, nt, W, 0, 0)
+    dev.sync()
+    got = dev.download(y, (R * top, W), np.float32)
+    want = np.zeros((R * top, W))
+    for r in range(R):
+        for j in range(top):
+            if real[r, j]:
+                want[pl[r, j]] = P.relu2_expert(x[r].double(), up[gs[r, j]].double(), dn[gs[r, j]].double()).numpy()
+    close(got[:seen], want[:seen], 1e-5 if kind == "f32" else 2e-2)
+
+
+@pytest.mark.parametrize("E,I,top,W,F,R", CASES)
+def test_mixture_step(dev, E, I, top, W, F, R):
+    x, logits, corr, up, dn = _mixture_case(E, I, top, W, F, min(R, 8))
+    wu, ldu = padded(up.reshape(E * F, W))
+    wd, ldd = padded(dn.reshape(E * W, F))
+    du, dd, dc = dev.upload(wu), dev.upload(wd), dev.upload(f32(corr))
+    act, sel, sw, y = dev.zeros(top * F * 4), dev.zeros(top * 4), dev.zeros(top * 4), dev.zeros(W * 4)
+    s = torch.softmax(logits.double(), -1)
+    idx = torch.topk(s + corr.double(), top, -1).indices
+    for r in range(len(x)):
+        dx = dev.upload(f32(x[r]))
+        dev.kernel("ExpertUpStreamGemv")(top * -(-F // 5), dev.upload(f32(logits[r])), dc, dx, du, act, sel, sw, E, E + I, top, F, W, ldu, 5, 1)
+        dev.kernel("ExpertDownStreamGemv")(-(-W // 9), act, dx, sel, sw, dd, y, E, top, W, F, ldd, 9)
+        assert dev.download(sel, top, np.int32).tolist() == idx[r].tolist()
+        want = sum(s[r, e] * (P.relu2_expert(x[r].double(), up[e].double(), dn[e].double()) if e < E else x[r].double()) for e in idx[r].tolist())
+        close(dev.download(y, W, np.float32), want, 1e-5)
+
+
+# ----------------------------------------------------------------- attention ---
+def test_rotary_table(dev):
+    f = P.frequencies(10, 300.0, P.rot()["scaling"])
+    t = dev.zeros(700 * 5 * 8)
+    dev.kernel("RotaryTable")(3, t, dev.upload(np.float64(f)), 700, 5)
+    a = np.arange(700)[:, None] * np.array(f)[None]
+    close(dev.download(t, (700, 5, 2), np.float32), np.stack([np.cos(a), np.sin(a)], -1), 1e-7)
+
+
+def _table(dev, freq, n):
+    t = dev.zeros(max(1, n * len(freq)) * 8)
+    if freq:
+        dev.kernel("RotaryTable")(4, t, dev.upload(np.float64(freq)), n, len(freq))
+    return t
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+@pytest.mark.parametrize("H,G,D,E,rd", [(4, 2, 16, 24, 8), (3, 1, 9, 7, 4), (2, 2, 128, 64, 128), (5, 5, 33, 1, 0), (1, 1, 300, 512, 64)])
+def test_projections_to_queries_and_cache(dev, H, G, D, E, rd, kind):
+    """Norms, rotation and append of a pass in the middle of a ring, and block means that reach back before it."""
+    rn, R, p0, cap, pool, eps = gen(D), 45, 100, 128, 6, 1e-2
+    freq = P.frequencies(rd, 50.0) if rd else []
+    n = H * D + G * (D + E) + 3
+    u, qn, kn = rn(R, n), rn(D), rn(D)
+    q = P.rotate(P.rms(u[:, :H * D].reshape(R, H, D).double(), eps, qn.double()), freq, p0)
+    k = P.rotate(P.rms(u[:, H * D:(H + G) * D].reshape(R, G, D).double(), eps, kn.double()), freq, p0)
+    v = u[:, (H + G) * D:(H + G) * D + G * E].reshape(R, G, E).double()
+    old_k, old_v = rn(cap, G, D), rn(cap, G, E)
+    conv = f32 if kind == "f32" else bits
+    dk, dv, dq = dev.upload(conv(old_k)), dev.upload(conv(old_v)), dev.zeros(R * H * D * 4)
+    dc, du, t = dev.upload(ctrl(range(p0, p0 + R))), dev.upload(f32(u)), _table(dev, freq, 200)
+    sfx = "F32" if kind == "f32" else "B16"
+    args = lambda koff: (t, dc, dq, dk, dv, R, H, G, D, E, rd, cap, n, koff, (H + G) * D, eps)   # noqa: E731
+    kernel = dev.kernel("QkvRows" + sfx)
+    kernel(-(-R * (H + 2 * G) // 8), du, dev.upload(f32(qn)), dev.upload(f32(kn)), *args(H * D))
+    dev.sync()
+    tol = 1e-5 if kind == "f32" else 1e-2
+    close(down(dev, dq, (R, H, D), kind), q, tol)
+    gk, gv = down(dev, dk, (cap, G, D), kind), down(dev, dv, (cap, G, E), kind)
+    slots = [p % cap for p in range(p0, p0 + R)]
+    close(gk[slots], k, tol)
+    close(gv[slots], v, tol)
+    untouched = [s for s in range(cap) if s not in slots]
+    ref = (lambda x: x.float().numpy()) if kind == "f32" else (lambda x: bf16(x).float().numpy())
+    assert np.array_equal(gk[untouched], ref(old_k)[untouched]) and np.array_equal(gv[untouched], ref(old_v)[untouched])
+    pk, pv = dev.zeros(64 * G * D * 4), dev.zeros(64 * G * E * 4)
+    dev.kernel("PoolRows" + sfx)((R // pool + 1) * -(-G * (D + E) // 256), dk, dv, pk, pv, dc, R, G * D, G * E, cap, pool)
+    dev.sync()
+    mk, mv = down(dev, pk, (64, G, D), kind), down(dev, pv, (64, G, E), kind)
+    done = [b for b in range(64) if p0 <= (b + 1) * pool - 1 < p0 + R]
+    assert len(done) == 8
+    for b in done:
+        at = [p % cap for p in range(b * pool, (b + 1) * pool)]
+        close(mk[b], torch.tensor(gk[at]).double().mean(0), 1e-5 if kind == "f32" else 1e-2)
+        close(mv[b], torch.tensor(gv[at]).double().mean(0), 1e-5 if kind == "f32" else 1e-2)
+    rest = [b for b in range(64) if b not in done]
+    assert not mk[rest].any() and not mv[rest].any()
+    # queries alone: nothing is appended
+    before = dev.download(dk, cap * G * D * (4 if kind == "f32" else 2), np.uint8)
+    kernel(-(-R * H // 8), du, 0, 0, *args(-1))
+    dev.sync()
+    assert np.array_equal(before, dev.download(dk, cap * G * D * (4 if kind == "f32" else 2), np.uint8))
+    close(down(dev, dq, (R, H, D), kind), P.rotate(u[:, :H * D].reshape(R, H, D).double(), freq, p0), tol)
+
+
+def _edges(T, size, pool):
+    """(row, key index) pairs whose score is made to stand out: tokens just inside and just outside the window, the
+    first token, and tokens of blocks that are just seen and just not yet seen."""
+    out = []
+    for i in range(size, T, 7):
+        out.append((i, [i - size + 1, i - size, 0][(i // 7) % 3]))
+    if pool:
+        for b in range(1, T // pool):
+            for i in ((b + 1) * pool - 1 + size, (b + 1) * pool - 2 + size):
+                if i < T:
+                    out.append((i, b * pool + b % pool))
+    return out
+
+
+def _attn_case(T, H, G, D, E, size, pool, seed):
+    rn = gen(seed)
+    q, k, v = rn(T, H, D), rn(T, G, D), rn(T, G, E)
+    for n, (i, j) in enumerate(_edges(T, size, pool)):
+        h = n % H
+        q[i, h] = k[j, h // (H // G)] * 3.0      # one head asks for that key
+    return bf16(q).float(), bf16(k).float(), bf16(v).float(), rn(H) + 1.0, rn(T, H * E)
+
+
+ATTN = [  # T, H, G, D, E, window, block, ring, cap of the scores
+    (70, 4, 2, 16, 24, 20, 6, 128, 9.0), (33, 3, 3, 20, 8, 1, 5, 64, None), (90, 8, 2, 64, 64, 30, 1, 128, 20.0), (40, 5, 1, 33, 17, 1000, 4, 64, 5.0),
+    (150, 4, 4, 128, 96, 64, 16, 192, 30.0), (260, 6, 2, 96, 32, 65, 7, 320, None), (300, 4, 2, 40, 40, 17, 3, 320, 50.0), (200, 2, 1, 256, 200, 63, 64, 256, 8.0),
+    (129, 3, 1, 176, 192, 40, 100, 192, 15.0), (140, 2, 2, 8, 8, 9, None, 192, 6.0), (460, 2, 1, 16, 16, 12, 2, 512, 12.0), (128, 1, 1, 64, 128, 128, 32, 128, 10.0)]
+
+
+def _mma(base, D, E):
+    return base + str(next(p for p in (32, 64, 96, 128, 192, 256) if max(D, E) <= p))
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16", "mma"])
+@pytest.mark.parametrize("T,H,G,D,E,size,pool,cap,softcap", ATTN)
+def test_attention_over_rows(dev, T, H, G, D, E, size, pool, cap, softcap, kind):
+    """Whole, and from the middle with what came before in the cache; output gate and sink; then without them."""
+    if kind == "mma" and (D % 8 or E % 8):
+        pytest.skip("sizes for the CUDA-core form")
+    q, k, v, sink, gate = _attn_case(T, H, G, D, E, size, pool, T)
+    conv = f32 if kind == "f32" else bits
+    ring_k, ring_v = torch.randn(cap, G, D), torch.randn(cap, G, E)
+    ring_k[:T], ring_v[:T] = k, v
+    nb = -(-(T // (pool or T) + 1) // 64) * 64
+    mk, mv = torch.randn(nb, G, D), torch.randn(nb, G, E)
+    if pool:
+        mk[:T // pool], mv[:T // pool] = P.block_means(k, pool), P.block_means(v, pool)
+    scale = 0.35
+    dk, dv, dmk, dmv, dsink = dev.upload(conv(ring_k)), dev.upload(conv(ring_v)), dev.upload(conv(mk)), dev.upload(conv(mv)), dev.upload(f32(sink))
+    ldo = -(-H * E // 8) * 8
+    for start, plain in ((0, False), (T // 3, False), (T // 2 + 1, True)):
+        want = P.sink_attention(q.double(), k.double(), v.double(), scale, softcap, size, pool, None if plain else sink.double()).reshape(T, H * E)
+        if not plain:
+            want = want * torch.sigmoid(gate.double())
+        R = T - start
+        o = dev.zeros(R * ldo * 4)
+        name, rows = {"f32": ("WindowAttnRowsF32", 16), "b16": ("WindowAttnRowsB16", 16), "mma": (_mma("WindowAttnMma", D, E), 64)}[kind]
+        g = torch.zeros(R, H * E + 5)
+        g[:, 3:3 + H * E] = gate[start:]
+        dg = dev.upload(f32(g))
+        dev.kernel(name)(-(-R // rows) * H, dev.upload(conv(q[start:])), dk, dv, dmk if pool else 0, dmv if pool else 0, 0 if plain else dsink,
+                         0 if plain else dg + 12, dev.upload(ctrl(range(start, T))), o, R, H, G, D, E, cap, size, pool or 0, H * E + 5, ldo, scale,
+                         float(softcap or 0))
+        dev.sync()
+        got = down(dev, o, (R, ldo), "f32" if kind == "f32" else "b16")[:, :H * E]
+        close(got, want[start:], 2e-5 if kind == "f32" else 3e-2)
+
+
+STEP = [  # H, G, D, E, window, block, rotated, splits, ring, cap of the scores
+    (4, 2, 16, 24, 20, 6, 8, 1, 64, 9.0), (16, 1, 96, 96, 100, 5, 96, 4, 128, None), (6, 2, 20, 7, 33, 3, 6, 5, 64, 12.0), (8, 1, 64, 32, 70, 1, 64, 2, 128, 30.0),
+    (3, 3, 33, 40, 1, 4, 0, 3, 64, 5.0), (4, 4, 128, 128, 40, 16, 64, 8, 64, 20.0), (20, 1, 40, 16, 50, 9, 40, 16, 64, 7.0), (4, 2, 192, 256, 64, None, 32, 2, 128, 15.0),
+    (2, 1, 8, 8, 9, 50, 8, 16, 64, 6.0)]
+
+
+@pytest.mark.parametrize("reader", [False, True])
+@pytest.mark.parametrize("kind", ["f32", "b16", "mma"])
+@pytest.mark.parametrize("H,G,D,E,size,pool,rd,splits,cap,softcap", STEP)
+def test_attention_step(dev, H, G, D, E, size, pool, rd, splits, cap, softcap, kind, reader):
+    """Three sequences decode side by side from position 0, at different times; the rings are shorter than
+    the run and hold leftovers. reader: a second launch with other queries reads the same cache and
+    averages blocks of its own size."""
+    if kind == "mma" and (D % 8 or E % 8 or H // G > 16):
+        pytest.skip("sizes for the CUDA-core form")
+    if reader and pool is None:
+        pytest.skip("no blocks")
+    T, eps, scale = 230, 1e-2, 0.35
+    rn = gen(D + H)
+    freq = P.frequencies(rd, 100.0, P.rot()["scaling"]) if rd else []
+    qd, kd, vd = H * D, G * D, G * E
+    n = qd + kd + vd + H * E + 2
+    u, qn, kn, sink = rn(3, T, n), 1.5 * rn(D), rn(D), rn(H)
+    u2 = rn(3, T, qd)
+    pool2, size2 = (pool or 0) + 2, max(1, size - 3)
+    lag, want, want2 = [0, 17, 60], [], []
+    stored = (lambda x: x) if kind == "f32" else (lambda x: bf16(x).double())
+    head = lambda x, w, N: P.rotate(P.rms(x.reshape(T, N, D).double(), eps, w.double()), freq)   # noqa: E731
+    for s in range(3):
+        for i, j in _edges(T, size, pool):       # before norm and rotation: raw queries along raw keys
+            h = (i + j) % H
+            u[s, i, h * D:(h + 1) * D] = u[s, j, qd + (h // (H // G)) * D:][:D]
+        k = stored(head(u[s, :, qd:qd + kd], kn, G))
+        v = stored(u[s, :, qd + kd:qd + kd + vd].reshape(T, G, E).double())
+        q, q2 = head(u[s, :, :qd], qn, H), head(u2[s], qn, H)
+        if kind == "mma":
+            q, q2 = bf16(q).double(), bf16(q2).double()
+        g = torch.sigmoid(u[s, :, qd + kd + vd:qd + kd + vd + H * E].double())
+        want.append(P.sink_attention(q, k, v, scale, softcap, size, pool, sink.double()).reshape(T, -1) * g)
+        want2.append(P.sink_attention(q2, k, v, scale, None, size2, pool2, None).reshape(T, -1))
+    t = _table(dev, freq, 256)
+    nb, es = 64 * -(-(T // (pool or T) + 1) // 64), 4 if kind == "f32" else 2
+    junk = lambda *s: dev.upload(f32(rn(*s)) if kind == "f32" else bits(rn(*s)))   # noqa: E731
+    kc, vc, pk, pv, pk2, pv2 = junk(3, cap, kd), junk(3, cap, vd), junk(3, nb, kd), junk(3, nb, vd), junk(3, nb, kd), junk(3, nb, vd)
+    assert es and size2 <= cap and pool2 <= cap
+    part, cnt = dev.zeros(3 * splits * H * (E + 4) * 4), dev.zeros(3 * G * 4)
+    o, du, du2, dc = dev.zeros(3 * H * E * 4), dev.zeros(3 * n * 4), dev.zeros(3 * qd * 4), dev.zeros(48)
+    dqn, dkn, ds = dev.upload(f32(qn)), dev.upload(f32(kn)), dev.upload(f32(sink))
+    k = dev.kernel({"f32": "WindowAttnStepF32", "b16": "WindowAttnStepB16", "mma": _mma("WindowAttnStepMma", D, E)}[kind])
+    got, got2 = np.zeros((3, T, H * E), np.float32), np.zeros((3, T, H * E), np.float32)
+    for step in range(T + 60):
+        pos = [min(max(step - lag[s], 0), T - 1) for s in range(3)]
+        dev.write(du, f32(torch.stack([u[s, pos[s]] for s in range(3)])))
+        dev.write(dc, ctrl(pos))
+        k(3 * G * (splits + 1), du, dqn, dkn, t, dc, kc, vc, pk if pool else 0, pv if pool else 0, cap * kd, cap * vd, nb * kd, nb * vd, ds, part, cnt, o, 3, H, G,
+          D, E, rd, cap, size, pool or 0, qd, qd + kd, qd + kd + vd, 1, splits, n, H * E, 0, scale, float(softcap or 0), eps)
+        r = dev.download(o, (3, H * E), np.float32)
+        if reader:
+            dev.write(du2, f32(torch.stack([u2[s, pos[s]] for s in range(3)])))
+            k(3 * G * (splits + 1), du2, dqn, 0, t, dc, kc, vc, pk2, pv2, cap * kd, cap * vd, nb * kd, nb * vd, 0, part, cnt, o, 3, H, G, D, E, rd, cap, size2,
+              pool2, -1, 0, -1, 1, splits, qd, H * E, 0, scale, 0.0, eps)
+            r2 = dev.download(o, (3, H * E), np.float32)
+        for s in range(3):
+            got[s, pos[s]] = r[s]
+            if reader:
+                got2[s, pos[s]] = r2[s]
+    for s in range(3):
+        close(got[s], want[s], 3e-5 if kind == "f32" else 2.5e-2)
+        if reader:
+            close(got2[s], want2[s], 3e-5 if kind == "f32" else 2.5e-2)
+
+
+# -------------------------------------------------------------------- models ---
+@pytest.fixture(scope="module", params=sorted(MODELS))
+def bundle(request, dev, rt, tmp_path_factory):
+    c, w = MODELS[request.param], weights(request.param)
+    folder = str(tmp_path_factory.mktemp(request.param))
+    P.write_model(folder, c, w)
+    model, plain = rt.Model(dev, folder), P.Plain(c, w)
+    toks = P.steady_tokens(plain, 130, 5)
+    yield c, plain, model, toks, plain.forward(toks).numpy(), folder
+    model.close()
+
+
+def logit_err(got, want):
+    d = got - want
+    return np.sqrt((d * d).mean(-1)).max() / want.std()
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+def test_prompt_decoding_and_portions(rt, bundle, kind):
+    c, _, model, toks, want, _ = bundle
+    T = len(toks)
+    s = rt.Session(model, 200, rt.Session.F32 if kind == "f32" else 0)
+    assert logit_err(s.prefill_logits(toks, range(T)), want) < TOL[kind]
+    assert logit_err(s.prefill_logits(toks, [0, 3, 64, T - 1]), want[[0, 3, 64, T - 1]]) < TOL[kind]    # state from before is not read at position 0
+    s.reset()
+    got = []
+    for i, t in enumerate(toks):
+        s.step(t, i)
+        got.append(s.logits())
+    assert logit_err(np.stack(got), want) < TOL[kind]
+    for sizes in ([2], [3, 2, 7], [17, 2, 1, 40, 5], [96, 2], [33]):
+        s.reset()
+        got, i, j = [], 0, 0
+        while i < T:
+            n = min(sizes[j % len(sizes)], T - i)
+            if n == 1:
+                s.step(toks[i], i)
+                got.append(s.logits()[None])
+            else:
+                got.append(s.prefill_logits(toks[i:i + n], range(n), i))
+            i, j = i + n, j + 1
+        assert logit_err(np.concatenate(got), want) < TOL[kind], sizes
+    # passes of few rows inside one call, then decoding
+    s.prefill_rows(5)
+    s.reset()
+    s.prefill(toks[:77])
+    got = []
+    for i in range(77, T):
+        s.step(toks[i], i)
+        got.append(s.logits())
+    assert logit_err(np.stack(got), want[77:]) < TOL[kind]
+    s.close()
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+def test_batch_of_unequal_sequences_and_reused_slots(rt, bundle, kind):
+    """Three slots; sequences start at different steps, one slot is given to another sequence in the
+    middle. Every sequence against the plain model alone."""
+    c, plain, model, toks, _, _ = bundle
+    seqs = [toks[:100]] + [P.steady_tokens(plain, n, 20 + n) for n in (100, 60, 40)]
+    plan = [(0, 0, 0), (1, 1, 9), (2, 2, 0), (3, 2, 61)]        # (sequence, slot, first step)
+    refs = [plain.forward(q).numpy() for q in seqs]
+    bd = rt.BatchDecode(model, 3, 160, flags=rt.BatchDecode.F32 if kind == "f32" else 0)
+    err = 0.0
+    for step in range(110):
+        tok, pos, who = [0, 1, 2], [0, 0, 0], [None] * 3
+        for q, slot, s0 in plan:
+            if s0 <= step < s0 + len(seqs[q]):
+                tok[slot], pos[slot], who[slot] = seqs[q][step - s0], step - s0, q
+        bd.set_inputs(tok, pos)
+        bd.step()
+        bd.dev.sync()
+        lg = bd.read("logits", np.float32).reshape(3, -1)
+        for slot in range(3):
+            if who[slot] is not None:
+                err = max(err, np.sqrt(((lg[slot] - refs[who[slot]][pos[slot]]) ** 2).mean()) / refs[who[slot]].std())
+    assert err < TOL[kind]
+    bd.close()
+
+
+def test_large_batch_follows_single_sequences(rt, bundle):
+    """70 sequences of one token more each step, against sessions alone (32-bit)."""
+    c, plain, model, toks, _, _ = bundle
+    B = 70
+    bd = rt.BatchDecode(model, B, 64, flags=rt.BatchDecode.F32)
+    ids = np.random.default_rng(3).integers(0, c["vocab"], (B, 9))
+    for t in range(9):
+        bd.set_inputs(ids[:, t].tolist(), [t] * B)
+        bd.step()
+    bd.dev.sync()
+    lg = bd.read("logits", np.float32).reshape(B, -1)
+    for b in (0, 1, 31, 69):
+        assert logit_err(lg[b][None], plain.forward(ids[b].tolist()).numpy()[-1:]) < TOL["f32"]
+    bd.close()
+
+
+def test_sessions_do_not_leak_into_the_next_request(rt, bundle):
+    c, _, model, toks, want, _ = bundle
+    s = rt.Session(model, 200, rt.Session.F32)
+    other = [(5 * t + 1) % c["vocab"] for t in toks]
+    s.prefill(other)
+    for i in range(3):
+        s.step(other[i], 130 + i)
+    a = s.prefill_logits(toks[:90], range(90))             # no reset: position 0 starts anew
+    assert logit_err(a, want[:90]) < TOL["f32"]
+    s.reset()
+    b = s.prefill_logits(toks[:90], range(90))
+    assert np.array_equal(a, b)
+    s.close()
+
+
+def test_greedy_generation_everywhere(rt, bundle):
+    """Session loop (32-bit: the plain model's tokens), recorded per-layer lists, the command line, the
+    server's worker, batched decode, and the folder converted to a container."""
+    from ainfer_b200 import server
+    c, plain, model, toks, _, folder = bundle
+    prompt, n = toks[:21], 24
+    want = plain.greedy(prompt, n)
+    s = rt.Session(model, 96, rt.Session.F32)
+    assert s.generate(prompt, n).tolist() == want
+    s.reset()
+    s.prefill(prompt[:-1])
+    assert s.generate(prompt[-1:], n, start_pos=len(prompt) - 1).tolist() == want
+    tok, _ = s.sample(0.7, top_k=1, rng=3)
+    assert tok == int(s.logits().argmax())
+    s.close()
+    s = rt.Session(model, 96, rt.Session.F32 | rt.Session.PER_LAYER_LISTS)
+    assert s.generate(prompt, n).tolist() == want
+    s.close()
+    bd = rt.BatchDecode(model, 2, 96, flags=rt.BatchDecode.F32)     # the step advances tokens and positions itself
+    got = []
+    for i in range(len(prompt) + n - 1):
+        if i < len(prompt):
+            bd.set_inputs([prompt[i]] * 2, [i] * 2)
+        bd.step()
+        bd.dev.sync()
+        if i >= len(prompt) - 1:
+            got.append(bd.read("out_tok", np.int32).tolist())
+    assert got == [[t, t] for t in want]
+    bd.close()
+    eng = server.Engine(folder, 512, f32=True)
+    assert eng.generate(prompt, n, {})[0] == want
+    srv = server.serve(eng, server.IdTokenizer(eng.vocab), port=0)
+    threading.Thread(target=srv.serve_forever, daemon=True).start()
+    req = urllib.request.Request(f"http://127.0.0.1:{srv.server_address[1]}/v1/completions",
+                                 data=json.dumps({"prompt": prompt, "max_tokens": n}).encode(), headers={"Content-Type": "application/json"})
+    assert json.loads(urllib.request.urlopen(req, timeout=60).read())["choices"][0]["token_ids"] == want
+    srv.shutdown()
+    eng.close()
+    for spec in (folder, folder + "/m.binfer"):
+        if spec != folder:
+            rt.from_safetensors(folder, json.dumps(c), spec)
+        r = subprocess.run([rt.DECODE_EXE, spec, "0", str(n - 1), "--ids=" + ",".join(map(str, prompt)), "--dtype=float32", "--eos=-1"],
+                           capture_output=True, text=True, timeout=120)
+        assert r.returncode == 0, r.stderr
+        line = [x for x in r.stdout.splitlines() if x.startswith("generated:")][0]
+        assert [int(x) for x in line.split()[1:]] == want, spec
+
+
+def test_residual_after_every_layer(rt, bundle):
+    c, plain, model, toks, _, _ = bundle
+    _, layers = plain.forward(toks[:60], want_layers=True)
+    s = rt.Session(model, 96, rt.Session.F32 | rt.Session.DIAG)
+    s.prefill(toks[:50])
+    for i in range(50, 60):
+        s.step(toks[i], i)
+        got = s.read("layer_out", np.float32).reshape(len(c["layers"]), -1)
+        for n in range(len(c["layers"])):
+            close(got[n], layers[n, i], 5e-5)
+    s.close()
+
+
+def test_bf16_generation_follows_the_plain_logits(rt, bundle):
+    c, plain, model, toks, _, _ = bundle
+    s = rt.Session(model, 96)
+    got = s.generate(toks[:21], 24).tolist()
+    s.close()
+    ref = plain.forward(toks[:21] + got[:-1])
+    clear = (plain.margin.cummin(0).values[20:] > 0.03).numpy()       # up to the first close call of a router
+    ref = ref.numpy()[20:]
+    lost = [ref[i].max() - ref[i][g] for i, g in enumerate(got) if clear[i]]
+    assert lost and max(lost) < 6 * TOL["b16"] * ref.std()
+
+
+@pytest.mark.parametrize("kind", ["f32", "b16"])
+def test_long_context_over_ring_ends(dev, rt, tmp_path, kind):
+    """A context longer than the rings hold (a window and one pass of rows), blocks of thousands of tokens
+    ago, window and block edges inside passes, in prompts and in decoding; batched decode goes round a
+    ring of little more than the window many times."""
+    c = P.make_config(width=32, vocab=64, layers=[P.attention(heads=2, kv_heads=1, dim=16, vdim=16, size=150, pool=20, turn=P.rot(16, 1e4), scale=0.9, softcap=20.0,
+                                                              mlp=P.dense(48)),
+                                                  P.mingru(24), P.attention(heads=4, kv_heads=1, dim=16, vdim=16, size=90, pool=33, turn=P.rot(16, 1e4), scale=0.9,
+                                                                            kv_from=0)])
+    w = P.make_weights(c, 9)
+    P.write_model(str(tmp_path), c, w)
+    T = 2900
+    toks = [int(t) for t in np.random.default_rng(1).integers(0, 64, T)]
+    want = P.Plain(c, w).forward(toks).numpy()
+    model = rt.Model(dev, str(tmp_path))
+    s = rt.Session(model, 4096, rt.Session.F32 if kind == "f32" else 0)
+    edges = sorted({p for size, pool in ((150, 20), (90, 33)) for b in range(T // pool) for p in (b * pool + size - 2, b * pool + size - 1, b * pool + size)
+                    if p < T} | set(range(0, 6)) | {T - 1})
+    tol = TOL[kind]
+    assert logit_err(s.prefill_logits(toks, edges), want[edges]) < tol
+    s.reset()
+    s.prefill(toks[:2430])
+    got = []
+    for i in range(2430, 2730):
+        s.step(toks[i], i)
+        got.append(s.logits())
+    assert logit_err(np.stack(got), want[2430:2730]) < tol
+    assert logit_err(s.prefill_logits(toks[2730:], range(T - 2730), 2730), want[2730:]) < tol
+    s.close()
+    bd = rt.BatchDecode(model, 2, 4096, flags=rt.BatchDecode.F32 if kind == "f32" else 0)
+    err = []
+    for i in range(700):
+        bd.set_inputs([toks[i], toks[max(0, i - 40)]], [i, max(0, i - 40)])
+        bd.step()
+        bd.dev.sync()
+        lg = bd.read("logits", np.float32).reshape(2, -1)
+        err += [logit_err(lg[:1], want[i:i + 1]), logit_err(lg[1:], want[max(0, i - 40)][None])]
+    assert np.sqrt(np.mean(np.square(err))) < tol
+    bd.close()
+    model.close()
+
+
+def test_far_block_and_lost_state_show(dev, rt, tmp_path):
+    """Two prompts that differ in one early token, far outside every window: later logits differ as the
+    plain model says, through the blocks and the recurrence (32-bit)."""
+    c = P.make_config(width=32, vocab=64, layers=[P.mingru(24), P.attention(heads=2, kv_heads=1, size=10, pool=8, scale=0.9, softcap=20.0)])
+    w = P.make_weights(c, 2)
+    w["l0.mix.z.b"] = w["l0.mix.z.b"] - 4
+    P.write_model(str(tmp_path), c, w)
+    plain, model = P.Plain(c, w), rt.Model(dev, str(tmp_path))
+    a = [int(t) for t in np.random.default_rng(2).integers(0, 64, 120)]
+    b = list(a)
+    b[5] = (b[5] + 17) % 64
+    diff = (plain.forward(a) - plain.forward(b)).numpy()[100:]
+    assert np.abs(diff).max() > 100 * TOL["f32"]
+    s = rt.Session(model, 128, rt.Session.F32)
+    got = s.prefill_logits(a, range(100, 120)) - s.prefill_logits(b, range(100, 120))
+    assert np.abs(got - diff).max() < 20 * TOL["f32"]
+    s.close()
+    model.close()
+
+
+def test_named_model_and_limits(dev, rt):
+    named = rt.Model(dev, "synth:robopel-tiny:seed=3")
+    s = rt.Session(named, 4096, rt.Session.PERSISTENT)      # no persistent step: a recorded list
+    assert s.launches_per_token() > 1 and len(s.generate([1, 2, 3], 5)) == 5
+    assert s.read("gru", np.float32).any() and s.read("Kc", np.uint16).any()
+    with pytest.raises(rt.RuntimeError_, match="no MTP head"):
+        s.mtp_draft(1, 1)
+    s.close()
+    s = rt.Session(named, 24)
+    with pytest.raises(rt.RuntimeError_, match="context overflow"):
+        s.prefill(list(range(25)))
+    s.prefill(list(range(24)))
+    with pytest.raises(rt.RuntimeError_, match="context overflow"):
+        s.step(1, 24)
+    s.close()
+    named.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_replay(rt, bundle, tmp_path, dtype):
+    """bin/trace_run: two requests that alternate, wanted places in any order, a request that ends and
+    whose session serves another."""
+    c, plain, _, toks, want, folder = bundle
+    other = P.steady_tokens(plain, 50, 8)
+    ref = plain.forward(other).numpy()
+    steps = [
+        {"step": 0, "entries": [{"id": "a", "tokens": toks[:40], "want": [0, 39]}], "end": []},
+        {"step": 1, "entries": [{"id": "b", "tokens": other[:7], "want": []}], "end": []},
+        {"step": 2, "entries": [{"id": "a", "tokens": toks[40:41], "want": [0]}, {"id": "b", "tokens": other[7:50], "want": [42, 1]}], "end": ["b"]},
+        {"step": 3, "entries": [{"id": "c", "tokens": other[:1], "want": [0]}], "end": []},
+    ]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "160"],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr
+    assert r.stdout.split("\n")[:4] == ["done 0", "done 1", "done 2", "done 3"]
+    rd = lambda i: np.fromfile(tmp_path / f"{i}.f32", "<f4").reshape(-1, c["vocab"])   # noqa: E731
+    assert not (tmp_path / "1.f32").exists()
+    for got, exp in ((rd(0), want[[0, 39]]), (rd(2), np.stack([want[40], ref[49], ref[8]])), (rd(3), ref[:1])):
+        assert np.sqrt(((got - exp) ** 2).mean()) / want.std() < TOL["f32" if dtype == "float32" else "b16"]
