@@ -6,7 +6,7 @@
 //   U      [rows][3 K]: z (before the logistic), u, g; biases included
 //   State  [seq][2][K] fp32, position p in slot p & 1: a step reads the slot it does not write
 //
-//   MinGruChunk             the pair of every chunk, and the state before the pass
+//   MinGruChunkF32/B16      the pair of every chunk, and the state before the pass
 //   MinGruScanF32/B16       the rows' outputs s silu(g), and the state after the pass
 //   MinGruStepRowsF32/B16   one step of every sequence of a batch
 //   MinGruStreamGemv        one step of one sequence in the prologue of the output projection
@@ -15,13 +15,22 @@
 
 namespace ainfer {
 
-constexpr int kMgRows = 32;   // rows of a chunk
+constexpr int kMgRows = 32, kMgBatch = 8;   // rows of a chunk, rows whose loads are in flight together
 struct MinGruGate { float keep, add; };
+// The logistic function in 32 bits; T = uint16_t (rows that leave in bf16): by approximate instructions of a
+// few ulp.
+template <typename T>
+__device__ __forceinline__ float gate_logistic(float v) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-v));
+  else return logistic(v);
+}
+template <typename T>
 __device__ __forceinline__ MinGruGate mingru_gate(float zp, float u) {
-  const float z = logistic(zp), c = u >= 0.0f ? u + 0.5f : logistic(u);
+  const float z = gate_logistic<T>(zp), c = u >= 0.0f ? u + 0.5f : gate_logistic<T>(u);
   return MinGruGate{1.0f - z, z * c};
 }
-__device__ __forceinline__ float mingru_out(float s, float g) { return s * (g / (1.0f + expf(-g))); }
+template <typename T>
+__device__ __forceinline__ float mingru_out(float s, float g) { return s * (g * gate_logistic<T>(g)); }
 
 struct MinGruChunkArgs {
   const float *U;          // [rows][3 K]
@@ -30,30 +39,51 @@ struct MinGruChunkArgs {
   float *Pair;             // [1 + chunks][2][K]: the state before the pass (second value), then decay and gain
   int32_t rows, K;
 };
-__global__ void __launch_bounds__(256) MinGruChunk(const MinGruChunkArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
+template <typename T>
+__device__ __forceinline__ void mingru_chunk_body(const MinGruChunkArgs &a) {
   const int cb = (a.K + 255) / 256, k = (blockIdx.x % cb) * 256 + threadIdx.x, c = blockIdx.x / cb;
   if (k >= a.K) return;
-  const int r0 = c * kMgRows, r1 = min(a.rows, r0 + kMgRows);
+  const int r0 = c * kMgRows, n = min(kMgRows, a.rows - r0);
   if (c == 0) {
     const int pos = a.Ctrl[CTRL_POS];
     a.Pair[a.K + k] = pos > 0 ? a.State[(size_t)((pos - 1) & 1) * a.K + k] : 0.0f;
   }
+  const float *u = a.U + (size_t)r0 * 3 * a.K + k;
+  const size_t step = (size_t)3 * a.K;
   float A = 1.0f, B = 0.0f;
-#pragma unroll 8
-  for (int r = r0; r < r1; ++r) {
-    const float *u = a.U + (size_t)r * 3 * a.K + k;
-    const MinGruGate g = mingru_gate(u[0], u[a.K]);
-    A = A * g.keep;
-    B = fmaf(B, g.keep, g.add);
+  for (int r = 0; r < n; r += kMgBatch) {
+    float z[kMgBatch], x[kMgBatch];
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i) {   // past the end: the last row again, not used
+      const float *p = u + (size_t)min(r + i, n - 1) * step;
+      z[i] = p[0];
+      x[i] = p[a.K];
+    }
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i)
+      if (r + i < n) {
+        const MinGruGate g = mingru_gate<T>(z[i], x[i]);
+        A = A * g.keep;
+        B = fmaf(B, g.keep, g.add);
+      }
   }
   float *p = a.Pair + (size_t)(c + 1) * 2 * a.K + k;
   p[0] = A;
   p[a.K] = B;
 }
+__global__ void __launch_bounds__(256) MinGruChunkF32(const MinGruChunkArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  mingru_chunk_body<float>(a);
+}
+__global__ void __launch_bounds__(256) MinGruChunkB16(const MinGruChunkArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  mingru_chunk_body<uint16_t>(a);
+}
 #define F(f) AINFER_ARG(MinGruChunkArgs, f)
-AINFER_REGISTER(MinGruChunk, MinGruChunkArgs, 256, 0, 0, nullptr, F(U), F(State), F(Ctrl), F(Pair), F(rows), F(K));
+AINFER_REGISTER(MinGruChunkF32, MinGruChunkArgs, 256, 0, 0, nullptr, F(U), F(State), F(Ctrl), F(Pair), F(rows), F(K));
+AINFER_REGISTER(MinGruChunkB16, MinGruChunkArgs, 256, 0, 0, nullptr, F(U), F(State), F(Ctrl), F(Pair), F(rows), F(K));
 #undef F
 
 struct MinGruScanArgs {
@@ -67,21 +97,41 @@ template <typename T>
 __device__ __forceinline__ void mingru_scan_body(const MinGruScanArgs &a) {
   const int cb = (a.K + 255) / 256, k = (blockIdx.x % cb) * 256 + threadIdx.x, c = blockIdx.x / cb;
   if (k >= a.K) return;
-  const int r0 = c * kMgRows, r1 = min(a.rows, r0 + kMgRows);
+  const int r0 = c * kMgRows, n = min(kMgRows, a.rows - r0);
   float s = a.Pair[a.K + k];
-#pragma unroll 8
-  for (int j = 1; j <= c; ++j) {
-    const float *p = a.Pair + (size_t)j * 2 * a.K + k;
-    s = fmaf(s, p[0], p[a.K]);
+  for (int j = 1; j <= c; j += kMgBatch) {
+    float A[kMgBatch], B[kMgBatch];
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i) {
+      const float *p = a.Pair + (size_t)min(j + i, c) * 2 * a.K + k;
+      A[i] = p[0];
+      B[i] = p[a.K];
+    }
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i)
+      if (j + i <= c) s = fmaf(s, A[i], B[i]);
   }
-#pragma unroll 8
-  for (int r = r0; r < r1; ++r) {
-    const float *u = a.U + (size_t)r * 3 * a.K + k;
-    const MinGruGate g = mingru_gate(u[0], u[a.K]);
-    s = fmaf(s, g.keep, g.add);
-    st_val(reinterpret_cast<T *>(a.A) + (size_t)r * a.lda + k, mingru_out(s, u[2 * a.K]));
+  const float *u = a.U + (size_t)r0 * 3 * a.K + k;
+  const size_t step = (size_t)3 * a.K;
+  T *o = reinterpret_cast<T *>(a.A) + (size_t)r0 * a.lda + k;
+  for (int r = 0; r < n; r += kMgBatch) {
+    float z[kMgBatch], x[kMgBatch], g[kMgBatch];
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i) {
+      const float *p = u + (size_t)min(r + i, n - 1) * step;
+      z[i] = p[0];
+      x[i] = p[a.K];
+      g[i] = p[2 * a.K];
+    }
+#pragma unroll
+    for (int i = 0; i < kMgBatch; ++i)
+      if (r + i < n) {
+        const MinGruGate q = mingru_gate<T>(z[i], x[i]);
+        s = fmaf(s, q.keep, q.add);
+        st_val(o + (size_t)(r + i) * a.lda, mingru_out<T>(s, g[i]));
+      }
   }
-  if (r1 == a.rows) a.State[(size_t)(a.Ctrl[4 * (a.rows - 1) + CTRL_POS] & 1) * a.K + k] = s;
+  if (r0 + n == a.rows) a.State[(size_t)(a.Ctrl[4 * (a.rows - 1) + CTRL_POS] & 1) * a.K + k] = s;
 }
 __global__ void __launch_bounds__(256) MinGruScanF32(const MinGruScanArgs a) {
   pdl_launch_dependents();
@@ -98,14 +148,6 @@ AINFER_REGISTER(MinGruScanF32, MinGruScanArgs, 256, 0, 0, nullptr, F(U), F(Pair)
 AINFER_REGISTER(MinGruScanB16, MinGruScanArgs, 256, 0, 0, nullptr, F(U), F(Pair), F(State), F(Ctrl), F(A), F(rows), F(K), F(lda));
 #undef F
 
-// Element k of one step; next may be null (another block stores it).
-__device__ __forceinline__ float mingru_step(const float *u, const float *prev, float *next, int K, int k) {
-  const MinGruGate g = mingru_gate(u[k], u[K + k]);
-  const float s = fmaf(prev ? prev[k] : 0.0f, g.keep, g.add);
-  if (next) next[k] = s;
-  return mingru_out(s, u[2 * K + k]);
-}
-
 struct MinGruStepRowsArgs {
   const float *U;          // [seq][3 K]
   float *State;            // [seq][2][K]
@@ -119,8 +161,11 @@ __device__ __forceinline__ void mingru_step_rows_body(const MinGruStepRowsArgs &
   if (k >= a.K || q >= a.nseq) return;
   const int pos = a.Ctrl[4 * q + CTRL_POS];
   float *st = a.State + (size_t)q * 2 * a.K;
-  const float y = mingru_step(a.U + (size_t)q * 3 * a.K, pos > 0 ? st + (size_t)((pos - 1) & 1) * a.K : nullptr, st + (size_t)(pos & 1) * a.K, a.K, k);
-  st_val(reinterpret_cast<T *>(a.A) + (size_t)q * a.lda + k, y);
+  const float *u = a.U + (size_t)q * 3 * a.K + k;
+  const MinGruGate g = mingru_gate<T>(u[0], u[a.K]);
+  const float s = fmaf(pos > 0 ? st[(size_t)((pos - 1) & 1) * a.K + k] : 0.0f, g.keep, g.add);
+  st[(size_t)(pos & 1) * a.K + k] = s;
+  st_val(reinterpret_cast<T *>(a.A) + (size_t)q * a.lda + k, mingru_out<T>(s, u[2 * a.K]));
 }
 __global__ void __launch_bounds__(256) MinGruStepRowsF32(const MinGruStepRowsArgs a) {
   pdl_launch_dependents();
@@ -145,7 +190,7 @@ struct MinGruStreamGemvArgs {
   float *Y;                // [N]
   int32_t N, K, ldw, rows_pb;
 };
-__global__ void __launch_bounds__(kSgThreads, 4) MinGruStreamGemv(const MinGruStreamGemvArgs a) {
+__global__ void __launch_bounds__(kSgThreads, 3) MinGruStreamGemv(const MinGruStreamGemvArgs a) {
   __shared__ GemvShared sh;
   pdl_launch_dependents();
   const GemvDims d = gemv_dims(a.ldw);
@@ -157,10 +202,29 @@ __global__ void __launch_bounds__(kSgThreads, 4) MinGruStreamGemv(const MinGruSt
   } else {
     pdl_wait();
     const int pos = a.Ctrl[CTRL_POS];
-    const float *prev = pos > 0 ? a.State + (size_t)((pos - 1) & 1) * a.K : nullptr;
+    const float *prev = a.State + (size_t)((pos - 1) & 1) * a.K;
     float *next = blockIdx.x == 0 ? a.State + (size_t)(pos & 1) * a.K : nullptr;
-#pragma unroll 4
-    for (int k = threadIdx.x; k < a.ldw; k += kSgWarps * 32) sg_put(lo, hi, k, k < a.K ? mingru_step(a.U, prev, next, a.K, k) : 0.0f);
+    constexpr int Q = 8, nth = kSgWarps * 32;   // elements of a thread whose loads are in flight together
+    for (int k0 = threadIdx.x; k0 < a.ldw; k0 += nth * Q) {
+      float z[Q], x[Q], g[Q], p[Q];
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int k = min(k0 + i * nth, a.K - 1);
+        z[i] = a.U[k];
+        x[i] = a.U[a.K + k];
+        g[i] = a.U[2 * a.K + k];
+        p[i] = pos > 0 ? prev[k] : 0.0f;
+      }
+#pragma unroll
+      for (int i = 0; i < Q; ++i) {
+        const int k = k0 + i * nth;
+        if (k >= a.ldw) continue;
+        const MinGruGate q = mingru_gate<float>(z[i], x[i]);
+        const float s = fmaf(p[i], q.keep, q.add);
+        if (next && k < a.K) next[k] = s;
+        sg_put(lo, hi, k, k < a.K ? mingru_out<float>(s, g[i]) : 0.0f);
+      }
+    }
     asm volatile("bar.sync 1, 256;" ::: "memory");
     gemv_consume(c, d, &sh, sg_smem, lo, hi, part);
   }
@@ -176,7 +240,8 @@ AINFER_REGISTER(MinGruStreamGemv, MinGruStreamGemvArgs, kSgThreads, 0, 0, mingru
                 F(ldw), F(rows_pb));
 #undef F
 
-AINFER_EARLY_LAUNCH(MinGruChunk);
+AINFER_EARLY_LAUNCH(MinGruChunkF32);
+AINFER_EARLY_LAUNCH(MinGruChunkB16);
 AINFER_EARLY_LAUNCH(MinGruScanF32);
 AINFER_EARLY_LAUNCH(MinGruScanB16);
 AINFER_EARLY_LAUNCH(MinGruStepRowsF32);

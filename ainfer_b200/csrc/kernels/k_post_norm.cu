@@ -17,7 +17,7 @@ namespace ainfer {
 // -------------------------------------------------------- PostNormRows ---
 struct PostNormRowsArgs {
   const float *X;          // [rows][W]
-  const float *Y;          // [rows][W], or the experts' rows [...][W]; null: no update
+  const void *Y;           // [rows][W] fp32, or the experts' rows [...][W] in the type of H; null: no update
   const float *G;          // [W] gain of y's norm
   float *Xout;             // [rows][W]; null: not stored
   const int32_t *Place;    // [rows][top] row of Y, < 0: identity
@@ -34,22 +34,23 @@ __device__ __forceinline__ void post_norm_row(const PostNormRowsArgs &a, float *
   const int W = a.W, tid = threadIdx.x, out = blockIdx.x, r = a.Idx ? a.Idx[out] : out;
   const float *x = a.X + (size_t)r * W;
   T *h = a.H ? reinterpret_cast<T *>(a.H) + (size_t)out * a.ldh : nullptr;
-  auto load = [&](const float *p, float (&v)[V]) {
+  auto load = [&](const auto *p, float (&v)[V]) {
     if constexpr (V == 4) { const float4 t = ld_val4(p); v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w; }
-    else v[0] = *p;
+    else v[0] = ld_val(p);
   };
   float ss = 0.0f;
   if (a.Y) {
     for (int w = tid * V; w < W; w += 256 * V) {
       float y[V];
       if (a.top == 0) {
-        load(a.Y + (size_t)r * W + w, y);
+        load(reinterpret_cast<const float *>(a.Y) + (size_t)r * W + w, y);
       } else {
         float t[V];
 #pragma unroll
         for (int i = 0; i < V; ++i) y[i] = 0.0f;
         for (int s = 0; s < a.top; ++s) {
-          load(place[s] >= 0 ? a.Y + (size_t)place[s] * W + w : x + w, t);
+          if (place[s] >= 0) load(reinterpret_cast<const T *>(a.Y) + (size_t)place[s] * W + w, t);
+          else load(x + w, t);
 #pragma unroll
           for (int i = 0; i < V; ++i) y[i] = fmaf(pw[s], t[i], y[i]);
         }

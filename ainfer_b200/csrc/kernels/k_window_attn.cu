@@ -46,15 +46,22 @@ __device__ __forceinline__ void qkv_rows_body(const QkvRowsArgs &a) {
   const float2 *rot = a.Rot + (size_t)pos * (a.rd >> 1);
   if (u < a.H) {
     T *q = reinterpret_cast<T *>(a.Q) + ((size_t)r * a.H + u) * a.D;
-    head_norm_turn(src + (size_t)u * a.D, a.D, a.QN, a.eps, rot, a.rd, [&](int d, float v) { st_val(q + d, v); });
+    head_norm_turn(src + (size_t)u * a.D, a.D, a.QN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { st_pair(q + d, x, y, both); });
   } else if (u < a.H + a.G) {
     const int g = u - a.H;
     T *k = reinterpret_cast<T *>(a.Kc) + ((size_t)(pos % a.cap) * a.G + g) * a.D;
-    head_norm_turn(src + a.koff + (size_t)g * a.D, a.D, a.KN, a.eps, rot, a.rd, [&](int d, float v) { st_val(k + d, v); });
+    head_norm_turn(src + a.koff + (size_t)g * a.D, a.D, a.KN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { st_pair(k + d, x, y, both); });
   } else {
     const int g = u - a.H - a.G;
     T *v = reinterpret_cast<T *>(a.Vc) + ((size_t)(pos % a.cap) * a.G + g) * a.E;
-    for (int d = lane; d < a.E; d += 32) st_val(v + d, src[a.voff + (size_t)g * a.E + d]);
+    const float *s = src + a.voff + (size_t)g * a.E;
+    const bool wide = (reinterpret_cast<unsigned long long>(s) & 7) == 0;
+#pragma unroll 4
+    for (int d = lane * 2; d < a.E; d += 64) {
+      const bool both = d + 1 < a.E;
+      const float2 t = both && wide ? *reinterpret_cast<const float2 *>(s + d) : make_float2(s[d], both ? s[d + 1] : 0.0f);
+      st_pair(v + d, t.x, t.y, both);
+    }
   }
 }
 __global__ void __launch_bounds__(256) QkvRowsF32(const QkvRowsArgs a) {
@@ -294,7 +301,7 @@ __device__ __forceinline__ void window_attn_step_body(const WindowAttnStepArgs &
   const bool fresh = a.koff >= 0;
   auto new_key = [&]() {   // warp 0: the key, warp 1: the value, as the cache holds them
     if (!fresh) return;
-    if (warp == 0) head_norm_turn(u + a.koff + (size_t)g * D, D, a.KN, a.eps, rot, a.rd, [&](int d, float v) { kn[d] = as_stored<T>(v); });
+    if (warp == 0) head_norm_turn(u + a.koff + (size_t)g * D, D, a.KN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { kn[d] = as_stored<T>(x); if (both) kn[d + 1] = as_stored<T>(y); });
     if (warp == 1)
       for (int d = lane; d < E; d += 32) vn[d] = as_stored<T>(u[a.voff + (size_t)g * E + d]);
   };
@@ -323,7 +330,7 @@ __device__ __forceinline__ void window_attn_step_body(const WindowAttnStepArgs &
   if (split >= active) return;
   const int j_lo = split * per, j_hi = min(n, j_lo + per);   // blocks 0..nb-1, then tokens lo..pos
   for (int hh = warp; hh < HG; hh += kWsThreads / 32)
-    head_norm_turn(u + (size_t)(g * HG + hh) * D, D, a.QN, a.eps, rot, a.rd, [&](int d, float v) { qs[hh * D + d] = v; });
+    head_norm_turn(u + (size_t)(g * HG + hh) * D, D, a.QN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { qs[hh * D + d] = x; if (both) qs[hh * D + d + 1] = y; });
   new_key();
   for (int i = tid; i < HG * E; i += kWsThreads) acc[i] = 0.0f;
   for (int i = tid; i < HG; i += kWsThreads) { hm[i] = -INFINITY; hl[i] = 0.0f; }

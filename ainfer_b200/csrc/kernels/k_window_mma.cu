@@ -18,27 +18,17 @@ __device__ __forceinline__ float fast_rcp(float x) {   // one instruction, 1 ulp
 }
 __device__ __forceinline__ float fast_logistic(float v) { return fast_rcp(1.0f + fast_exp2(-v * kLog2e)); }
 // A product q . k to a score in powers of two: scale, and cap tanh(. / cap) as cap - 2 cap / (1 + e^(2 . / cap)).
+// bounded: a cap so low that weights relative to it, 2^(score - cap), cannot underflow.
+constexpr float kUnseen = -3.0e38f;   // in the place of a product whose key the row does not see
 struct ScoreMap {
   float mul, c, c2;   // c2 = 0: no cap
+  bool bounded;
   __device__ __forceinline__ ScoreMap(float scale, float cap)
-      : mul(cap > 0.0f ? 2.0f * scale / cap * kLog2e : scale * kLog2e), c(cap * kLog2e), c2(cap > 0.0f ? -2.0f * cap * kLog2e : 0.0f) {}
-  __device__ __forceinline__ float plain(float s) const { return s * mul; }
-  __device__ __forceinline__ float capped(float s) const { return fmaf(c2, fast_rcp(1.0f + fast_exp2(s * mul)), c); }
+      : mul(cap > 0.0f ? 2.0f * scale / cap * kLog2e : scale * kLog2e), c(cap * kLog2e), c2(cap > 0.0f ? -2.0f * cap * kLog2e : 0.0f),
+        bounded(cap > 0.0f && 2.0f * cap * kLog2e < 100.0f) {}
+  __device__ __forceinline__ float below(float s) const { return c2 * fast_rcp(1.0f + fast_exp2(s * mul)); }   // score - cap
+  __device__ __forceinline__ float operator()(float s) const { return c2 != 0.0f ? below(s) + c : s * mul; }
 };
-template <int N>
-__device__ __forceinline__ void map_scores(float (&s)[N][4], const ScoreMap &f) {
-  if (f.c2 != 0.0f) {
-#pragma unroll
-    for (int n = 0; n < N; ++n)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) s[n][i] = f.capped(s[n][i]);
-  } else {
-#pragma unroll
-    for (int n = 0; n < N; ++n)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) s[n][i] = f.plain(s[n][i]);
-  }
-}
 
 // ------------------------------------------------------ WindowAttnMma ---
 struct WindowAttnMmaArgs {
@@ -58,7 +48,7 @@ __device__ __forceinline__ void window_attn_mma_body(const WindowAttnMmaArgs &a)
   extern __shared__ __align__(128) unsigned char wm_raw[];
   constexpr int LD = DP + 8;
   uint16_t *Qs = reinterpret_cast<uint16_t *>(wm_raw);                // [64][LD]
-  const uint32_t qa = cm_smem(Qs), ka = qa + kWmRows * LD * 2, va = ka + 2 * kCmKeys * LD * 2;   // keys [2][64][LD], values [2][64][LD]
+  const uint32_t qa = cm_smem(Qs), ka = qa + kWmRows * LD * 2, va = ka + 2 * kCmKeys * LD * 2;   // keys [2][64][LD], values [64][LD]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int tiles = (a.rows + kWmRows - 1) / kWmRows;
   const int h = blockIdx.x % a.H, r0 = (tiles - 1 - blockIdx.x / a.H) * kWmRows, g = h / (a.H / a.G);   // long rows first
@@ -76,20 +66,14 @@ __device__ __forceinline__ void window_attn_mma_body(const WindowAttnMmaArgs &a)
   const int lo0 = max(0, p0 - a.window + 1), kb0 = lo0 / kCmKeys * kCmKeys;
   const int nbt = (nb1 + kCmKeys - 1) / kCmKeys, nt = nbt + (p1 - kb0) / kCmKeys + 1;
   const uint16_t *K = a.Kc + (size_t)g * a.D, *V = a.Vc + (size_t)g * a.E, *PK = a.Pk + (size_t)g * a.D, *PV = a.Pv + (size_t)g * a.E;
-  int slot = kb0 % a.cap;
-  auto fetch = [&](int t) {
-    const uint32_t o = (uint32_t)((t & 1) * kCmKeys * LD) * 2;
+  auto fetch = [&](int t, bool vals) {   // one commit group: the keys or the values of tile t
     const bool pooled = t < nbt;
-    const int at = pooled ? t * kCmKeys : slot;
-    load_keys<DP, 128>(ka + o, pooled ? PK : K, at, KW, a.D);
-    load_keys<DP, 128>(va + o, pooled ? PV : V, at, VW, a.E);
+    const int at = pooled ? t * kCmKeys : (kb0 + (t - nbt) * kCmKeys) % a.cap;
+    if (vals) load_keys<DP, 128>(va, pooled ? PV : V, at, VW, a.E);
+    else load_keys<DP, 128>(ka + (uint32_t)((t & 1) * kCmKeys * LD) * 2, pooled ? PK : K, at, KW, a.D);
     cpa_commit();
-    if (!pooled) {
-      slot += kCmKeys;
-      if (slot == a.cap) slot = 0;
-    }
   };
-  fetch(0);
+  fetch(0, false);
   const ScoreMap map(a.scale, a.softcap);
   float o[DP / 8][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 #pragma unroll
@@ -99,15 +83,13 @@ __device__ __forceinline__ void window_attn_mma_body(const WindowAttnMmaArgs &a)
   const uint32_t qw = qa + (uint32_t)((warp * 16 + (lane & 15)) * LD + (lane >> 4) * 8) * 2;
   const int rw = warp * 16 + (lane >> 2);                 // this thread's rows rw and rw + 8
   for (int t = 0; t < nt; ++t) {
+    cpa_wait<0>();
+    __syncthreads();   // the keys are there; every warp is done with the values before and the keys two tiles ago
+    fetch(t, true);
     const bool more = t + 1 < nt;
-    if (more) fetch(t + 1);
-    if (more) cpa_wait<1>(); else cpa_wait<0>();
-    __syncthreads();
+    if (more) fetch(t + 1, false);
     float s[kCmKeys / 8][4];
-    const uint32_t off = (uint32_t)((t & 1) * kCmKeys * LD) * 2;
-    scores_smem<DP, kCmKeys>(s, qw, ka + off, lane);
-    map_scores(s, map);
-    float mx[2] = {m[0], m[1]};
+    scores_smem<DP, kCmKeys>(s, qw, ka + (uint32_t)((t & 1) * kCmKeys * LD) * 2, lane);
     const bool pooled = t < nbt;
     const int k0 = pooled ? t * kCmKeys : kb0 + (t - nbt) * kCmKeys;
     const bool whole = pooled ? k0 + kCmKeys <= nb0 : k0 + kCmKeys - 1 <= p0 && k0 > p1 - a.window;   // every row sees every key of the tile
@@ -121,41 +103,61 @@ __device__ __forceinline__ void window_attn_mma_body(const WindowAttnMmaArgs &a)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             const int key = k0 + n * 8 + (lane & 3) * 2 + e;
-            if (key < first || key > last) s[n][2 * x + e] = -INFINITY;
+            if (key < first || key > last) s[n][2 * x + e] = kUnseen;
           }
       }
     }
-#pragma unroll
-    for (int n = 0; n < kCmKeys / 8; ++n)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) mx[i >> 1] = fmaxf(mx[i >> 1], s[n][i]);
-    float corr[2], base[2];
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      mx[x] = quad_max(mx[x]);
-      base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
-      corr[x] = fast_exp2(m[x] - base[x]);
-      m[x] = mx[x];
-    }
     float sum[2] = {0.0f, 0.0f};
+    if (map.bounded) {   // weights relative to the cap itself: no maximum to follow
 #pragma unroll
-    for (int n = 0; n < kCmKeys / 8; ++n)
+      for (int n = 0; n < kCmKeys / 8; ++n)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        s[n][i] = fast_exp2(s[n][i] - base[i >> 1]);
-        sum[i >> 1] += s[n][i];
+        for (int i = 0; i < 4; ++i) {
+          const float w = fast_exp2(map.below(s[n][i]));
+          s[n][i] = whole || s[n][i] != kUnseen ? w : 0.0f;
+          sum[i >> 1] += s[n][i];
+        }
+      l[0] += sum[0];
+      l[1] += sum[1];
+    } else {
+      float mx[2] = {m[0], m[1]};
+#pragma unroll
+      for (int n = 0; n < kCmKeys / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float v = map(s[n][i]);
+          s[n][i] = whole || s[n][i] != kUnseen ? v : -INFINITY;
+          mx[i >> 1] = fmaxf(mx[i >> 1], s[n][i]);
+        }
+      float corr[2], base[2];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        mx[x] = quad_max(mx[x]);
+        base[x] = mx[x] == -INFINITY ? 0.0f : mx[x];
+        corr[x] = fast_exp2(m[x] - base[x]);
+        m[x] = mx[x];
       }
 #pragma unroll
-    for (int x = 0; x < 2; ++x) l[x] = fmaf(l[x], corr[x], sum[x]);
-    if (__any_sync(kFull, corr[0] != 1.0f || corr[1] != 1.0f)) {   // some row's maximum moved
+      for (int n = 0; n < kCmKeys / 8; ++n)
 #pragma unroll
-      for (int d = 0; d < DP / 8; ++d)
+        for (int i = 0; i < 4; ++i) {
+          s[n][i] = fast_exp2(s[n][i] - base[i >> 1]);
+          sum[i >> 1] += s[n][i];
+        }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+      for (int x = 0; x < 2; ++x) l[x] = fmaf(l[x], corr[x], sum[x]);
+      if (__any_sync(kFull, corr[0] != 1.0f || corr[1] != 1.0f)) {   // some row's maximum moved
+#pragma unroll
+        for (int d = 0; d < DP / 8; ++d)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) o[d][i] *= corr[i >> 1];
+      }
     }
-    values<DP, kCmKeys>(o, s, va + off, lane);
-    __syncthreads();
+    if (more) cpa_wait<1>(); else cpa_wait<0>();
+    __syncthreads();   // the values are there
+    values<DP, kCmKeys>(o, s, va, lane);
   }
+  if (map.bounded) m[0] = m[1] = map.c;
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     float den = quad_sum(l[x]);
@@ -183,12 +185,12 @@ __device__ __forceinline__ void window_attn_mma_body(const WindowAttnMmaArgs &a)
     pdl_wait();                                                                                                     \
     window_attn_mma_body<DP>(a);                                                                                    \
   }                                                                                                                 \
-  static uint32_t window_mma_smem##DP(const void *) { return (kWmRows + 4 * kCmKeys) * (DP + 8) * 2; }
+  static uint32_t window_mma_smem##DP(const void *) { return (kWmRows + 3 * kCmKeys) * (DP + 8) * 2; }
 WINDOW_MMA(32, 4)
 WINDOW_MMA(64, 4)
 WINDOW_MMA(96, 3)
-WINDOW_MMA(128, 2)
-WINDOW_MMA(192, 1)
+WINDOW_MMA(128, 3)
+WINDOW_MMA(192, 2)
 WINDOW_MMA(256, 1)
 #define F(f) AINFER_ARG(WindowAttnMmaArgs, f)
 #define WM_FIELDS                                                                                                                              \
@@ -241,7 +243,7 @@ __device__ __forceinline__ void window_step_mma_body(const WindowAttnStepMmaArgs
   const bool fresh = a.koff >= 0;
   auto new_key = [&]() {   // warp 2: the key, warp 3: the value
     if (!fresh) return;
-    if (warp == 2) head_norm_turn(u + a.koff + (size_t)g * D, D, a.KN, a.eps, rot, a.rd, [&](int d, float v) { kn[d] = f32_to_bf16(v); });
+    if (warp == 2) head_norm_turn(u + a.koff + (size_t)g * D, D, a.KN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { st_pair(kn + d, x, y, both); });
     if (warp == 3)
       for (int d = lane; d < E; d += 32) vn[d] = f32_to_bf16(u[a.voff + (size_t)g * E + d]);
   };
@@ -289,7 +291,7 @@ __device__ __forceinline__ void window_step_mma_body(const WindowAttnStepMmaArgs
   for (int i = tid; i < 16 * LD; i += 128) Qs[i] = 0;
   __syncthreads();
   for (int hh = warp; hh < HG; hh += 4)
-    head_norm_turn(u + (size_t)(g * HG + hh) * D, D, a.QN, a.eps, rot, a.rd, [&](int d, float v) { Qs[hh * LD + d] = f32_to_bf16(v); });
+    head_norm_turn(u + (size_t)(g * HG + hh) * D, D, a.QN, a.eps, rot, a.rd, [&](int d, float x, float y, bool both) { st_pair(Qs + hh * LD + d, x, y, both); });
   new_key();
   __syncthreads();
   uint32_t q[DP / 16][4];
@@ -316,7 +318,6 @@ __device__ __forceinline__ void window_step_mma_body(const WindowAttnStepMmaArgs
     const uint32_t off = (uint32_t)((stage * kCmKeys + warp * 16) * LD) * 2;
     float s[2][4];
     scores<DP, 16>(s, q, ka + off, lane);
-    map_scores(s, map);
     const int first = pooled ? 0 : lo, last = pooled ? nb - 1 : pos;
     float mx[2] = {m[0], m[1]};
 #pragma unroll
@@ -324,7 +325,7 @@ __device__ __forceinline__ void window_step_mma_body(const WindowAttnStepMmaArgs
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int key = k0 + n * 8 + (lane & 3) * 2 + (i & 1);
-        if (key < first || key > last) s[n][i] = -INFINITY;
+        s[n][i] = key < first || key > last ? -INFINITY : map(s[n][i]);
         mx[i >> 1] = fmaxf(mx[i >> 1], s[n][i]);
       }
     float corr[2], sum[2] = {0.0f, 0.0f}, base[2];

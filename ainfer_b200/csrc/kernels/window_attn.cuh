@@ -20,9 +20,20 @@ __device__ __forceinline__ int blocks_seen(int i, int window, int pool) {
 }
 __device__ __forceinline__ float cap_score(float s, float cap) { return cap > 0.0f ? cap * tanhf(s / cap) : s; }
 
+// Neighbouring values (d even) of a row; as one access where the row is aligned to pairs.
+__device__ __forceinline__ void st_pair(float *p, float x, float y, bool both) {
+  if (both && (reinterpret_cast<unsigned long long>(p) & 7) == 0) *reinterpret_cast<float2 *>(p) = make_float2(x, y);
+  else { p[0] = x; if (both) p[1] = y; }
+}
+__device__ __forceinline__ void st_pair(uint16_t *p, float x, float y, bool both) {
+  if (both && (reinterpret_cast<unsigned long long>(p) & 3) == 0)
+    *reinterpret_cast<uint32_t *>(p) = (uint32_t)f32_to_bf16(x) | ((uint32_t)f32_to_bf16(y) << 16);
+  else { p[0] = f32_to_bf16(x); if (both) p[1] = f32_to_bf16(y); }
+}
+
 // One warp: a head's D values at src, divided by their root mean square and times w (w null: as they
-// are), then the first rd of them turned in neighbouring pairs by rot (cosine, sine per pair); put(d, v).
-// D <= 512.
+// are), then the first rd of them turned in neighbouring pairs by rot (cosine, sine per pair);
+// put(d, x, y, both): values d and d + 1, the second only if `both`. D <= 512.
 constexpr int kHeadPairs = 8;   // pairs of a lane
 template <typename P>
 __device__ __forceinline__ void head_norm_turn(const float *src, int D, const float *w, float eps, const float2 *rot, int rd, P put) {
@@ -62,8 +73,7 @@ __device__ __forceinline__ void head_norm_turn(const float *src, int D, const fl
       y = y * r.x + x * r.y;
       x = t;
     }
-    if (d < D) put(d, x);
-    if (d + 1 < D) put(d + 1, y);
+    if (d < D) put(d, x, y, d + 1 < D);
   }
 }
 

@@ -488,7 +488,7 @@ struct Engine : RowEngineBase {
   void post_norm(KernelCalls &k, int rows, const float *final_gain, const int32_t *idx) {
     const bool last = final_gain != nullptr;
     if (f32 && !last && !pending.gain) return;
-    k.launch(f32 ? "PostNormRowsF32" : "PostNormRowsB16", (uint32_t)rows, (const float *)X[0], (const float *)(pending.gain ? Y : nullptr), pending.gain,
+    k.launch(f32 ? "PostNormRowsF32" : "PostNormRowsB16", (uint32_t)rows, (const float *)X[0], (const void *)(pending.gain ? Y : nullptr), pending.gain,
              (float *)(last ? nullptr : X[0]), (const int32_t *)Place, (const float *)SelW, final_gain, idx, (void *)(f32 && !last ? nullptr : H),
              (int32_t)m->cfg.hidden, (int32_t)rows, (int32_t)pending.top, (int32_t)ldw, (float)m->cfg.rms_eps);
     pending = Pending();
@@ -521,22 +521,26 @@ struct Engine : RowEngineBase {
       return;
     }
     const uint32_t chunks = (uint32_t)((sp.rows + 31) / 32);
-    k.launch("MinGruChunk", cb * chunks, (const float *)U, (const float *)s.gru, sp.ctrl, Pair, (int32_t)sp.rows, (int32_t)r.width);
+    k.launch(f32 ? "MinGruChunkF32" : "MinGruChunkB16", cb * chunks, (const float *)U, (const float *)s.gru, sp.ctrl, Pair, (int32_t)sp.rows, (int32_t)r.width);
     k.launch(f32 ? "MinGruScanF32" : "MinGruScanB16", cb * chunks, (const float *)U, (const float *)Pair, s.gru, sp.ctrl, (void *)Att, (int32_t)sp.rows,
              (int32_t)r.width, (int32_t)lda);
+  }
+  // Rows of a tile: an expert's rows, two standard deviations above their mean, in as few even tiles as possible.
+  static int expert_tile_rows(double mean) {
+    const double most = mean + 2.0 * std::sqrt(mean);
+    const int tiles = (int)std::ceil(most / 256.0);
+    return std::max(16, std::min(256, round_up((int)std::ceil(most / tiles), 16)));
   }
   void mixture_rows(KernelCalls &k, const RowLayerConfig &r, const LayerWeights &lw, int R) {
     const int EI = r.experts + r.identity, slots = R * r.top, lde = round_up(r.ff, 8), W = m->cfg.hidden;
     linear(k, lw.router, operand(), operand_ld(), R, Logits, EI, ACT_NONE, false);
     k.launch("RouterTopRows", (uint32_t)((R + 3) / 4), (const float *)Logits, lw.correction, Sel, SelW, (int32_t)R, (int32_t)EI, (int32_t)r.top);
-    // rows of a tile by the rows an expert gets on average
-    const int mean = slots / EI;
-    const int nt = f32 ? 64 : mean <= 12 ? 16 : mean <= 24 ? 32 : mean <= 48 ? 64 : mean <= 256 ? 128 : 256;
+    const int nt = f32 ? 64 : expert_tile_rows((double)slots / EI);
     k.launch("MoePlanRows", 1, (const int32_t *)Sel, Place, RowOf, Tiles, Count, (int32_t)R, (int32_t)r.top, (int32_t)r.experts, (int32_t)nt);
     k.launch("GatherRows", (uint32_t)std::min(slots, 8 * sm_count), (void *)Hp, (const void *)operand(), (const int32_t *)RowOf, (const int32_t *)Count,
              (int64_t)(operand_ld() * esz()), (int64_t)(ldw * esz()), (int32_t)(operand_ld() * esz()));
     grouped(k, lw.up, r, Hp, ldw, slots, Act, lde, ACT_RELU2, !f32, nt);
-    grouped(k, lw.down, r, Act, lde, slots, Y, W, ACT_NONE, false, nt);
+    grouped(k, lw.down, r, Act, lde, slots, Y, W, ACT_NONE, !f32, nt);
   }
   // the experts' products over their rows: Y[place][N] = act(X W_e^T)
   void grouped(KernelCalls &k, const RowMatrix &mt, const RowLayerConfig &r, const char *Xp, int ldx, int slots, void *Yp, int ldy, int act, bool out16,
@@ -660,7 +664,7 @@ struct Engine : RowEngineBase {
   }
   void record_residual(KernelCalls &k, float *dst) override {
     const int W = m->cfg.hidden;
-    k.launch("PostNormRowsF32", 1, (const float *)X[cur], (const float *)(pending.gain ? Y : nullptr), pending.gain, dst, (const int32_t *)nullptr,
+    k.launch("PostNormRowsF32", 1, (const float *)X[cur], (const void *)(pending.gain ? Y : nullptr), pending.gain, dst, (const int32_t *)nullptr,
              (const float *)nullptr, (const float *)nullptr, (const int32_t *)nullptr, (void *)nullptr, (int32_t)W, (int32_t)1, (int32_t)0, (int32_t)W,
              (float)m->cfg.rms_eps);
   }

@@ -154,7 +154,8 @@ void RowEngineBase::linear(KernelCalls &k, const RowMatrix &mt, const char *Xp, 
   }
   const int n_tiles = (mt.N + 127) / 128, kb = (mt.K + 63) / 64;
   int nt = rows <= 16 ? 16 : rows <= 32 ? 32 : rows <= 64 ? 64 : 128;
-  if (rows > 128) {
+  const bool few = 2 * n_tiles * ((rows + 127) / 128) <= sm_count;   // tiles of 128 rows leave most SMs idle: split K instead
+  if (rows > 128 && !few) {
     // rows of a tile: as large as possible (operand traffic), but a launch lasts whole rounds of tiles over the SMs
     long best = -1;
     for (int t = 256; t >= 96; t -= 16) {
@@ -164,7 +165,7 @@ void RowEngineBase::linear(KernelCalls &k, const RowMatrix &mt, const char *Xp, 
   }
   const int tiles = n_tiles * ((rows + nt - 1) / nt);
   int splits = 1;   // few tiles: a cluster of blocks per tile, each a part of K
-  while (rows <= 128 && splits < 8 && tiles * splits * 2 <= sm_count && kb >= splits * 4) splits *= 2;
+  while ((rows <= 128 || few) && splits < 8 && tiles * splits * 2 <= sm_count && kb >= splits * 4) splits *= 2;
   TensorMap wm, xm;
   if (ainfer_tensor_map_bf16(dev, &wm, mt.w, (uint64_t)mt.N, (uint64_t)mt.K, (uint64_t)mt.ldw, 128) != AINFER_OK ||
       ainfer_tensor_map_bf16(dev, &xm, Xp, (uint64_t)rows, (uint64_t)mt.K, (uint64_t)ldx, (uint32_t)nt) != AINFER_OK) {

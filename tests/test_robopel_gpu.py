@@ -94,7 +94,7 @@ def test_output_norm_rows(dev, W, top, kind):
     x, g, fg = rn(R, W), rn(W), rn(W)
     place, pw = torch.full((R, max(top, 1)), -1, dtype=torch.int32), torch.rand(R, max(top, 1))
     if top:
-        y = rn(R * top, W)
+        y = rn(R * top, W) if kind == "f32" else bf16(rn(R * top, W)).float()
         perm = torch.randperm(R * top, generator=torch.Generator().manual_seed(1)).int().reshape(R, top)
         place = torch.where(torch.arange(R * top).reshape(R, top) % 3 == 1, torch.tensor(-1, dtype=torch.int32), perm)
         rows = torch.where((place >= 0)[..., None], y[place.clamp(min=0).long()], x[:, None, :].expand(R, top, W)).double()
@@ -105,14 +105,15 @@ def test_output_norm_rows(dev, W, top, kind):
     want = x.double() + P.rms(yy, eps, g.double())
     up = lambda t: dev.upload(f32(t))   # noqa: E731
     dx, xo, h = up(x), dev.zeros(R * W * 4), dev.zeros(R * ld * 4)
+    dy = dev.upload(bits(y)) if top and kind == "b16" else up(y)
     k = dev.kernel("PostNormRowsF32" if kind == "f32" else "PostNormRowsB16")
     tail = [dev.upload(place.numpy()), up(pw)]
-    k(R, dx, up(y), up(g), xo, *tail, 0, 0, h, W, R, top, ld, eps)
+    k(R, dx, dy, up(g), xo, *tail, 0, 0, h, W, R, top, ld, eps)
     dev.sync()
     close(dev.download(xo, (R, W), np.float32), want, 1e-5)
     close(down(dev, h, (R, ld), kind)[:, :W], want, 1e-5 if kind == "f32" else 1e-2)
     idx = np.int32([5, 0, 3])
-    k(3, dx, up(y), up(g), 0, *tail, up(fg), dev.upload(idx), h, W, 3, top, ld, eps)
+    k(3, dx, dy, up(g), 0, *tail, up(fg), dev.upload(idx), h, W, 3, top, ld, eps)
     dev.sync()
     close(down(dev, h, (R, ld), kind)[:3, :W], P.rms(want, eps, fg.double())[idx.tolist()], 1e-5 if kind == "f32" else 1e-2)
     k(R, dx, 0, 0, xo, *tail, 0, 0, h, W, R, 0, ld, eps)          # nothing pending: a copy
@@ -189,7 +190,7 @@ def test_recurrence_over_rows_and_steps(dev, K, kind):
     for n in (1, 31, 32, 33, 2, 64, 3, 40):
         du, dc, a = dev.upload(f32(u[at:at + n])), dev.upload(ctrl(range(at, at + n))), dev.zeros(n * lda * 4)
         ch = -(-n // 32)
-        dev.kernel("MinGruChunk")(cb * ch, du, st1, dc, pair, n, K)
+        dev.kernel("MinGruChunk" + sfx)(cb * ch, du, st1, dc, pair, n, K)
         dev.kernel("MinGruScan" + sfx)(cb * ch, du, pair, st1, dc, a, n, K, lda)
         got.append(down(dev, a, (n, lda), kind)[:, :K])
         at += n
