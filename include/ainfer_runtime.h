@@ -37,7 +37,7 @@ const char *ainfer_rt_last_error(void);
  * CRCs and trailing SHA-256 (docs/binfer_spec.md section 11). */
 int ainfer_binfer_validate(const char *path, int level);
 /* Writes a synthetic model of a named shape ("tiny", "mini", "mini-mtp",
- * "small", "full", "sinepel-tiny", "sinepel-small") on the host. Counterpart of tools/binfer.py cmd_quantize
+ * "small", "full", "sinepel-tiny", "sinepel-small", "robopel-tiny", "robopel-small") on the host. Counterpart of tools/binfer.py cmd_quantize
  * (:155-353) with seeded N(0, 0.02) weights in place of a checkpoint. */
 int ainfer_synth_write(const char *path, const char *preset, uint64_t seed);
 /* Checkpoint ingestion: a SafeTensors file, or a directory holding model.safetensors.index.json
@@ -89,9 +89,10 @@ enum {
 int ainfer_session_create(ainfer_model_t m, int max_ctx, int flags, ainfer_session_t *out);
 int ainfer_session_destroy(ainfer_session_t s);
 int ainfer_session_reset(ainfer_session_t s);
-/* Device buffers of the session, for state upload/download by tests (architectures with residual
- * streams: "shift", "conv", "Kc", all layers of each, "state" for the three together, and the common
- * "logits", "ctrl", "history", "layer_out"):
+/* Device buffers of the session, for state upload/download by tests (architectures with a row engine:
+ * "state", all of a session's state, and its parts, all layers of each: Sinepel "shift", "conv", "Kc",
+ * Robopel "gru", "Kc" (rings of keys and values), "means"; and the common "logits", "ctrl", "history",
+ * "layer_out"):
  * "conv", "S", "Kc", "Vc", "Ks", "Vs", "logits", "x", "ctrl", "layer_out",
  * "routed", "near_gap", "history", "stage_stamps". */
 int ainfer_session_buffer(ainfer_session_t s, const char *which, void **dptr, uint64_t *bytes);
@@ -181,7 +182,7 @@ int ainfer_ep_moe_stack(ainfer_ep_t ep, int first, int count, float *seg_ms);
 typedef struct ainfer_batch_s *ainfer_batch_t;
 enum { AINFER_BATCH_F32 = 32 /* as AINFER_SESSION_F32; beside AINFER_EP_ROUTER_BIAS in `flags` */ };
 /* A sequence whose control block says position 0 starts anew, whatever its slot held before. (Models
- * with residual streams; the INT4 hybrid's slots are zeroed by the caller.) */
+ * with a row engine; the INT4 hybrid's slots are zeroed by the caller.) */
 int ainfer_batch_create(ainfer_model_t m, const void *id128, int rank, int world, int batch, int max_ctx, int flags,
                         ainfer_batch_t *out);
 int ainfer_batch_destroy(ainfer_batch_t b);
