@@ -203,7 +203,7 @@ int ainfer_session_prefill_rows(ainfer_session_t h, int rows) {
 int ainfer_session_prefill_ep(ainfer_session_t h, const void *id128, int rank, int world) {
   if (!h) return set_err(2, "usage: null argument");
   Session *s = h->s;
-  if (s->rows && world > 1) return set_err(2, "usage: this architecture has no experts to split");
+  if (s->rows && world > 1) return set_err(2, "usage: only the INT4 hybrid splits experts over ranks");
   if (world < 1 || world > 64 || 64 % world || rank < 0 || rank >= world || (world > 1 && !id128))
     return set_err(2, "usage: 0 <= rank < world, world divides 64, and an id for more than one rank");
   if (s->prefill) { prefill_destroy(s->prefill); s->prefill = nullptr; }
@@ -267,7 +267,7 @@ int ainfer_ep_unique_id(void *out128) {
 }
 int ainfer_ep_create(ainfer_model_t m, const void *id128, int rank, int world, int batch, int flags, ainfer_ep_t *out) {
   if (!m || !out) return set_err(2, "usage: null argument");
-  if (m->m->rows) return set_err(2, "usage: this architecture has no experts");
+  if (m->m->rows) return set_err(2, "usage: the expert-parallel block is the INT4 hybrid's");
   *out = nullptr;
   ainfer_ep_s *h = new ainfer_ep_s;
   int r = h->e.create(m->m, id128, rank, world, batch, flags);

@@ -232,9 +232,9 @@ def _mixture_case(E, I, top, W, F, R):
 CASES = [(5, 2, 3, 40, 24, 70), (16, 0, 1, 50, 33, 9), (3, 1, 4, 64, 130, 40), (40, 8, 6, 128, 72, 200), (1, 0, 1, 16, 8, 3), (200, 56, 8, 64, 40, 33)]
 
 
-@pytest.mark.parametrize("kind", ["f32", "b16"])
-@pytest.mark.parametrize("E,I,top,W,F,R", CASES)
-def test_mixture_over_rows(dev, E, I, top, W, F, R, kind):
+@pytest.mark.parametrize("kind,nt", [("f32", 64), ("b16", 16), ("b16", 48), ("b16", 144), ("b16", 256)])
+@pytest.mark.parametrize("E,I,top,W,F,R", CASES + [(2, 1, 2, 40, 130, 400)])
+def test_mixture_over_rows(dev, E, I, top, W, F, R, kind, nt):
     x, logits, corr, up, dn = _mixture_case(E, I, top, W, F, R)
     s = torch.softmax(logits.double(), -1)
     idx = torch.topk(s + corr.double(), top, -1).indices
@@ -244,7 +244,7 @@ def test_mixture_over_rows(dev, E, I, top, W, F, R, kind):
     gs = dev.download(sel, (R, top), np.int32)
     assert np.array_equal(gs, idx.numpy())
     close(dev.download(sw, (R, top), np.float32), s.gather(1, idx), 1e-5)
-    nt, count = (64 if kind == "f32" else 16), dev.zeros(8)
+    count = dev.zeros(8)
     tiles = dev.zeros((R * top // 16 + E + 1) * 16)
     dev.kernel("MoePlanRows")(1, sel, place, rowof, tiles, count, R, top, E, nt)
     pl, ct = dev.download(place, (R, top), np.int32), dev.download(count, 2, np.int32)
